@@ -39,7 +39,7 @@
 extern "C" {
 #endif
 
-#define TGIS_ABI_VERSION 11
+#define TGIS_ABI_VERSION 12
 #define TGIS_MAX_REQUEST_ID 96
 #define TGIS_MAX_TOPN 12 /* reference forces max_logprobs >= 11: tgis_utils/args.py:214-216 */
 #define TGIS_MAX_STOP_TOKEN_IDS 8
@@ -94,6 +94,15 @@ typedef struct tgis_engine tgis_engine;
  *          no LoRA slots. */
 #define TGIS_ARCH_SIKAZEN 5
 
+/*   BISUZEN: a layer list as well (tgis_engine_create_spec), fp32 residual stream.  Every norm is elementwise with one slope,
+ *          dyt(x) = tanh(alpha x) * w + b, and sublayers are pre-normed: x += mixer(dyt1(x)); x += ff(dyt2(x))
+ *          (TGIS_STYLE_PRE_DYT).  A span of layers may run several passes in a row on the same weights, every pass with cache rows
+ *          and state of its own.  Mixers: windowed attention with kept first tokens and a sink beside lightning attention, both
+ *          outputs normed and averaged (TGIS_MIXER_WINDOW_LIGHTNING); chunked attention (TGIS_MIXER_POOLED_ATTENTION with `chunk`).
+ *          Feed-forward: gelu-gated (TGIS_MLP_DENSE_GELU) or experts with identity experts and a group-limited choice
+ *          (TGIS_MLP_MOE_GROUPED).  Logits times logit_scale.  bf16 or fp32 operands.  Single GPU, no LoRA slots. */
+#define TGIS_ARCH_BISUZEN 6
+
 /* Model + runtime configuration (bf16 decoder-only transformer; see TGIS_ARCH_*). */
 typedef struct tgis_config {
   int32_t abi_version; /* must be TGIS_ABI_VERSION */
@@ -144,18 +153,26 @@ typedef struct tgis_config {
 #define TGIS_MIXER_POOLED_ATTENTION 8 /* grouped-query softmax attention: rotary positions, unit-norm queries and keys, a window
                                        * of tokens and one mean key / value for every block of `pool` tokens behind it */
 #define TGIS_MIXER_HGRN 9            /* outer-product memory that writes with the complement of its forget gate (bounded below per channel) */
+#define TGIS_MIXER_WINDOW_LIGHTNING 10 /* left: grouped-query attention as TGIS_MIXER_POOLED_ATTENTION; right: lightning attention (an
+                                       * outer-product memory with one fixed decay per head); both outputs rms-normed over the
+                                       * width with a plain weight, averaged */
 #define TGIS_MLP_NONE 0
 #define TGIS_MLP_MOE 1
 #define TGIS_MLP_DENSE_GELU 2        /* down(gelu_tanh(gate h) * (up h)), width `ff` */
 #define TGIS_MLP_MOE_SIGMOID 3       /* experts down(relu(up (s h))^2) weighted on their input by s = sigmoid(router logit), the
                                       * `top` largest, their scores used as they are; shared expert of width shared_ff added (0: none) */
 #define TGIS_MLP_DENSE_SILU 4        /* down(silu(gate h) * (up h)), width `ff` */
+#define TGIS_MLP_MOE_GROUPED 5       /* experts down(gelu(up h)), exact gelu, plus `identity` experts whose output is their input; scores
+                                      * softmax over all of them, choice by score + correction among the best expert_groups_keep of
+                                      * expert_groups equal groups (a group counts as its best choice score), weights: the chosen
+                                      * scores divided by their sum */
 /* tgis_layer_spec.flags */
 #define TGIS_LAYER_ROT_INTERLEAVED 1 /* rotary pairs are (2i, 2i + 1) instead of (i, i + rot_dims / 2) */
 #define TGIS_LAYER_SINK 2            /* the softmax denominator of head h also holds exp(sink_h): "l<i>.mix.sink" */
 #define TGIS_LAYER_NO_OUT_GATE 4     /* latent attention without the sigmoid output gate (no "l<i>.mix.g") */
 #define TGIS_LAYER_QKV_BIAS 8        /* "l<i>.mix.q.b|k.b|v.b" are added to the projections */
 #define TGIS_LAYER_UNIT_QK 16        /* queries and keys are divided by their root mean square per head after the rotation */
+#define TGIS_LAYER_OUT_BIAS 32       /* the attention's output projection has a bias: "o.b" */
 typedef struct tgis_layer_spec {
   int32_t mixer;        /* TGIS_MIXER_* */
   int32_t heads, dim, rot_dim, vdim, kv_rank, q_rank; /* per head: dim unrotated + rot_dim rotated query/key dims, vdim values */
@@ -198,7 +215,16 @@ typedef struct tgis_layer_spec {
   int32_t pool;
   float rot_linear;
   int32_t flags;
+  /* TGIS_MIXER_POOLED_ATTENTION and the attention of TGIS_MIXER_WINDOW_LIGHTNING: keep_first > 0: the window's queries also see the
+   * first keep_first positions of the sequence (no pooled blocks then); chunk > 0: a query sees only keys of its own chunk of
+   * `chunk` positions, counted from position 0 */
+  int32_t keep_first, chunk;
+  /* TGIS_MLP_MOE_GROUPED: experts, top, expert_ff as above; identity experts come after the others in the router's outputs */
+  int32_t identity, expert_groups, expert_groups_keep;
   int32_t reserved2;
+  /* TGIS_MIXER_WINDOW_LIGHTNING, right side: mm_heads heads, queries / keys of mm_dim, values of mm_vdim; decay [mm_heads] (host
+   * memory, read by tgis_engine_create_spec) */
+  const float* decay;
 } tgis_layer_spec;
 #define TGIS_STYLE_POST_NORM 1 /* x += rmsnorm(sublayer(x)) * w with a plain weight; unset: pre- and post-norm, weights stored
                                 * as deviations from one */
@@ -206,6 +232,8 @@ typedef struct tgis_layer_spec {
 #define TGIS_STYLE_PARALLEL_GATED 4 /* one norm per layer; x += sigmoid(R1 n + b1) * mixer(shift(n)) + sigmoid(R2 n + b2) * ff(n) */
 #define TGIS_STYLE_PARALLEL_PAIR 8  /* two norms of ONE number each; x += mixer(rms(x) g1) + ff(rms(x) g2), then the per-layer token
                                      * input (side_dim > 0): x += rms(side.proj (gelu_tanh(side.gate x) * e)) * side.norm */
+#define TGIS_STYLE_PRE_DYT 16       /* every norm is tanh(alpha x) * w + b ("<norm>", "<norm>.b", "<norm>.alpha"); x += mixer(dyt1(x)), then
+                                     * x += ff(dyt2(x)) */
 #define TGIS_DTYPE_BF16 0 /* bf16 operands, fp32 accumulation; norms, softmax, routers and the residual sum in fp32 */
 #define TGIS_DTYPE_F32 1  /* everything in true fp32 (no TF32) */
 typedef struct tgis_model_spec {
@@ -220,9 +248,10 @@ typedef struct tgis_model_spec {
   int32_t side_dim;     /* TGIS_STYLE_PARALLEL_PAIR: columns of the side table "side.embed" [vocab, n_layers * side_dim] that layer i
                            reads at [i * side_dim, (i + 1) * side_dim); 0: no per-layer token input */
   /* layers [loop_start, loop_stop) run loop_times passes in a row on the same weights, every pass with cache rows and state of
-   * its own; before every pass but the first the embedding output is added to the stream.  loop_times <= 1: no loop */
+   * its own; loop_add_embed != 0: before every pass but the first the embedding output is added to the stream.  loop_times <= 1: no
+   * loop */
   int32_t loop_start, loop_stop, loop_times;
-  int32_t reserved;
+  int32_t loop_add_embed;
 } tgis_model_spec;
 
 /* What the adapter's proto->SamplingParams mapping (grpc_server.py:508-628) hands to the engine. */
@@ -339,6 +368,9 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
 /* cfg->arch == TGIS_ARCH_SIKAZEN; parameter names: "embed", "side.embed", "head", "final.norm" (one number), "l<i>.norm1|norm2" (one
  * number each), "l<i>.mlp.gate|up|down", "l<i>.side.gate|proj|norm"; TGIS_MIXER_POOLED_ATTENTION "l<i>.mix.q|q.b|k|k.b|v|v.b|o";
  * TGIS_MIXER_LATENT_ATTENTION "l<i>.mix.dq|dq.norm|uq|dkv|dkv.norm|uk|uv|sink|o"; TGIS_MIXER_HGRN "l<i>.mix.q|f|f.b|lower|v|norm|o". */
+/* cfg->arch == TGIS_ARCH_BISUZEN; parameter names: "embed", "head", every norm as "<norm>|<norm>.b|<norm>.alpha" (alpha: one number):
+ * "final.norm", "l<i>.norm1|norm2"; "l<i>.mlp.gate|up|down" or "l<i>.mlp.router|correction|e<j>.up|e<j>.down"; TGIS_MIXER_POOLED_ATTENTION
+ * "l<i>.mix.q|k|v|o"; TGIS_MIXER_WINDOW_LIGHTNING "l<i>.mix.left.q|q.b|k|k.b|v|v.b|sink|o|o.b|out", "l<i>.mix.right.q|k|v|g|norm|o|out". */
 /* name: HF Llama parameter name ("model.layers.3.self_attn.q_proj.weight", "lm_head.weight", ...) or
  * "tgis.rope_cos_sin" ([max_model_len,128] bf16 = cos|sin); arch OPT: HF OPT parameter names
  * ("model.decoder.layers.3.self_attn.q_proj.bias", "model.decoder.embed_positions.weight" with >= max_model_len + 2 rows,

@@ -142,6 +142,15 @@ int tgis_k_latent_attn(const float* q_abs, const void* cache, int32_t dt, const 
                        const tgis_k_latent_geom* g);
 int tgis_k_moe_route(const float* logits, int32_t ld, const float* bias, int32_t E, int32_t top, int32_t* ids, float* w,
                      float* side_gate, int32_t T);
+/* scores softmax(logits) over E outputs, the `top` largest of score + bias among the `keep` best of `groups` equal groups; w: the chosen
+ * scores over their sum */
+int tgis_k_moe_route_grouped(const float* logits, int32_t ld, const float* bias, int32_t E, int32_t top, int32_t groups, int32_t keep,
+                             int32_t* ids, float* w, int32_t T);
+/* csrc/elementwise.cu dyt_tail_kernel (csrc/kernels.h DytTail): in / next are (w [hidden], b [hidden], alpha [1]) triples */
+int tgis_k_dyt_tail(const float* y_main, const float* b_main, const float* y_pair, const float* w_main, const float* w_pair, float eps,
+                    const float* y_rows, const int32_t* inv, const int32_t* ids, const float* mix_w, int32_t top, int32_t n_experts,
+                    const float* in_w, const float* in_b, const float* in_alpha, float* resid, const float* w, const float* b,
+                    const float* alpha, float out_scale, void* out, int32_t out_dt, int32_t T, int32_t hidden);
 int tgis_k_moe_align(const int32_t* ids, int32_t T, int32_t top, int32_t E, int32_t* seg_off, int32_t* order, int32_t* inv);
 
 /* ---- softcapped grouped-query attention (csrc/attention_capped.cu) ---- */
@@ -171,6 +180,8 @@ typedef struct tgis_k_poolattn_geom {
   int32_t heads, kv_heads, dim, vdim, window, pool, rot_dims;
   float scale;
   int32_t unit_norm;
+  int32_t keep_first, chunk, rot_interleaved;   /* the first keep_first tokens stay visible behind the window; chunks of `chunk` positions */
+  const float* sink;                            /* device, fp32 [heads], or NULL */
 } tgis_k_poolattn_geom;
 /* y fp32 [T, ldy] = [.. q .. k .. v ..] at the given columns (+ bias [q | k | v] or NULL) -> rotated, unit-normed queries and
  * cache rows at slots[t] */
@@ -216,6 +227,11 @@ int tgis_k_outer_scan(int32_t mode, const float* q, const float* k, const float*
                       const float* fg, int32_t ldg, const float* ig_b, const float* fg_b, float gate_cap, float* S, float* n,
                       float* m, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const float* x, float* x_last,
                       int32_t width, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot);
+/* lightning attention: S <- decay_h S + silu(k) silu(v)^T, o = S^T silu(q); q, k [T, heads * dim], v [T, heads * vdim], decay device
+ * [heads], S [slots][heads][dim][vdim] */
+int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_t ldq, int32_t ldk, int32_t ldv, const float* decay,
+                          float* S, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const int32_t* seqs_host,
+                          int32_t n_seqs, const int32_t* tok_slot);
 int tgis_k_head_norm_gate(const float* o, int32_t ldo, int32_t heads, int32_t vdim, const float* w, const float* gate, int32_t ldg,
                           int32_t act, float eps, void* out, int32_t out_dt, int32_t T);
 /* resid += rmsnorm((rmsnorm(y_main) * w_main + rmsnorm(y_pair) * w_pair) / 2) * w_post; out = rmsnorm(resid) * w_pre, or the

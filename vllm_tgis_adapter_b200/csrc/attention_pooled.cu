@@ -1,9 +1,12 @@
-// Grouped-query softmax attention over a sliding window of tokens plus pooled blocks of the tokens that left it
-// (kernels.h: PoolAttnGeom).  A query at position i sees
+// Grouped-query softmax attention over a sliding window of tokens plus pooled blocks of the tokens that left it, over a window plus
+// the first tokens of the sequence, or inside chunks (kernels.h: PoolAttnGeom).  With a window and pooled blocks, a query at position i sees
 //   * the tokens j with 0 <= i - j < window, each with its own key and value, and
 //   * every block b of `pool` consecutive positions with b * pool + pool - 1 <= i - window through ONE key and ONE value: the
 //     means of the block's cached keys (after rotation and norm) and values,
-// all under one softmax.  Tokens behind the window whose block is still incomplete at i - window are not seen at all.
+// all under one softmax.  Tokens behind the window whose block is still incomplete at i - window are not seen at all.  Without
+// pooled blocks it may see, beside the window, the tokens j < keep_first; with chunks it sees only tokens of its own chunk.  A sink
+// is one more term of the softmax's denominator: the running state (maximum, sum) starts as if one key of that score and of
+// weight but without a value had been seen.
 //
 //   poolattn_prep_kernel   per token and head: bias, rotary turn (fp32 table), unit RMS norm of queries and keys, cache write
 //   poolattn_pool_kernel   the blocks that this step's tokens complete: mean of the block's cache rows -> the pooled cache
@@ -11,8 +14,9 @@
 //   poolattn_kernel        any sizes and fp32 rows (FMA pipe)
 //
 // The attention kernels take one CTA per (tile of POOLATTN_TILE query tokens of one sequence, query head) and walk "chunks" of
-// 32 keys in a fixed order: first the pooled rows 0..31, 32..63, ... that the tile's last query sees, then the sequence's
-// 32-token cache blocks from the first one the tile's window touches.  Scores, the running softmax (maximum, sum) and the
+// 32 keys in a fixed order: first the pooled rows 0..31, 32..63, ... that the tile's last query sees, or the cache blocks of the
+// first keep_first tokens as far as they lie before the window, then the sequence's 32-token cache blocks from the first one the
+// tile's window (or chunk) touches.  Scores, the running softmax (maximum, sum) and the
 // accumulators are fp32; a key that a query does not see weighs exactly zero.  So a query row's arithmetic depends on its own
 // position and on the 32-row grids of its sequence only: not on the tile it shares with other queries, on how the prompt was cut,
 // on the other sequences of the step, or on which physical pages hold the rows.
@@ -53,6 +57,13 @@ __device__ __forceinline__ int pooled_visible(int pos, int window, int pool) {
   const int e = pos - window + 1;   // positions [0, e) lie behind the window
   return (window > 0 && pool > 0 && e > 0) ? e / pool : 0;
 }
+// What a query at position `pos` sees token by token: the keys j <= pos with j >= lo or j < keep
+struct Visible { int lo, keep; };
+__device__ __forceinline__ Visible visible_tokens(int pos, const PoolAttnGeom& g) {
+  const int cl = g.chunk > 0 ? pos / g.chunk * g.chunk : 0;   // first position of the query's chunk
+  const int wl = g.window > 0 ? max(0, pos - g.window + 1) : 0;
+  return {max(cl, wl), cl > 0 ? 0 : g.keep_first};
+}
 // row of pooled block b inside the pooled cache (page table bt of the sequence)
 __device__ __forceinline__ size_t pooled_row(int b, int pool, int rpp, const int32_t* bt) {
   const int page = (int)(((long long)b * pool) / KV_BLOCK);
@@ -92,9 +103,10 @@ poolattn_prep_kernel(const float* __restrict__ y, int ldy, int q_off, int k_off,
       if (i < g.dim) {
         v = src[i] + (b ? b[i] : 0.f);
         if (i < g.rot_dims) {
-          const int j = i < half ? i + half : i - half, f = i < half ? i : i - half;
+          const bool first = g.rot_interleaved ? (i & 1) == 0 : i < half;   // of its pair; the partner is j, the angle's index f
+          const int j = g.rot_interleaved ? i ^ 1 : (first ? i + half : i - half), f = g.rot_interleaved ? i >> 1 : (first ? i : j);
           const float w = src[j] + (b ? b[j] : 0.f);
-          v = i < half ? v * cs[f] - w * cs[half + f] : v * cs[f] + w * cs[half + f];
+          v = first ? v * cs[f] - w * cs[half + f] : v * cs[f] + w * cs[half + f];
         }
       }
       val[e] = v;
@@ -212,29 +224,33 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
     for (int cc = 0; cc < PA_CC; ++cc) acc[qi][cc] = 0.f;
   float m_run[4], l_run[4];   // this warp's four query rows (valid in every lane)
   int n_vis[4];               // pooled blocks each of them sees
+  Visible vis[4];             // ... and tokens
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    m_run[i] = -INFINITY;
-    l_run[i] = 0.f;
+    m_run[i] = g.sink != nullptr ? g.sink[h] : -INFINITY;
+    l_run[i] = g.sink != nullptr ? 1.f : 0.f;
+    vis[i] = visible_tokens(pos0 + warp * 4 + i, g);
     n_vis[i] = pooled_visible(pos0 + warp * 4 + i, g.window, g.pool);
   }
   const int n_pooled = pooled_visible(pos_last, g.window, g.pool);
-  const int n_pc = (n_pooled + KV_BLOCK - 1) / KV_BLOCK;
-  const int kmin = g.window > 0 ? max(0, pos0 - g.window + 1) : 0;
-  const int blk0 = kmin / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
+  const Visible first = visible_tokens(pos0, g);
+  const int blk0 = first.lo / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
+  // chunks in front of the window's blocks: pooled rows, or the blocks of the kept first tokens
+  const int n_pc = g.pool > 0 ? (n_pooled + KV_BLOCK - 1) / KV_BLOCK : min((first.keep + KV_BLOCK - 1) / KV_BLOCK, blk0);
   const int n_chunks = n_pc + blk1 - blk0 + 1;
   const int rpp = g.rows_per_page();
   const int32_t* bt = block_table + (size_t)sq.block_row * bt_stride;
   for (int c = 0; c < n_chunks; ++c) {
-    const bool pooled = c < n_pc;
+    const bool pooled = g.pool > 0 && c < n_pc;
+    const int blk = c < n_pc ? c : blk0 + c - n_pc;   // pooled chunk, or cache block of the sequence
     __syncthreads();   // the previous chunk's Ks / Vs / Ps / rowoff are consumed (first pass: Qs complete)
     if (tid < KV_BLOCK) {
       long long r;
       if (pooled) {
-        const int b = c * KV_BLOCK + tid;
+        const int b = blk * KV_BLOCK + tid;
         r = b < n_pooled ? (long long)pooled_row(b, g.pool, rpp, bt) : -1;
       } else {
-        r = (long long)bt[blk0 + c - n_pc] * KV_BLOCK + tid;
+        r = (long long)bt[blk] * KV_BLOCK + tid;
       }
       rowoff[tid] = r;
     }
@@ -261,11 +277,11 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
 #pragma unroll
       for (int i = 0; i < 4; ++i) s[i] = fmaf(qr[i * d + kk], kv, s[i]);
     }
-    const int kidx = (pooled ? c : blk0 + c - n_pc) * KV_BLOCK + lane;   // pooled block number, or token position
+    const int kidx = blk * KV_BLOCK + lane;   // pooled block number, or token position
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int qi = warp * 4 + i, pi = pos0 + qi;
-      const bool ok = qi < nq && (pooled ? kidx < n_vis[i] : (kidx <= pi && (g.window <= 0 || pi - kidx < g.window)));
+      const bool ok = qi < nq && (pooled ? kidx < n_vis[i] : (kidx <= pi && (kidx >= vis[i].lo || kidx < vis[i].keep)));
       const float sc = ok ? s[i] : -INFINITY;
       const float m_new = fmaxf(m_run[i], warp_max_f(sc));
       const float p = ok ? expf(sc - m_new) : 0.f;
@@ -388,12 +404,21 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
   for (int j = 0; j < MMA_NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_part[2] = {0.f, 0.f};   // rows gq and gq + 8
+  if (g.sink != nullptr) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      m_run[r] = g.sink[h_base + (gq + r * 8) % gs];
+      l_part[r] = (warp == 0 && (lane & 3) == 0) ? 1.f : 0.f;   // (the row's sum adds up the parts of all its threads)
+    }
+  }
   const int tqr[2] = {gq / gs, (gq + 8) / gs};   // tokens of this thread's two rows
+  const Visible vis[2] = {visible_tokens(pos0 + tqr[0], g), visible_tokens(pos0 + tqr[1], g)};
   const int n_vis[2] = {pooled_visible(pos0 + tqr[0], g.window, g.pool), pooled_visible(pos0 + tqr[1], g.window, g.pool)};
   const int n_pooled = pooled_visible(pos_last, g.window, g.pool);
-  const int n_pc = (n_pooled + KV_BLOCK - 1) / KV_BLOCK;
-  const int kmin = g.window > 0 ? max(0, pos0 - g.window + 1) : 0;
-  const int blk0 = kmin / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
+  const Visible first = visible_tokens(pos0, g);
+  const int blk0 = first.lo / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
+  // chunks in front of the window's blocks: pooled rows, or the blocks of the kept first tokens
+  const int n_pc = g.pool > 0 ? (n_pooled + KV_BLOCK - 1) / KV_BLOCK : min((first.keep + KV_BLOCK - 1) / KV_BLOCK, blk0);
   const int n_chunks = n_pc + blk1 - blk0 + 1;
   const int rpp = g.rows_per_page();
   const int32_t* bt = block_table + (size_t)sq.block_row * bt_stride;
@@ -403,13 +428,14 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   const int fj = tid >> 2, fl = tid & 3;
   auto fetch = [&](int c) {
     if (c < n_chunks) {
-      const bool pooled = c < n_pc;
+      const bool pooled = g.pool > 0 && c < n_pc;
+      const int blk = c < n_pc ? c : blk0 + c - n_pc;   // pooled chunk, or cache block of the sequence
       long long r;
       if (pooled) {
-        const int b = c * KV_BLOCK + fj;
+        const int b = blk * KV_BLOCK + fj;
         r = b < n_pooled ? (long long)pooled_row(b, g.pool, rpp, bt) : -1;
       } else {
-        r = (long long)bt[blk0 + c - n_pc] * KV_BLOCK + fj;
+        r = (long long)bt[blk] * KV_BLOCK + fj;
       }
       bf* Kd = Ks2 + ((size_t)(c % PA_NST) * KV_BLOCK + fj) * LDK;
       bf* Vd = Vs2 + ((size_t)(c % PA_NST) * KV_BLOCK + fj) * LDV;
@@ -428,7 +454,8 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
   for (int c = 0; c < PA_NST - 1; ++c) fetch(c);
   for (int c = 0; c < n_chunks; ++c) {
-    const bool pooled = c < n_pc;
+    const bool pooled = g.pool > 0 && c < n_pc;
+    const int blk = c < n_pc ? c : blk0 + c - n_pc;
     // the stage that chunk c + PA_NST - 1 goes to was last read in the previous pass, which ended with a barrier
     fetch(c + PA_NST - 1);
     asm volatile("cp.async.wait_group %0;\n" ::"n"(PA_NST - 1) : "memory");
@@ -448,8 +475,8 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int r = e >> 1, pi = pos0 + tqr[r];
-      const int kidx = (pooled ? c : blk0 + c - n_pc) * KV_BLOCK + warp * 8 + t2 + (e & 1);   // pooled block number, or token position
-      ok[e] = tqr[r] < nq && (pooled ? kidx < n_vis[r] : (kidx <= pi && (g.window <= 0 || pi - kidx < g.window)));
+      const int kidx = blk * KV_BLOCK + warp * 8 + t2 + (e & 1);   // pooled block number, or token position
+      ok[e] = tqr[r] < nq && (pooled ? kidx < n_vis[r] : (kidx <= pi && (kidx >= vis[r].lo || kidx < vis[r].keep)));
       sc[e] = ok[e] ? sc[e] * g.scale : -INFINITY;
     }
     float mx[2] = {fmaxf(sc[0], sc[1]), fmaxf(sc[2], sc[3])};
@@ -559,7 +586,8 @@ cudaError_t launch_fma(const void* q, const void* k_cache, const void* v_cache, 
 
 bool geom_ok(const PoolAttnGeom& g) {
   return g.heads >= 1 && g.kv_heads >= 1 && g.heads % g.kv_heads == 0 && g.heads <= 65535 && g.dim >= 1 && g.vdim >= 1 &&
-         g.dim <= PREP_MAX_DIM && g.vdim <= POOLATTN_MAX_VDIM && g.rot_dims >= 0 && g.rot_dims <= g.dim && (g.rot_dims & 1) == 0;
+         g.dim <= PREP_MAX_DIM && g.vdim <= POOLATTN_MAX_VDIM && g.rot_dims >= 0 && g.rot_dims <= g.dim && (g.rot_dims & 1) == 0 &&
+         (g.pool <= 0 || (g.keep_first <= 0 && g.chunk <= 0));
 }
 
 }  // namespace

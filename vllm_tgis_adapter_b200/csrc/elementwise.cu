@@ -898,6 +898,104 @@ cudaError_t gated_tail_launch(const GatedTail& a, int T, int hidden, cudaStream_
   return launch_k(gated_tail_kernel<1>, dim3(T), dim3(NORM_THREADS), (size_t)hidden * sizeof(float), stream, a, hidden, T);
 }
 
+// ---- sublayers of a stream whose norms are elementwise (kernels.h: DytTail) ----
+template <int VEC>
+__device__ __forceinline__ FV<VEC> dyt_fv(const DytNorm& n, float alpha, const FV<VEC>& x, int i) {
+  const FV<VEC> w = ld_fv<VEC>(n.w + i), b = ld_fv<VEC>(n.b + i);
+  FV<VEC> r;
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) r.v[e] = fmaf(tanhf(alpha * x.v[e]), w.v[e], b.v[e]);
+  return r;
+}
+template <int VEC>
+__global__ void __launch_bounds__(NORM_THREADS) dyt_tail_kernel(DytTail a, int hidden) {
+  __shared__ float red[NORM_THREADS / 32];
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x;
+  const size_t base = (size_t)t * hidden;
+  float rs_a = 1.f, rs_b = 1.f;
+  if (a.y_pair != nullptr) {   // two mixers side by side: each output is normed by itself
+    float sa = 0.f, sb = 0.f;
+    for (int i = threadIdx.x * VEC; i < hidden; i += NORM_THREADS * VEC) {
+      FV<VEC> ya = ld_fv<VEC>(a.y_main + base + i);
+      const FV<VEC> yb = ld_fv<VEC>(a.y_pair + base + i);
+      if (a.b_main != nullptr) {
+        const FV<VEC> b = ld_fv<VEC>(a.b_main + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) ya.v[e] += b.v[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) {
+        sa = fmaf(ya.v[e], ya.v[e], sa);
+        sb = fmaf(yb.v[e], yb.v[e], sb);
+      }
+    }
+    rs_a = 1.f / sqrtf(block_sum<NORM_THREADS>(sa, red) / (float)hidden + a.eps);
+    rs_b = 1.f / sqrtf(block_sum<NORM_THREADS>(sb, red) / (float)hidden + a.eps);
+  }
+  const float alpha_in = a.in.alpha != nullptr ? *a.in.alpha : 0.f, alpha = *a.next.alpha;
+  for (int i = threadIdx.x * VEC; i < hidden; i += NORM_THREADS * VEC) {
+    FV<VEC> x = ld_fv<VEC>(a.resid + base + i);
+    if (a.y_main != nullptr) {
+      FV<VEC> y = ld_fv<VEC>(a.y_main + base + i);
+      if (a.b_main != nullptr) {
+        const FV<VEC> b = ld_fv<VEC>(a.b_main + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y.v[e] += b.v[e];
+      }
+      if (a.y_pair != nullptr) {
+        const FV<VEC> yb = ld_fv<VEC>(a.y_pair + base + i), wa = ld_fv<VEC>(a.w_main + i), wb = ld_fv<VEC>(a.w_pair + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y.v[e] = 0.5f * (y.v[e] * rs_a * wa.v[e] + yb.v[e] * rs_b * wb.v[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x.v[e] += y.v[e];
+      st_fv<VEC>(a.resid + base + i, x);
+    } else if (a.y_rows != nullptr) {
+      FV<VEC> y;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) y.v[e] = 0.f;
+      for (int k = 0; k < a.top; ++k) {   // fixed k order
+        const size_t tk = (size_t)t * a.top + k;
+        const float w = a.mix_w[tk];
+        const FV<VEC> r = a.ids[tk] < a.n_experts ? ld_fv<VEC>(a.y_rows + (size_t)a.inv[tk] * hidden + i) : dyt_fv<VEC>(a.in, alpha_in, x, i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(w, r.v[e], y.v[e]);
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) x.v[e] += y.v[e];
+      st_fv<VEC>(a.resid + base + i, x);
+    }
+    FV<VEC> n = dyt_fv<VEC>(a.next, alpha, x, i);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) n.v[e] *= a.out_scale;
+    if (VEC == 4 && a.out_dtype == DT_BF16) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(n.v[0], n.v[1 % VEC]), hi = __floats2bfloat162_rn(n.v[2 % VEC], n.v[3 % VEC]);
+      uint2 pk;
+      pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+      pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + base + i) = pk;
+    } else {
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) st_dt(a.out, a.out_dtype, base + i + e, n.v[e]);
+    }
+  }
+}
+cudaError_t dyt_tail_launch(const DytTail& a, int T, int hidden, cudaStream_t stream) {
+  if (T <= 0) return cudaSuccess;
+  const bool next_ok = a.next.w != nullptr && a.next.b != nullptr && a.next.alpha != nullptr;
+  if (a.resid == nullptr || a.out == nullptr || !next_ok || (a.y_pair != nullptr && (a.y_main == nullptr || a.w_main == nullptr || a.w_pair == nullptr)) ||
+      (a.y_rows != nullptr && (a.y_main != nullptr || a.inv == nullptr || a.ids == nullptr || a.mix_w == nullptr || a.top < 1 ||
+                               a.in.w == nullptr || a.in.b == nullptr || a.in.alpha == nullptr)))
+    return cudaErrorInvalidValue;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  const bool vec = hidden % 4 == 0 && al16(a.y_main) && al16(a.b_main) && al16(a.y_pair) && al16(a.w_main) && al16(a.w_pair) && al16(a.y_rows) &&
+                   al16(a.in.w) && al16(a.in.b) && al16(a.resid) && al16(a.next.w) && al16(a.next.b) && al16(a.out);
+  if (vec) return launch_k(dyt_tail_kernel<4>, dim3(T), dim3(NORM_THREADS), 0, stream, a, hidden);
+  return launch_k(dyt_tail_kernel<1>, dim3(T), dim3(NORM_THREADS), 0, stream, a, hidden);
+}
+
 __global__ void gather_rows_any_kernel(const int32_t* __restrict__ idx, const uint8_t* __restrict__ x,
                                        uint8_t* __restrict__ out, int row_bytes) {
   griddep_launch();

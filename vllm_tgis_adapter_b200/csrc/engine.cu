@@ -238,6 +238,7 @@ struct tgis_engine {
   bool pnx_on = false;
   tgis_model_spec pnx_spec{};
   std::vector<tgis_layer_spec> pnx_layer_specs;
+  std::vector<std::vector<float>> pnx_decays;        // per layer: tgis_layer_spec.decay
   struct PnxLayer {
     tgis_layer_spec sp{};
     LatentGeom g{};
@@ -287,9 +288,16 @@ struct tgis_engine {
     float* side_norm = nullptr;
     int weights_of = -1;              // the layer of the checkpoint whose weights this run uses
     bool add_x0 = false;              // the embedding output is added to the stream right before this run
+    // ---- layers of the dyt style (TGIS_ARCH_BISUZEN): elementwise norms before both sublayers.  Attention: pa, w_in, in_bias, sink, w_o,
+    // k_cache / v_cache; lightning side: c_mq .. c_mg, w_o2, mm_norm, st_S, out_l / out_r; experts: w_router, router_b (correction),
+    // w_gu_e (up-projections), w_d_e
+    DytNorm dyt1{}, dyt2{};
+    float *o_bias = nullptr, *decay = nullptr;       // [width] output bias of the attention; [mm_heads] decays
     int c_f = 0;                      // TGIS_MIXER_HGRN (w_in: q | f | v): column of the gate logits
   };
-  std::vector<PnxLayer> pair_runs;    // parallel pair style: one entry per layer RUN (a looped span repeats), weights shared
+  std::vector<PnxLayer> layer_runs;    // styles with loops (pair, dyt): one entry per layer RUN (a looped span repeats), weights shared
+  bool dyt_style = false;             // TGIS_STYLE_PRE_DYT
+  DytNorm pnx_final_dyt{};
   bool pair_style = false;            // TGIS_STYLE_PARALLEL_PAIR
   void *pnx_side = nullptr, *pnx_hB = nullptr;       // side table [vocab, n_layers * side_dim]; norm2's rows (operand type)
   float* pnx_x0 = nullptr;                           // the embedding output, kept for the passes of a loop
@@ -528,7 +536,8 @@ struct tgis_engine {
     Fl = c.ffn / tp;
     Vl = c.vocab / tp;
     opt = c.arch == TGIS_ARCH_OPT;
-    pnx_on = c.arch == TGIS_ARCH_PONENEX || c.arch == TGIS_ARCH_FALERAX || c.arch == TGIS_ARCH_REVEPEL || c.arch == TGIS_ARCH_SIKAZEN;  // the layer-list architectures
+    pnx_on = c.arch == TGIS_ARCH_PONENEX || c.arch == TGIS_ARCH_FALERAX || c.arch == TGIS_ARCH_REVEPEL || c.arch == TGIS_ARCH_SIKAZEN ||
+             c.arch == TGIS_ARCH_BISUZEN;  // the layer-list architectures
     if (pnx_on) logits_bf16 = false;  // fp32 logits straight from the accumulators
     model_head_dim = opt ? c.head_dim : HEAD_DIM;
     attn_scale = 1.0f / std::sqrt((float)model_head_dim);  // zero-padded head dims add nothing to q . k
@@ -1198,7 +1207,7 @@ struct tgis_engine {
   }
 
   // ------------------------------------------------------------------------------------------------ layer-list models
-  // TGIS_ARCH_PONENEX / TGIS_ARCH_FALERAX.  Scheduler, sequence slots, block manager, step metadata, lm_head rows, sampler and CUDA-graph
+  // TGIS_ARCH_PONENEX and the families after it.  Scheduler, sequence slots, block manager, step metadata, lm_head rows, sampler and CUDA-graph
   // replay are the engine's; what differs is the layer stack (pnx_forward) and the per-layer cache of latent rows, which
   // is paged with the same block ids as every other model's KV cache.
   template <class T>
@@ -1249,6 +1258,12 @@ struct tgis_engine {
     return d;
   }
 
+  DytNorm alloc_dyt(size_t W) { return DytNorm{pnx_alloc<float>(W), pnx_alloc<float>(W), pnx_alloc<float>(1)}; }
+  // mixers whose attention keeps paged keys and values per layer run
+  static bool run_has_kv(const tgis_layer_spec& s) {
+    return s.mixer == TGIS_MIXER_POOLED_ATTENTION || s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
+  }
+
   void init_pnx() {
     const tgis_config& c = cfg;
     const size_t W = c.hidden, V = c.vocab, T = std::max(T_max, 256);
@@ -1260,10 +1275,15 @@ struct tgis_engine {
     tied_head = (pnx_spec.style & TGIS_STYLE_TIED_HEAD) != 0;
     gated_style = (pnx_spec.style & TGIS_STYLE_PARALLEL_GATED) != 0;
     pair_style = (pnx_spec.style & TGIS_STYLE_PARALLEL_PAIR) != 0;
+    dyt_style = (pnx_spec.style & TGIS_STYLE_PRE_DYT) != 0;
     pnx_embed = pnx_alloc_dt(V * W);
     pnx_head = tied_head ? pnx_embed : pnx_alloc_dt(V * W);
     pnx_final_norm = pnx_alloc<float>(W);
     pnx_expected_tensors = tied_head ? 2 : 3;
+    if (dyt_style) {
+      pnx_final_dyt = alloc_dyt(W);
+      pnx_expected_tensors += 2;  // final.norm.b, final.norm.alpha
+    }
     size_t m_f1 = 1, m_f2 = 1, m_f3 = 1, m_mix = 1;
     size_t m_down = 1, m_qr = 1, m_q = 1, m_qabs = 1, m_olat = 1, m_ov = 1, m_heads = 1, m_E = 1, m_top = 1, m_ff = 1, m_ffs = 1;
     size_t cache_row_bytes = 0;
@@ -1273,7 +1293,7 @@ struct tgis_engine {
       PnxLayer& l = pnx_layers[i];
       const tgis_layer_spec& s = pnx_layer_specs[i];
       l.sp = s;
-      if (pair_style) {   // weights only: cache rows and state belong to the layer RUNS (pair_runs, below)
+      if (pair_style) {   // weights only: cache rows and state belong to the layer RUNS (layer_runs, below)
         const size_t sd = pnx_spec.side_dim;
         l.weights_of = (int)i;
         l.norm1 = pnx_alloc<float>(W);
@@ -1348,6 +1368,73 @@ struct tgis_engine {
           m_heads = std::max<size_t>(m_heads, s.heads);
           pnx_tile_tokens = std::min(pnx_tile_tokens, latent_tile_tokens(s.heads));
         }
+        continue;
+      }
+      if (dyt_style) {   // weights only, as above
+        l.weights_of = (int)i;
+        l.dyt1 = alloc_dyt(W);
+        pnx_expected_tensors += 3;
+        if (s.mlp != TGIS_MLP_NONE) {
+          l.dyt2 = alloc_dyt(W);
+          pnx_expected_tensors += 3;
+        }
+        if (s.mlp == TGIS_MLP_DENSE_GELU) {
+          l.w_gu = pnx_alloc_dt((size_t)2 * s.ff * W);
+          l.w_d = pnx_alloc_dt(W * s.ff);
+          pnx_expected_tensors += 3;  // mlp.gate, mlp.up, mlp.down
+          m_ffs = std::max<size_t>(m_ffs, s.ff);
+        } else if (s.mlp == TGIS_MLP_MOE_GROUPED) {
+          const size_t E = s.experts, n_out = E + s.identity, ff = s.expert_ff;
+          l.w_router = pnx_alloc_dt(n_out * W);
+          l.router_b = pnx_alloc<float>(n_out);
+          l.w_gu_e = pnx_alloc_dt(E * ff * W);     // up-projections, one [ff, width] matrix per expert
+          l.w_d_e = pnx_alloc_dt(E * W * ff);
+          pnx_expected_tensors += 2 + 2 * E;       // router, correction, e<j>.{up, down}
+          m_E = std::max(m_E, n_out); m_top = std::max<size_t>(m_top, s.top); m_ff = std::max(m_ff, ff);
+        }
+        const int H = s.heads, G = s.kv_heads;
+        const bool par = s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
+        if ((s.flags & TGIS_LAYER_SINK) != 0) {
+          l.sink = pnx_alloc<float>(H);
+          pnx_expected_tensors += 1;
+        }
+        l.pa = PoolAttnGeom{H, G, s.dim, s.vdim, s.window, s.window > 0 ? s.pool : 0, s.rot_dims, s.scale,
+                            (s.flags & TGIS_LAYER_UNIT_QK) != 0 ? 1 : 0, s.window > 0 ? s.keep_first : 0, s.chunk,
+                            (s.flags & TGIS_LAYER_ROT_INTERLEAVED) != 0 ? 1 : 0, l.sink};
+        int col = 0;
+        auto cols = [&](int n) { const int r = col; col += n; return r; };
+        l.c_q = cols(H * s.dim); l.c_k = cols(G * s.dim); l.c_v = cols(G * s.vdim);
+        if (par) {
+          l.c_mq = cols(s.mm_heads * s.mm_dim); l.c_mk = cols(s.mm_heads * s.mm_dim);
+          l.c_mv = cols(s.mm_heads * s.mm_vdim); l.c_mg = cols(s.mm_heads * s.mm_vdim);
+        }
+        l.in_cols = (col + 7) / 8 * 8;
+        l.w_in = pnx_alloc_dt((size_t)l.in_cols * W, true);
+        l.w_o = pnx_alloc_dt(W * H * s.vdim);
+        pnx_expected_tensors += 4;  // q, k, v, o
+        if ((s.flags & TGIS_LAYER_QKV_BIAS) != 0) {
+          l.in_bias = pnx_alloc<float>(l.in_cols, true);
+          pnx_expected_tensors += 3;  // q.b, k.b, v.b
+        }
+        if ((s.flags & TGIS_LAYER_OUT_BIAS) != 0) {
+          l.o_bias = pnx_alloc<float>(W);
+          pnx_expected_tensors += 1;
+        }
+        l.cos_sin = s.rot_dims > 0 ? pnx_rope_table(s.rot_base, s.rot_dims) : nullptr;
+        if (par) {
+          const size_t mv = (size_t)s.mm_heads * s.mm_vdim;
+          l.w_o2 = pnx_alloc_dt(W * mv);
+          l.mm_norm = pnx_alloc<float>(mv);
+          l.out_l = pnx_alloc<float>(W);
+          l.out_r = pnx_alloc<float>(W);
+          l.decay = pnx_alloc<float>(s.mm_heads);
+          CK(cudaMemcpy(l.decay, pnx_decays[i].data(), sizeof(float) * s.mm_heads, cudaMemcpyHostToDevice));
+          pnx_expected_tensors += 8;  // right.{q, k, v, g, norm, o, out}, left.out
+          m_f1 = std::max(m_f1, mv);
+        }
+        m_q = std::max<size_t>(m_q, (size_t)H * s.dim);
+        m_ov = std::max<size_t>(m_ov, (size_t)H * s.vdim);
+        m_down = std::max<size_t>(m_down, l.in_cols);
         continue;
       }
       if (gated_style) {
@@ -1535,35 +1622,36 @@ struct tgis_engine {
       cache_row_bytes += row * dt_size(pnx_dt);
       pnx_tile_tokens = std::min(pnx_tile_tokens, latent_tile_tokens(s.heads));
     }
-    if (pair_style) {
+    if (pair_style || dyt_style) {
       // the layer runs: layers [loop_start, loop_stop) repeat loop_times passes in a row; every run owns cache rows and state
       const int L = (int)pnx_layers.size(), a = pnx_spec.loop_start, b = pnx_spec.loop_stop;
       const int passes = (pnx_spec.loop_times > 1 && b > a) ? pnx_spec.loop_times : 1;
       auto push = [&](int li, bool add) {
-        pair_runs.push_back(pnx_layers[li]);
-        pair_runs.back().add_x0 = add;
+        layer_runs.push_back(pnx_layers[li]);
+        layer_runs.back().add_x0 = add;
       };
       for (int li = 0; li < (passes > 1 ? a : L); ++li) push(li, false);
       if (passes > 1) {
         for (int p = 0; p < passes; ++p)
-          for (int li = a; li < b; ++li) push(li, p > 0 && li == a);
+          for (int li = a; li < b; ++li) push(li, pnx_spec.loop_add_embed != 0 && p > 0 && li == a);
         for (int li = b; li < L; ++li) push(li, false);
-        pnx_x0 = pnx_alloc<float>(T * W);
+        if (pnx_spec.loop_add_embed != 0) pnx_x0 = pnx_alloc<float>(T * W);
       }
-      for (PnxLayer& r : pair_runs) {
+      for (PnxLayer& r : layer_runs) {
         const tgis_layer_spec& s = r.sp;
-        if (s.mixer == TGIS_MIXER_POOLED_ATTENTION)
+        if (run_has_kv(s))
           cache_row_bytes += (size_t)s.kv_heads * (s.dim + s.vdim) * dt_size(pnx_dt);   // (+ the pooled rows: counted per block below)
         else if (s.mixer == TGIS_MIXER_LATENT_ATTENTION)
           cache_row_bytes += (size_t)r.g.row() * dt_size(pnx_dt);
         else
           r.st_S = pnx_alloc<float>((size_t)S_max * s.heads * s.dim * s.vdim, true);
+        if (s.mixer == TGIS_MIXER_WINDOW_LIGHTNING) r.st_S = pnx_alloc<float>((size_t)S_max * s.mm_heads * s.mm_dim * s.mm_vdim, true);
       }
       if (pnx_spec.side_dim > 0) {
         pnx_side = pnx_alloc_dt(V * pnx_layers.size() * pnx_spec.side_dim);
         pnx_expected_tensors += 1;
       }
-      pnx_hB = pnx_alloc_dt(T * W, true);
+      if (pair_style) pnx_hB = pnx_alloc_dt(T * W, true);
       if (const char* e = getenv("TGIS_PAIR_OVERLAP")) pair_overlap = atoi(e) != 0;
       if (pair_overlap) {
         CK(cudaStreamCreateWithFlags(&stream2, cudaStreamNonBlocking));
@@ -1618,14 +1706,14 @@ struct tgis_engine {
       kv_bytes = (size_t)(free_b * (double)(c.gpu_mem_fraction > 0 ? c.gpu_mem_fraction : 0.85f));
     }
     size_t bytes_per_block = (size_t)KV_BLOCK * cache_row_bytes;
-    for (PnxLayer& r : pair_runs)   // pooled rows of the windowed attention runs
-      if (r.sp.mixer == TGIS_MIXER_POOLED_ATTENTION)
+    for (PnxLayer& r : layer_runs)   // pooled rows of the windowed attention runs
+      if (run_has_kv(r.sp))
         bytes_per_block += (size_t)r.pa.rows_per_page() * r.pa.kv_heads * (r.pa.dim + r.pa.vdim) * dt_size(pnx_dt);
     size_t nb = std::min(kv_bytes / std::max<size_t>(bytes_per_block, 1), (size_t)S_max * bt_stride + 1);
     if (nb < 1) throw CudaError("cache too small for one block");
     num_blocks = (int)nb;
     for (PnxLayer& l : pnx_layers) {  // finite everywhere
-      if (pair_style) break;   // (the layer runs own the caches)
+      if (pair_style || dyt_style) break;   // (the layer runs own the caches)
       if (l.sp.mixer == TGIS_MIXER_LATENT_ATTENTION) l.cache = pnx_alloc_dt(nb * KV_BLOCK * l.g.row(), true);
       if (l.sp.mixer == TGIS_MIXER_PARALLEL) {
         l.k_cache = pnx_alloc_dt(nb * KV_BLOCK * l.ca.kv_heads * l.ca.dim, true);
@@ -1641,9 +1729,9 @@ struct tgis_engine {
         }
       }
     }
-    for (PnxLayer& r : pair_runs) {
+    for (PnxLayer& r : layer_runs) {
       if (r.sp.mixer == TGIS_MIXER_LATENT_ATTENTION) r.cache = pnx_alloc_dt(nb * KV_BLOCK * r.g.row(), true);
-      if (r.sp.mixer == TGIS_MIXER_POOLED_ATTENTION) {
+      if (run_has_kv(r.sp)) {
         r.k_cache = pnx_alloc_dt(nb * KV_BLOCK * r.pa.kv_heads * r.pa.dim, true);
         r.v_cache = pnx_alloc_dt(nb * KV_BLOCK * r.pa.kv_heads * r.pa.vdim, true);
         if (r.pa.pool > 0) {
@@ -1714,6 +1802,12 @@ struct tgis_engine {
     };
     if (name == "embed") return mat(pnx_embed, V, W);
     if (name == "head" && !tied_head) return mat(pnx_head, V, W);
+    auto dyt = [&](const DytNorm& d, const std::string& part) -> int {   // part: "", ".b" or ".alpha"
+      if (part == "") return vec(const_cast<float*>(d.w), W);
+      if (part == ".b") return vec(const_cast<float*>(d.b), W);
+      return part == ".alpha" ? vec(const_cast<float*>(d.alpha), 1) : fail("unknown weight " + name);
+    };
+    if (dyt_style && name.rfind("final.norm", 0) == 0) return dyt(pnx_final_dyt, name.substr(10));
     if (name == "final.norm") return pair_style ? one(pnx_final_norm, W) : vec(pnx_final_norm, W);
     if (name == "side.embed" && pnx_side != nullptr) return mat(pnx_side, V, (int64_t)pnx_layers.size() * pnx_spec.side_dim);
     if (name.size() < 3 || name[0] != 'l') return fail("unknown weight " + name);
@@ -1772,6 +1866,56 @@ struct tgis_engine {
         if (sub == "mix.uv") return mat(l.w_uv, (int64_t)s.heads * s.vdim, s.kv_rank);
         if (sub == "mix.sink" && l.sink != nullptr) return vec(l.sink, s.heads);
         if (sub == "mix.o") return mat(l.w_o, W, (int64_t)s.heads * s.vdim);
+      }
+      return fail("unknown layer weight " + name);
+    }
+    if (dyt_style) {
+      auto in_rows = [&](int col, int64_t r) { return mat(at(l.w_in, (size_t)col * W), r, W); };
+      if (sub.rfind("norm1", 0) == 0) return dyt(l.dyt1, sub.substr(5));
+      if (sub.rfind("norm2", 0) == 0)   // (of a layer without a feed-forward: nothing reads it)
+        return s.mlp != TGIS_MLP_NONE ? dyt(l.dyt2, sub.substr(5)) : (n == W || n == 1) ? 0 : bad_shape();
+      if (s.mlp == TGIS_MLP_DENSE_GELU) {
+        // gate / up rows interleave (row 2j = gate_j, row 2j + 1 = up_j): one product, the gated activation in its epilogue
+        if (sub == "mlp.gate") return place(l.w_gu, pnx_dt, s.ff, W, 2 * W, 1);
+        if (sub == "mlp.up") return place(at(l.w_gu, (size_t)W), pnx_dt, s.ff, W, 2 * W, 1);
+        if (sub == "mlp.down") return mat(l.w_d, W, s.ff);
+      } else if (s.mlp == TGIS_MLP_MOE_GROUPED) {
+        const int64_t n_out = (int64_t)s.experts + s.identity, ff = s.expert_ff;
+        if (sub == "mlp.router") return mat(l.w_router, n_out, W);
+        if (sub == "mlp.correction") return vec(l.router_b, n_out);
+        if (sub.rfind("mlp.e", 0) == 0) {
+          const size_t d2 = sub.find('.', 5);
+          if (d2 == std::string::npos) return fail("unknown layer weight " + name);
+          const int ei = atoi(sub.substr(5, d2 - 5).c_str());
+          if (ei < 0 || ei >= s.experts) return fail("expert index out of range in " + name);
+          const std::string which = sub.substr(d2 + 1);
+          if (which == "up") return mat(at(l.w_gu_e, (size_t)ei * ff * W), ff, W);
+          if (which == "down") return mat(at(l.w_d_e, (size_t)ei * W * ff), W, ff);
+        }
+      }
+      const int64_t H = s.heads, G = s.kv_heads, mH = s.mm_heads;
+      const bool par = s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
+      const std::string left = par ? "mix.left." : "mix.", right = "mix.right.";
+      if (sub == left + "q") return in_rows(l.c_q, H * s.dim);
+      if (sub == left + "k") return in_rows(l.c_k, G * s.dim);
+      if (sub == left + "v") return in_rows(l.c_v, G * s.vdim);
+      if (sub == left + "o") return mat(l.w_o, W, H * s.vdim);
+      if (sub == left + "sink" && l.sink != nullptr) return vec(l.sink, H);
+      if (sub == left + "o.b" && l.o_bias != nullptr) return vec(l.o_bias, W);
+      if (l.in_bias != nullptr) {
+        if (sub == left + "q.b") return vec(l.in_bias + l.c_q, H * s.dim);
+        if (sub == left + "k.b") return vec(l.in_bias + l.c_k, G * s.dim);
+        if (sub == left + "v.b") return vec(l.in_bias + l.c_v, G * s.vdim);
+      }
+      if (par) {
+        if (sub == "mix.left.out") return vec(l.out_l, W);
+        if (sub == right + "out") return vec(l.out_r, W);
+        if (sub == right + "q") return in_rows(l.c_mq, mH * s.mm_dim);
+        if (sub == right + "k") return in_rows(l.c_mk, mH * s.mm_dim);
+        if (sub == right + "v") return in_rows(l.c_mv, mH * s.mm_vdim);
+        if (sub == right + "g") return in_rows(l.c_mg, mH * s.mm_vdim);
+        if (sub == right + "norm") return vec(l.mm_norm, mH * s.mm_vdim);
+        if (sub == right + "o") return mat(l.w_o2, W, mH * s.mm_vdim);
       }
       return fail("unknown layer weight " + name);
     }
@@ -2226,7 +2370,7 @@ struct tgis_engine {
   //   token's row of the side table);   x += x0 if the NEXT run opens a pass of a loop
   // and the tail leaves the next run's two normed inputs (after the last run: the final norm) behind.
   void pair_layer(int ri, int T, int S) {
-    PnxLayer& l = pair_runs[ri];
+    PnxLayer& l = layer_runs[ri];
     const tgis_layer_spec& s = l.sp;
     const int W = cfg.hidden, A = pnx_dt;
     const float eps = pnx_spec.norm_eps;
@@ -2236,8 +2380,8 @@ struct tgis_engine {
     const int32_t* d_tokslot = ds<int32_t>(off_tokslot);
     const AttnSeq* d_seqs = ds<AttnSeq>(off_seqs);
     const int32_t* d_bt = ds<int32_t>(off_bt);
-    const bool last = ri + 1 == (int)pair_runs.size();
-    const PnxLayer* nx = last ? nullptr : &pair_runs[ri + 1];
+    const bool last = ri + 1 == (int)layer_runs.size();
+    const PnxLayer* nx = last ? nullptr : &layer_runs[ri + 1];
     // ---- feed-forward on the second norm's rows -> pnx_yS, beside the mixer
     const bool has_ff = s.mlp == TGIS_MLP_DENSE_SILU;
     auto feed_forward = [&]() {
@@ -2343,6 +2487,107 @@ struct tgis_engine {
     pnx_dump_resid(T);
   }
 
+  // One layer run of the dyt style (TGIS_STYLE_PRE_DYT).  On entry pnx_hA holds dyt1(x) (operand type):
+  //   x += mixer(hA);   x += ff(dyt2(x))
+  // and every tail leaves the next sublayer's input (after the last run: the final norm times the logit scale) behind.
+  void dyt_layer(int ri, int T, int S) {
+    PnxLayer& l = layer_runs[ri];
+    const tgis_layer_spec& s = l.sp;
+    const int W = cfg.hidden, A = pnx_dt;
+    const float eps = pnx_spec.norm_eps;
+    const int32_t* d_pos = ds<int32_t>(off_pos);
+    const int32_t* d_slot = ds<int32_t>(off_slotmap);
+    const int32_t* d_tokslot = ds<int32_t>(off_tokslot);
+    const AttnSeq* d_seqs = ds<AttnSeq>(off_seqs);
+    const int32_t* d_bt = ds<int32_t>(off_bt);
+    const bool last = ri + 1 == (int)layer_runs.size(), has_ff = s.mlp != TGIS_MLP_NONE;
+    const bool par = s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
+    const DytNorm next = last ? pnx_final_dyt : layer_runs[ri + 1].dyt1;
+    const float next_scale = last && pnx_spec.logit_scale != 0.f ? pnx_spec.logit_scale : 1.f;
+    const int H = s.heads, ld = l.in_cols;
+    // ---- mixer: every projection that reads hA in one product [q | k | v (| q' | k' | v' | gate')]
+    pnx_gemm(pnx_hA, A, W, l.w_in, pnx_y1, DT_F32, ld, T, ld, W);
+    auto lightning = [&](cudaStream_t st) {   // -> pnx_yS
+      const int mH = s.mm_heads, mv = mH * s.mm_vdim;
+      OuterScan os{};
+      os.mode = OUTER_SCAN_LIGHTNING;
+      os.q = pnx_y1 + l.c_mq; os.k = pnx_y1 + l.c_mk; os.v = pnx_y1 + l.c_mv; os.ldq = os.ldk = os.ldv = ld;
+      os.q_scale = 1.f;
+      os.decay = l.decay;
+      os.S = l.st_S;
+      os.out = flx_f1; os.ldo = mv;
+      os.heads = mH; os.dim = s.mm_dim; os.vdim = s.mm_vdim;
+      CK(outer_scan_launch(os, d_seqs, S, d_tokslot, st));
+      CK(head_norm_gate_launch(flx_f1, mv, 1, mv, l.mm_norm, pnx_y1 + l.c_mg, ld, /*sigmoid*/ 0, eps, flx_op2, A, T, st));
+      n_launches += 2;
+      pnx_gemm(flx_op2, A, mv, l.w_o2, pnx_yS, DT_F32, W, T, W, mv);
+    };
+    const bool forked = par && stream2 != nullptr;   // the two mixers side by side
+    if (forked) {
+      CK(cudaEventRecord(ev_fork, stream));
+      CK(cudaStreamWaitEvent(stream2, ev_fork, 0));
+      on_side_stream = true;
+      lightning(stream2);
+      on_side_stream = false;
+      CK(cudaEventRecord(ev_join, stream2));
+    }
+    CK(poolattn_prep_launch(pnx_y1, ld, l.c_q, l.c_k, l.c_v, l.in_bias, l.pa, l.cos_sin, eps, d_pos, d_slot, pnx_q, l.k_cache, l.v_cache,
+                            A, T, stream));
+    CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, nullptr, nullptr, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16, d_bt,
+                       bt_stride, pnx_oA, A, l.pa, stream));
+    n_launches += 2;
+    pnx_gemm(pnx_oA, A, H * s.vdim, l.w_o, pnx_o, DT_F32, W, T, W, H * s.vdim);
+    if (forked) CK(cudaStreamWaitEvent(stream, ev_join, 0));
+    else if (par) lightning(stream);
+    DytTail dt{};
+    dt.y_main = pnx_o; dt.b_main = l.o_bias; dt.eps = eps;
+    if (par) { dt.y_pair = pnx_yS; dt.w_main = l.out_l; dt.w_pair = l.out_r; }
+    dt.resid = pnx_resid; dt.out = pnx_hA; dt.out_dtype = A;
+    dt.next = has_ff ? l.dyt2 : next;
+    dt.out_scale = has_ff ? 1.f : next_scale;
+    CK(dyt_tail_launch(dt, T, W, stream));
+    ++n_launches;
+    // ---- feed-forward
+    if (has_ff) {
+      DytTail ft{};
+      ft.resid = pnx_resid; ft.out = pnx_hA; ft.out_dtype = A; ft.next = next; ft.out_scale = next_scale;
+      if (s.mlp == TGIS_MLP_DENSE_GELU) {
+        pnx_gemm(pnx_hA, A, W, l.w_gu, pnx_actS, A, s.ff, T, 2 * s.ff, W, GEMM_ANY_GEGLU);
+        pnx_gemm(pnx_actS, A, s.ff, l.w_d, pnx_o, DT_F32, W, T, W, s.ff);
+        ft.y_main = pnx_o;
+      } else {  // TGIS_MLP_MOE_GROUPED
+        const int E = s.experts, n_out = E + s.identity, top = s.top, ff = s.expert_ff;
+        pnx_gemm(pnx_hA, A, W, l.w_router, pnx_rl, DT_F32, n_out, T, n_out, W);
+        CK(moe_route_launch(pnx_rl, n_out, l.router_b, n_out, top, pnx_ids, pnx_mixw, nullptr, T, stream, MOE_W_SHARE, s.expert_groups,
+                            s.expert_groups_keep));
+        // one row segment per output; those of the identity experts come last and enter no product
+        CK(moe_align_launch(pnx_ids, T, top, n_out, pnx_segoff, pnx_order, pnx_inv, stream));
+        n_launches += 2;
+        if (E > 0) {
+          GemmAny a{};
+          a.X = pnx_hA; a.W = l.w_gu_e; a.Y = pnx_actE;
+          a.x_dtype = A; a.w_dtype = A; a.y_dtype = A;
+          a.T = T * top; a.N = ff; a.K = W; a.ldx = W; a.ldw = W; a.ldy = ff;
+          a.batch = 1; a.seg_off = pnx_segoff; a.n_groups = E; a.w_gs = (long long)ff * W;
+          a.gather = pnx_order; a.gather_div = top; a.mode = GEMM_ANY_GELU;
+          CK(gemm_any_launch(a, stream));
+          GemmAny b{};
+          b.X = pnx_actE; b.W = l.w_d_e; b.Y = pnx_yE;
+          b.x_dtype = A; b.w_dtype = A; b.y_dtype = DT_F32;
+          b.T = T * top; b.N = W; b.K = ff; b.ldx = ff; b.ldw = ff; b.ldy = W;
+          b.batch = 1; b.seg_off = pnx_segoff; b.n_groups = E; b.w_gs = (long long)W * ff;
+          CK(gemm_any_launch(b, stream));
+          n_launches += 2;
+        }
+        ft.y_rows = pnx_yE; ft.inv = pnx_inv; ft.ids = pnx_ids; ft.mix_w = pnx_mixw; ft.top = top; ft.n_experts = E;
+        ft.in = l.dyt2;
+      }
+      CK(dyt_tail_launch(ft, T, W, stream));
+      ++n_launches;
+    }
+    pnx_dump_resid(T);
+  }
+
   // embeddings + layer stack + final norm -> pnx_hA [T, hidden] (operand type), fp32 residual stream in pnx_resid
   void pnx_forward(int T, int S) {
     const int W = cfg.hidden, A = pnx_dt;
@@ -2355,12 +2600,20 @@ struct tgis_engine {
     const LatentTile* d_tiles = ds<LatentTile>(off_ltiles);
     CK(embed_scale_f32_launch(d_tok, pnx_embed, A, pnx_spec.embed_scale, pnx_resid, T, W, cfg.vocab, stream));
     if (pair_style) {
-      const PnxLayer& f = pair_runs[0];
+      const PnxLayer& f = layer_runs[0];
       if (pnx_x0 != nullptr) CK(cudaMemcpyAsync(pnx_x0, pnx_resid, (size_t)T * W * sizeof(float), cudaMemcpyDeviceToDevice, stream));
       CK(rmsnorm_f32_launch(pnx_resid, W, f.norm1, 0.f, pnx_hA, A, W, T, W, eps, stream));
       if (f.sp.mlp == TGIS_MLP_DENSE_SILU) CK(rmsnorm_f32_launch(pnx_resid, W, f.norm2, 0.f, pnx_hB, A, W, T, W, eps, stream));
       n_launches += 3;
-      for (int ri = 0; ri < (int)pair_runs.size(); ++ri) pair_layer(ri, T, S);
+      for (int ri = 0; ri < (int)layer_runs.size(); ++ri) pair_layer(ri, T, S);
+      return;
+    }
+    if (dyt_style) {
+      DytTail dt{};   // nothing to add yet: the first mixer's input
+      dt.resid = pnx_resid; dt.out = pnx_hA; dt.out_dtype = A; dt.next = layer_runs[0].dyt1; dt.out_scale = 1.f;
+      CK(dyt_tail_launch(dt, T, W, stream));
+      n_launches += 2;
+      for (int ri = 0; ri < (int)layer_runs.size(); ++ri) dyt_layer(ri, T, S);
       return;
     }
     if (gated_style) {
@@ -2927,7 +3180,7 @@ struct tgis_engine {
         LatentTile* lt = hs<LatentTile>(off_ltiles);
         for (int q0 = 0; q0 < q_len; q0 += pnx_tile_tokens)
           lt[step_n_ltiles++] = LatentTile{s, q0, std::min(pnx_tile_tokens, q_len - q0), 0};
-        if (pair_style) {
+        if (pair_style || dyt_style) {
           LatentTile* lt16 = hs<LatentTile>(off_ltiles16);
           for (int q0 = 0; q0 < q_len; q0 += POOLATTN_TILE)
             lt16[step_n_ltiles16++] = LatentTile{s, q0, std::min(POOLATTN_TILE, q_len - q0), 0};
@@ -3481,7 +3734,8 @@ int tgis_abi_version(void) { return TGIS_ABI_VERSION; }
 int tgis_engine_create(const tgis_config* cfg, tgis_engine** out) {
   if (!cfg || !out) return fail("null argument");
   if (cfg->abi_version != TGIS_ABI_VERSION) return fail("ABI version mismatch");
-  if (cfg->arch == TGIS_ARCH_PONENEX || cfg->arch == TGIS_ARCH_FALERAX || cfg->arch == TGIS_ARCH_REVEPEL || cfg->arch == TGIS_ARCH_SIKAZEN)
+  if (cfg->arch == TGIS_ARCH_PONENEX || cfg->arch == TGIS_ARCH_FALERAX || cfg->arch == TGIS_ARCH_REVEPEL || cfg->arch == TGIS_ARCH_SIKAZEN ||
+      cfg->arch == TGIS_ARCH_BISUZEN)
     return fail("this architecture is described layer by layer: use tgis_engine_create_spec");
   if (cfg->arch != TGIS_ARCH_LLAMA && cfg->arch != TGIS_ARCH_OPT) return fail("unknown arch");
   if (cfg->arch == TGIS_ARCH_OPT) {
@@ -3528,7 +3782,8 @@ int tgis_engine_create(const tgis_config* cfg, tgis_engine** out) {
 int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec, tgis_engine** out) {
   if (!cfg || !spec || !out || !spec->layers) return fail("null argument");
   if (cfg->abi_version != TGIS_ABI_VERSION) return fail("ABI version mismatch");
-  if (cfg->arch != TGIS_ARCH_PONENEX && cfg->arch != TGIS_ARCH_FALERAX && cfg->arch != TGIS_ARCH_REVEPEL && cfg->arch != TGIS_ARCH_SIKAZEN)
+  if (cfg->arch != TGIS_ARCH_PONENEX && cfg->arch != TGIS_ARCH_FALERAX && cfg->arch != TGIS_ARCH_REVEPEL && cfg->arch != TGIS_ARCH_SIKAZEN &&
+      cfg->arch != TGIS_ARCH_BISUZEN)
     return fail("tgis_engine_create_spec: arch must be a layer-list architecture");
   if (spec->n_layers < 1 || spec->n_layers > 4096) return fail("bad n_layers");
   if (spec->dtype != TGIS_DTYPE_BF16 && spec->dtype != TGIS_DTYPE_F32) return fail("dtype must be bf16 or fp32");
@@ -3564,6 +3819,34 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
       } else {
         return fail("unknown mixer type" + at);
       }
+      continue;
+    }
+    if ((spec->style & TGIS_STYLE_PRE_DYT) != 0) {
+      if (spec->style != TGIS_STYLE_PRE_DYT) return fail("the dyt style has its own norm placement and an untied head");
+      if (spec->loop_times > 1 && (spec->loop_start < 0 || spec->loop_stop > spec->n_layers || spec->loop_start >= spec->loop_stop))
+        return fail("the looped span must lie inside the layer list");
+      if (spec->loop_times > 64) return fail("more than 64 passes of a loop");
+      if (spec->loop_add_embed != 0) return fail("the dyt style adds nothing between the passes of a loop");
+      if (s.mlp == TGIS_MLP_MOE_GROUPED) {
+        const int n_out = s.experts + s.identity;
+        if (s.experts < 0 || s.identity < 0 || n_out < 1 || n_out > 2048 || s.top < 1 || s.top > 32 || (s.experts > 0 && s.expert_ff < 1))
+          return fail("bad mixture-of-experts sizes" + at);
+        if (s.expert_groups < 1 || n_out % s.expert_groups != 0 || s.expert_groups_keep < 1 || s.expert_groups_keep > s.expert_groups ||
+            s.top > n_out / s.expert_groups * s.expert_groups_keep)
+          return fail("bad expert groups" + at);
+      } else if (s.mlp == TGIS_MLP_DENSE_GELU ? s.ff < 1 : s.mlp != TGIS_MLP_NONE) {
+        return fail("bad feed-forward" + at);
+      }
+      if (s.mixer != TGIS_MIXER_POOLED_ATTENTION && s.mixer != TGIS_MIXER_WINDOW_LIGHTNING) return fail("unknown mixer type" + at);
+      if (s.heads < 1 || s.kv_heads < 1 || s.heads % s.kv_heads != 0 || s.dim < 1 || s.vdim < 1 || s.vdim > POOLATTN_MAX_VDIM || s.dim > 512)
+        return fail("bad attention sizes" + at);
+      if (s.rot_dims < 0 || s.rot_dims > s.dim || (s.rot_dims & 1) || (s.rot_dims > 0 && !(s.rot_base > 0.f)))
+        return fail("rot.dims must be even and <= dim, rot.base positive" + at);
+      if (s.pool > 0) return fail("pooled blocks do not run in the dyt style" + at);
+      if (s.keep_first < 0 || s.chunk < 0) return fail("bad mask" + at);
+      if (s.mixer == TGIS_MIXER_WINDOW_LIGHTNING &&
+          (s.mm_heads < 1 || s.mm_dim < 1 || s.mm_dim > OUTER_SCAN_MAX_DIM || s.mm_vdim < 1 || s.decay == nullptr))
+        return fail("bad lightning-attention sizes" + at);
       continue;
     }
     if ((spec->style & TGIS_STYLE_PARALLEL_GATED) != 0) {
@@ -3641,6 +3924,10 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
   e->pnx_spec = *spec;
   e->pnx_layer_specs.assign(spec->layers, spec->layers + spec->n_layers);
   e->pnx_spec.layers = nullptr;
+  for (tgis_layer_spec& s : e->pnx_layer_specs) {   // the caller's arrays are not kept
+    e->pnx_decays.emplace_back(s.decay, s.decay + (s.decay != nullptr ? s.mm_heads : 0));
+    s.decay = nullptr;
+  }
   try {
     e->init();
   } catch (const std::exception& ex) {

@@ -5,8 +5,8 @@
 //   batched  blockIdx.z walks equal problems whose operands lie a fixed stride apart (one problem per attention head),
 //   grouped  the rows are cut into segments (seg_off, on the device) and segment g multiplies with weight matrix g
 //            (one segment per expert of a mixture-of-experts layer); rows of X may be gathered through an index list,
-// and six epilogues (plain store, SwiGLU or GeGLU over interleaved gate/up rows, per-(row, batch) scale, tanh, squared ReLU of
-// the row-scaled sum).
+// and seven epilogues (plain store, SwiGLU or GeGLU over interleaved gate/up rows, per-(row, batch) scale, tanh, squared ReLU of
+// the row-scaled sum, exact gelu).
 //
 // Every output element is the sum over k = 0 .. K-1 in ascending order inside one thread, so a row's result depends
 // neither on the other rows of the launch nor on where in a segment it landed.
@@ -45,6 +45,7 @@ __device__ __forceinline__ float glu_pair(int mode, float g, float u) {
   return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
 }
 
+__device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
 // max(acc * s, 0)^2 with s the scale of the row's INPUT (GEMM_ANY_RELU2)
 __device__ __forceinline__ float relu2_scaled(float acc, float s) {
   const float z = fmaxf(acc * s, 0.f);
@@ -153,7 +154,7 @@ __global__ void __launch_bounds__(ANY_THREADS) gemm_any_kernel(GemmAny a) {
       const float s = a.mode == GEMM_ANY_ROWSCALE ? a.row_scale[(size_t)dst * a.scale_ld + z] : 1.f;
 #pragma unroll
       for (int j = 0; j < 4; ++j)
-        if (n + j < a.N) st_from_float(Y + (size_t)dst * a.ldy + n + j, a.mode == GEMM_ANY_TANH ? tanhf(acc[i][j]) : acc[i][j] * s);
+        if (n + j < a.N) st_from_float(Y + (size_t)dst * a.ldy + n + j, a.mode == GEMM_ANY_TANH ? tanhf(acc[i][j]) : a.mode == GEMM_ANY_GELU ? gelu_erf(acc[i][j]) : acc[i][j] * s);
     }
   }
 }
@@ -305,6 +306,9 @@ __global__ void __launch_bounds__(ANY_THREADS) gemm_any_mma_kernel(GemmAny a) {
         } else if (a.mode == GEMM_ANY_TANH) {
           if (n < a.N) st_from_float(Y + (size_t)dst * a.ldy + n, tanhf(v0));
           if (n + 1 < a.N) st_from_float(Y + (size_t)dst * a.ldy + n + 1, tanhf(v1));
+        } else if (a.mode == GEMM_ANY_GELU) {
+          if (n < a.N) st_from_float(Y + (size_t)dst * a.ldy + n, gelu_erf(v0));
+          if (n + 1 < a.N) st_from_float(Y + (size_t)dst * a.ldy + n + 1, gelu_erf(v1));
         } else if (a.mode == GEMM_ANY_RELU2) {
           if (n < a.N) st_from_float(Y + (size_t)dst * a.ldy + n, relu2_scaled(v0, s));
           if (n + 1 < a.N) st_from_float(Y + (size_t)dst * a.ldy + n + 1, relu2_scaled(v1, s));

@@ -243,6 +243,7 @@ constexpr int GEMM_ANY_GEGLU = 3;     // as SWIGLU with the tanh form of gelu on
 constexpr int GEMM_ANY_TANH = 4;      // Y[row, n] = tanh(acc)
 constexpr int GEMM_ANY_RELU2 = 5;     // Y[row, n] = max(acc * s, 0)^2, s = row_scale[gather ? gather[row] : row] (row_scale == nullptr: 1):
                                       // a squared-ReLU layer whose INPUT row was multiplied by s
+constexpr int GEMM_ANY_GELU = 6;      // Y[row, n] = gelu(acc), the exact (erf) form
 struct GemmAny {
   const void* X; const void* W; void* Y;
   int x_dtype, w_dtype, y_dtype;   // DT_*
@@ -308,6 +309,23 @@ struct GatedTail {
   const float* extra;                 // optional fp32 [T, hidden]: added to the stream together with the update
 };
 cudaError_t gated_tail_launch(const GatedTail& a, int T, int hidden, cudaStream_t stream);
+// A sublayer's tail on an fp32 residual stream whose norms are elementwise, dyt(v) = tanh(alpha v) * w + b, row per CTA:
+//   y[t]      = y_main[t] + b_main                                                      (y_main != nullptr; b_main optional), or
+//             = (rmsnorm(y_main[t] + b_main) * w_main + rmsnorm(y_pair[t]) * w_pair) / 2  (y_pair != nullptr), or the mixture
+//             = sum_k mix_w[t, k] * (ids[t, k] < n_experts ? y_rows[inv[t * top + k]] : h[t])   (y_rows != nullptr; fixed k order)
+//               h[t] = dyt_in(resid[t]): the sublayer's own input, recomputed from the stream it was made of
+//   resid[t] += y[t]                                              (no y at all: the stream stays, only its norm is taken)
+//   out[t]    = dyt(resid[t]) * out_scale                         the next sublayer's input in the operand type
+struct DytNorm { const float *w, *b, *alpha; };   // [hidden], [hidden], one number (device memory)
+struct DytTail {
+  const float *y_main, *b_main;
+  const float *y_pair, *w_main, *w_pair; float eps;
+  const float* y_rows; const int32_t *inv, *ids; const float* mix_w; int top, n_experts;
+  DytNorm in;
+  float* resid;
+  DytNorm next; float out_scale; void* out; int out_dtype;
+};
+cudaError_t dyt_tail_launch(const DytTail& a, int T, int hidden, cudaStream_t stream);
 // out[t, j] = gelu_tanh(z[t, j]) * table[tok[t], col0 + j]   j < n: a gate on per-token side rows (z fp32 [T, ldz], table DT_*
 // [vocab, ld_table], out DT_* [T, n])
 cudaError_t gelu_gate_rows_launch(const float* z, int ldz, const int32_t* token_ids, const void* table, int table_dtype,
@@ -405,18 +423,25 @@ cudaError_t sigattn_launch(const void* q, const void* k_cache, const void* v_cac
                            const LatentTile* tiles, int n_tiles, const int32_t* block_table, int bt_stride,
                            const float* head_bias, void* out, int out_dtype, const SigAttnGeom& g, cudaStream_t stream);
 
-// ---- attention_pooled.cu: grouped-query softmax attention over a sliding window plus pooled blocks of what left it -----
+// ---- attention_pooled.cu: grouped-query softmax attention over a sliding window plus pooled blocks of what left it, over a
+// window plus the first tokens of the sequence, or inside chunks ----------------------------------------------------------
 // Per head: rotary turn of the first rot_dims entries of every query and key ("rotate half": i pairs with i + rot_dims / 2),
 // then (unit_norm != 0) q and k divided by their root mean square over dim; score = scale * q . k.  Query i sees the tokens j
 // with 0 <= i - j < window one by one and, with pool > 0, every block b of `pool` consecutive positions that ends at or
 // before i - window (b * pool + pool - 1 <= i - window) through ONE key and ONE value: the means of the block's cached
 // keys and of its values.  Tokens behind the window whose block is not complete by then are not seen.  The softmax runs
 // over window tokens and visible blocks together.  window <= 0: every earlier position, no blocks.  Query head h reads key/value head h / (heads / kv_heads).
+// keep_first > 0 (pool == 0): query i also sees the tokens j <= i with j < keep_first, whatever their distance.  chunk > 0: of all
+// these only the tokens j with j / chunk == i / chunk (chunks are counted from position 0 of the sequence).  sink [heads]
+// (nullptr: none): the softmax denominator of head h also holds exp(sink[h]), a term of the normaliser alone.
 struct PoolAttnGeom {
   int heads, kv_heads, dim, vdim, window, pool;
   int rot_dims;
   float scale;
   int unit_norm;
+  int keep_first, chunk;
+  int rot_interleaved;   // != 0: rotary pairs are (2i, 2i + 1) instead of (i, i + rot_dims / 2)
+  const float* sink;     // fp32 [heads] or nullptr
   __host__ __device__ int rows_per_page() const { return pool > 0 ? (KV_BLOCK + pool - 1) / pool : 0; }   // pooled rows a cache page owns
 };
 constexpr int POOLATTN_TILE = 16;      // query tokens per CTA
@@ -479,7 +504,8 @@ cudaError_t selective_scan_launch(const SelScan& a, const AttnSeq* seqs, int n_s
 //   OUTER_SCAN_HGRN:   f = l + (1 - l) sigmoid(decay_raw + w0), l = u (a lower bound per head and key channel);
 //                      S <- diag(f) S + (1 - f) v^T;  o = S^T silu(q)   (no key: what the gate forgets is what it writes; the
 //                      query reads the state after the token's update)
-constexpr int OUTER_SCAN_DECAY = 0, OUTER_SCAN_GATED = 1, OUTER_SCAN_SSD = 2, OUTER_SCAN_HGRN = 3;
+//   OUTER_SCAN_LIGHTNING:  S <- decay_h S + silu(k) silu(v)^T;  o = S^T silu(q)   (one fixed decay per head)
+constexpr int OUTER_SCAN_DECAY = 0, OUTER_SCAN_GATED = 1, OUTER_SCAN_SSD = 2, OUTER_SCAN_HGRN = 3, OUTER_SCAN_LIGHTNING = 4;
 constexpr int OUTER_SCAN_MAX_DIM = 256;
 struct OuterScan {
   int mode;
@@ -493,6 +519,7 @@ struct OuterScan {
   const float* x; float* x_last; int width;   // optional: x_last[slot] = x[last row of the portion] (the token shift's state)
   int qk_heads;                                // q / k heads (head h reads h / (heads / qk_heads)); 0: one per head
   const float* step_raw; int lds; const float *step_b, *A_log, *D;   // SSD: [T, heads], [heads], [heads], [heads]
+  const float* decay;                          // LIGHTNING: [heads]
 };
 cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot,
                               cudaStream_t stream);
@@ -528,9 +555,14 @@ cudaError_t convert_f32_launch(const float* x, void* out, int out_dtype, size_t 
 // logits fp32 [T, ld] (columns [0, E): experts; column E, when side_gate != nullptr: the shared expert's gate logit):
 //   ids[t, k], w[t, k] = the `top` largest of logits + bias and the softmax over just those;  side_gate[t] = sigmoid(.)
 // weight_mode MOE_W_SIGMOID: w[t, k] = sigmoid(logit) of each chosen expert, used as it is
-constexpr int MOE_W_SOFTMAX = 0, MOE_W_SIGMOID = 1;
+// weight_mode MOE_W_SHARE: scores s = softmax(logits) over all E, choice scores s + bias, w[t, k] = s of each chosen expert over
+// the sum of the chosen ones' (+ 1e-20).
+// groups > 1: the E outputs form `groups` equal groups of neighbours; a group counts as the largest value a choice is made by,
+// and only members of the `keep` best groups can be chosen.  Ties go to the lower index.
+constexpr int MOE_W_SOFTMAX = 0, MOE_W_SIGMOID = 1, MOE_W_SHARE = 2;
 cudaError_t moe_route_launch(const float* logits, int ld, const float* bias, int E, int top, int32_t* ids, float* w,
-                             float* side_gate, int T, cudaStream_t stream, int weight_mode = MOE_W_SOFTMAX);
+                             float* side_gate, int T, cudaStream_t stream, int weight_mode = MOE_W_SOFTMAX, int groups = 1,
+                             int keep = 1);
 // seg_off[E + 1]: rows per expert, prefix-summed; order[p] = t * top + k of the p-th row; inv[t * top + k] = p
 cudaError_t moe_align_launch(const int32_t* ids, int T, int top, int E, int32_t* seg_off, int32_t* order, int32_t* inv,
                              cudaStream_t stream);

@@ -3,8 +3,9 @@
 // are matrix products (gemm_any.cu); the weighted sum of their outputs is part of the sublayer's tail (resid_tail_kernel).
 //
 // Router arithmetic is fp32 throughout: logits + bias, selection, and the weights of the selected experts: the softmax over
-// the selected logits only (MOE_W_SOFTMAX) or each one's own sigmoid (MOE_W_SIGMOID; the order of sigmoid scores is the order
-// of the logits).
+// the selected logits only (MOE_W_SOFTMAX), each one's own sigmoid (MOE_W_SIGMOID; the order of sigmoid scores is the order
+// of the logits), or the selected ones' shares of a softmax over all of them (MOE_W_SHARE; the bias then enters the choice, after
+// the softmax, and not the weights).
 #include <cfloat>
 
 #include "kernels.h"
@@ -16,22 +17,52 @@ namespace {
 
 constexpr int ROUTE_WARPS = 4;
 
-// one warp per token; dynamic shared memory: ROUTE_WARPS x E floats
+// one warp per token; dynamic shared memory: ROUTE_WARPS x (E + groups) floats
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int E, int top,
-                 int32_t* __restrict__ ids, float* __restrict__ w, float* __restrict__ side_gate, int T, int weight_mode) {
+                 int32_t* __restrict__ ids, float* __restrict__ w, float* __restrict__ side_gate, int T, int weight_mode, int groups, int keep) {
   extern __shared__ float sm[];
   griddep_launch();
   griddep_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * ROUTE_WARPS + warp;
   if (t >= T) return;
-  float* z = sm + (size_t)warp * E;
+  float* z = sm + (size_t)warp * (E + groups);
   const float* row = logits + (size_t)t * ld;
-  for (int e = lane; e < E; e += 32) z[e] = row[e] + (bias ? bias[e] : 0.f);
+  float z_max = 0.f, z_sum = 1.f;   // MOE_W_SHARE: the softmax over all logits
+  if (weight_mode == MOE_W_SHARE) {
+    z_max = -FLT_MAX;
+    for (int e = lane; e < E; e += 32) z_max = fmaxf(z_max, row[e]);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) z_max = fmaxf(z_max, __shfl_xor_sync(0xffffffffu, z_max, o));
+    z_sum = 0.f;
+    for (int e = lane; e < E; e += 32) z_sum += expf(row[e] - z_max);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) z_sum += __shfl_xor_sync(0xffffffffu, z_sum, o);
+  }
+  for (int e = lane; e < E; e += 32)
+    z[e] = (weight_mode == MOE_W_SHARE ? expf(row[e] - z_max) / z_sum : row[e]) + (bias ? bias[e] : 0.f);
   if (side_gate != nullptr && lane == 0) side_gate[t] = 1.f / (1.f + expf(-row[E]));
   __syncwarp();
+  if (groups > 1) {   // members of all but the `keep` best groups are out of the choice
+    const int per = E / groups;
+    float* gs = z + E;
+    for (int g = lane; g < groups; g += 32) {
+      float m = -FLT_MAX;
+      for (int e = g * per; e < (g + 1) * per; ++e) m = fmaxf(m, z[e]);
+      gs[g] = m;
+    }
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {
+      const int g = e / per;
+      int better = 0;   // groups that come before this one
+      for (int o = 0; o < groups; ++o) better += (gs[o] > gs[g] || (gs[o] == gs[g] && o < g)) ? 1 : 0;
+      if (better >= keep) z[e] = -FLT_MAX;
+    }
+    __syncwarp();
+  }
   float my_val = -FLT_MAX;  // lane k keeps the k-th selected logit
+  int my_id = 0;
   for (int k = 0; k < top; ++k) {
     float best = -FLT_MAX;
     int bi = 0x7fffffff;
@@ -45,7 +76,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restri
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
     }
-    if (lane == (k & 31)) my_val = best;
+    if (lane == (k & 31)) { my_val = best; my_id = bi; }
     if (lane == 0) {
       ids[(size_t)t * top + k] = bi;
       z[bi] = -FLT_MAX;
@@ -54,6 +85,14 @@ moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restri
   }
   if (weight_mode == MOE_W_SIGMOID) {   // every chosen expert weighs its own sigmoid score; nothing is renormalised
     if (lane < top) w[(size_t)t * top + lane] = 1.f / (1.f + expf(-my_val));
+    return;
+  }
+  if (weight_mode == MOE_W_SHARE) {   // the chosen scores (without the bias) over their sum
+    const float s = lane < top ? expf(row[my_id] - z_max) / z_sum : 0.f;
+    float tot = s;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) tot += __shfl_xor_sync(0xffffffffu, tot, o);
+    if (lane < top) w[(size_t)t * top + lane] = s / (tot + 1e-20f);
     return;
   }
   // softmax over the selected logits (the first selected one is the largest)
@@ -99,11 +138,13 @@ moe_align_kernel(const int32_t* __restrict__ ids, int n, int E, int32_t* __restr
 }  // namespace
 
 cudaError_t moe_route_launch(const float* logits, int ld, const float* bias, int E, int top, int32_t* ids, float* w,
-                             float* side_gate, int T, cudaStream_t stream, int weight_mode) {
+                             float* side_gate, int T, cudaStream_t stream, int weight_mode, int groups, int keep) {
   if (T <= 0) return cudaSuccess;
-  if (top < 1 || top > 32 || top > E || (size_t)ROUTE_WARPS * E * 4 > 48 * 1024) return cudaErrorInvalidValue;
+  if (groups < 1 || E % groups != 0 || keep < 1 || keep > groups) return cudaErrorInvalidValue;
+  if (top < 1 || top > 32 || top > E / groups * keep || (size_t)ROUTE_WARPS * (E + groups) * 4 > 48 * 1024) return cudaErrorInvalidValue;
   return launch_k(moe_route_kernel, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
-                  (size_t)ROUTE_WARPS * E * sizeof(float), stream, logits, ld, bias, E, top, ids, w, side_gate, T, weight_mode);
+                  (size_t)ROUTE_WARPS * (E + groups) * sizeof(float), stream, logits, ld, bias, E, top, ids, w, side_gate, T, weight_mode,
+                  groups, keep);
 }
 
 cudaError_t moe_align_launch(const int32_t* ids, int T, int top, int E, int32_t* seg_off, int32_t* order, int32_t* inv,

@@ -246,7 +246,8 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
   float u_r[RPT];   // DECAY: the bonus u of this thread's rows; GATED: the normaliser n of its rows (the same in every lane)
   float m_run = 0.f;
   const float ssd_rate = MODE == OUTER_SCAN_SSD ? -expf(a.A_log[h]) : 0.f, ssd_skip = MODE == OUTER_SCAN_SSD ? a.D[h] : 0.f;
-  if (MODE == OUTER_SCAN_SSD || MODE == OUTER_SCAN_HGRN) {
+  const float fixed_decay = MODE == OUTER_SCAN_LIGHTNING ? a.decay[h] : 0.f;
+  if (MODE == OUTER_SCAN_SSD || MODE == OUTER_SCAN_HGRN || MODE == OUTER_SCAN_LIGHTNING) {
 #pragma unroll
     for (int j = 0; j < RPT; ++j) u_r[j] = 0.f;
   } else if (MODE == OUTER_SCAN_DECAY) {
@@ -311,6 +312,9 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
             v3[i] = silu_f(pq[e]) * a.q_scale;
             v3[D + i] = (1.f - pk[e]) * sigmoid_f(-pd[e]);                 // 1 - f without the cancellation near f = 1
             v3[2 * D + i] = pk[e] + (1.f - pk[e]) * sigmoid_f(pd[e]);
+          } else if (MODE == OUTER_SCAN_LIGHTNING) {
+            v3[i] = silu_f(pq[e]) * a.q_scale;
+            v3[D + i] = silu_f(pk[e]);
           } else {
             v3[i] = pq[e] * a.q_scale;
             v3[D + i] = pk[e];
@@ -319,8 +323,8 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
         }
       }
     }
-    vcol[st_tt * OS_COLS + 2 * st_l] = pv[0];
-    vcol[st_tt * OS_COLS + 2 * st_l + 1] = pv[1];
+    vcol[st_tt * OS_COLS + 2 * st_l] = MODE == OUTER_SCAN_LIGHTNING ? silu_f(pv[0]) : pv[0];
+    vcol[st_tt * OS_COLS + 2 * st_l + 1] = MODE == OUTER_SCAN_LIGHTNING ? silu_f(pv[1]) : pv[1];
     if (MODE == OUTER_SCAN_GATED && tid < nt) {
       gates[tid][0] = a.gate_cap * tanhf((pg0 + a.ig_b[h]) / a.gate_cap);
       gates[tid][1] = logsigmoid_f(a.gate_cap * tanhf((pg1 + a.fg_b[h]) / a.gate_cap));
@@ -352,6 +356,15 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
           const int i = g + j * OS_GROUPS;
           if (i < D) {
             S[j] = fmaf(v3[2 * D + i], S[j], v3[D + i] * vc);
+            o = fmaf(v3[i], S[j], o);
+          }
+        }
+      } else if (MODE == OUTER_SCAN_LIGHTNING) {
+#pragma unroll
+        for (int j = 0; j < RPT; ++j) {
+          const int i = g + j * OS_GROUPS;
+          if (i < D) {
+            S[j] = fmaf(fixed_decay, S[j], v3[D + i] * vc);
             o = fmaf(v3[i], S[j], o);
           }
         }
@@ -736,6 +749,10 @@ cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seq
   if (a.mode == OUTER_SCAN_SSD) {
     if (a.step_raw == nullptr || a.step_b == nullptr || a.A_log == nullptr || a.D == nullptr) return cudaErrorInvalidValue;
     return outer_scan_mode<OUTER_SCAN_SSD>(a, seqs, n_seqs, tok_slot, stream);
+  }
+  if (a.mode == OUTER_SCAN_LIGHTNING) {
+    if (a.decay == nullptr) return cudaErrorInvalidValue;
+    return outer_scan_mode<OUTER_SCAN_LIGHTNING>(a, seqs, n_seqs, tok_slot, stream);
   }
   if (a.mode == OUTER_SCAN_HGRN) {
     if (a.decay_raw == nullptr || a.w0 == nullptr || a.u == nullptr) return cudaErrorInvalidValue;

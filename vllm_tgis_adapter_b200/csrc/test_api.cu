@@ -600,6 +600,27 @@ int tgis_k_moe_route(const float* logits, int32_t ld, const float* bias, int32_t
   return 0;
 }
 
+int tgis_k_moe_route_grouped(const float* logits, int32_t ld, const float* bias, int32_t E, int32_t top, int32_t groups, int32_t keep,
+                             int32_t* ids, float* w, int32_t T) {
+  KCK(moe_route_launch(logits, ld, bias, E, top, ids, w, nullptr, T, 0, MOE_W_SHARE, groups, keep));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
+
+int tgis_k_dyt_tail(const float* y_main, const float* b_main, const float* y_pair, const float* w_main, const float* w_pair, float eps,
+                    const float* y_rows, const int32_t* inv, const int32_t* ids, const float* mix_w, int32_t top, int32_t n_experts,
+                    const float* in_w, const float* in_b, const float* in_alpha, float* resid, const float* w, const float* b,
+                    const float* alpha, float out_scale, void* out, int32_t out_dt, int32_t T, int32_t hidden) {
+  DytTail a{};
+  a.y_main = y_main; a.b_main = b_main; a.y_pair = y_pair; a.w_main = w_main; a.w_pair = w_pair; a.eps = eps;
+  a.y_rows = y_rows; a.inv = inv; a.ids = ids; a.mix_w = mix_w; a.top = top; a.n_experts = n_experts;
+  a.in = DytNorm{in_w, in_b, in_alpha};
+  a.resid = resid; a.next = DytNorm{w, b, alpha}; a.out_scale = out_scale; a.out = out; a.out_dtype = out_dt;
+  KCK(dyt_tail_launch(a, T, hidden, 0));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
+
 int tgis_k_moe_align(const int32_t* ids, int32_t T, int32_t top, int32_t E, int32_t* seg_off, int32_t* order, int32_t* inv) {
   KCK(moe_align_launch(ids, T, top, E, seg_off, order, inv, 0));
   KCK(cudaDeviceSynchronize());
@@ -674,7 +695,8 @@ int tgis_k_sigattn(const void* q, const void* k_cache, const void* v_cache, int3
 }
 
 static PoolAttnGeom to_pool(const tgis_k_poolattn_geom* g) {
-  return PoolAttnGeom{g->heads, g->kv_heads, g->dim, g->vdim, g->window, g->window > 0 ? g->pool : 0, g->rot_dims, g->scale, g->unit_norm};
+  return PoolAttnGeom{g->heads, g->kv_heads, g->dim, g->vdim, g->window, g->window > 0 ? g->pool : 0, g->rot_dims, g->scale, g->unit_norm,
+                      g->keep_first, g->chunk, g->rot_interleaved, g->sink};
 }
 
 int tgis_k_poolattn_prep(const float* y, int32_t ldy, int32_t q_off, int32_t k_off, int32_t v_off, const float* bias,
@@ -792,6 +814,22 @@ int tgis_k_outer_scan(int32_t mode, const float* q, const float* k, const float*
   a.ig = ig; a.fg = fg; a.ldg = ldg; a.ig_b = ig_b; a.fg_b = fg_b; a.gate_cap = gate_cap;
   a.S = S; a.n = n; a.m = m; a.out = out; a.ldo = ldo; a.heads = heads; a.dim = dim; a.vdim = vdim;
   a.x = x; a.x_last = x_last; a.width = width;
+  KCK(outer_scan_launch(a, d_seqs.p, n_seqs, tok_slot, 0));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
+
+int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_t ldq, int32_t ldk, int32_t ldv, const float* decay,
+                          float* S, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const int32_t* seqs_host,
+                          int32_t n_seqs, const int32_t* tok_slot) {
+  std::vector<AttnSeq> seqs;
+  host_seqs(seqs_host, n_seqs, seqs);
+  Tmp<AttnSeq> d_seqs;
+  KCK(d_seqs.upload(seqs.data(), seqs.size()));
+  OuterScan a{};
+  a.mode = OUTER_SCAN_LIGHTNING;
+  a.q = q; a.k = k; a.v = v; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.q_scale = 1.f;
+  a.decay = decay; a.S = S; a.out = out; a.ldo = ldo; a.heads = heads; a.dim = dim; a.vdim = vdim;
   KCK(outer_scan_launch(a, d_seqs.p, n_seqs, tok_slot, 0));
   KCK(cudaDeviceSynchronize());
   return 0;

@@ -10,14 +10,14 @@ import ctypes as C
 import os
 from pathlib import Path
 
-ABI_VERSION = 11
-ARCH_LLAMA, ARCH_OPT, ARCH_PONENEX, ARCH_FALERAX, ARCH_REVEPEL, ARCH_SIKAZEN = 0, 1, 2, 3, 4, 5
+ABI_VERSION = 12
+ARCH_LLAMA, ARCH_OPT, ARCH_PONENEX, ARCH_FALERAX, ARCH_REVEPEL, ARCH_SIKAZEN, ARCH_BISUZEN = 0, 1, 2, 3, 4, 5, 6
 MIXER_LATENT_ATTENTION, MIXER_PARALLEL, MIXER_SELECTIVE_SCAN, MIXER_WKV = 1, 2, 3, 4
 MIXER_SIGMOID_ATTENTION, MIXER_SSD, MIXER_CHANNEL_DELTA = 5, 6, 7
-MIXER_POOLED_ATTENTION, MIXER_HGRN = 8, 9
-MLP_NONE, MLP_MOE, MLP_DENSE_GELU, MLP_MOE_SIGMOID, MLP_DENSE_SILU = 0, 1, 2, 3, 4
-LAYER_ROT_INTERLEAVED, LAYER_SINK, LAYER_NO_OUT_GATE, LAYER_QKV_BIAS, LAYER_UNIT_QK = 1, 2, 4, 8, 16
-STYLE_POST_NORM, STYLE_TIED_HEAD, STYLE_PARALLEL_GATED, STYLE_PARALLEL_PAIR = 1, 2, 4, 8
+MIXER_POOLED_ATTENTION, MIXER_HGRN, MIXER_WINDOW_LIGHTNING = 8, 9, 10
+MLP_NONE, MLP_MOE, MLP_DENSE_GELU, MLP_MOE_SIGMOID, MLP_DENSE_SILU, MLP_MOE_GROUPED = 0, 1, 2, 3, 4, 5
+LAYER_ROT_INTERLEAVED, LAYER_SINK, LAYER_NO_OUT_GATE, LAYER_QKV_BIAS, LAYER_UNIT_QK, LAYER_OUT_BIAS = 1, 2, 4, 8, 16, 32
+STYLE_POST_NORM, STYLE_TIED_HEAD, STYLE_PARALLEL_GATED, STYLE_PARALLEL_PAIR, STYLE_PRE_DYT = 1, 2, 4, 8, 16
 DTYPE_BF16, DTYPE_F32 = 0, 1
 MAX_REQUEST_ID = 96
 MAX_TOPN = 12
@@ -51,7 +51,9 @@ class TgisLayerSpec(C.Structure):
         ("decay_rank", C.c_int32), ("reserved", C.c_int32),
         ("kv_from", C.c_int32), ("yarn_factor", C.c_float), ("yarn_original", C.c_float), ("yarn_fast", C.c_float),
         ("yarn_slow", C.c_float), ("groups", C.c_int32), ("norm_groups", C.c_int32), ("gate_rank", C.c_int32),
-        ("pool", C.c_int32), ("rot_linear", C.c_float), ("flags", C.c_int32), ("reserved2", C.c_int32),
+        ("pool", C.c_int32), ("rot_linear", C.c_float), ("flags", C.c_int32), ("keep_first", C.c_int32),
+        ("chunk", C.c_int32), ("identity", C.c_int32), ("expert_groups", C.c_int32), ("expert_groups_keep", C.c_int32),
+        ("reserved2", C.c_int32), ("decay", C.POINTER(C.c_float)),
     ]
 
 
@@ -80,6 +82,7 @@ class TgisKPoolAttnGeom(C.Structure):
     _fields_ = [
         ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32),
         ("pool", C.c_int32), ("rot_dims", C.c_int32), ("scale", C.c_float), ("unit_norm", C.c_int32),
+        ("keep_first", C.c_int32), ("chunk", C.c_int32), ("rot_interleaved", C.c_int32), ("sink", C.c_void_p),
     ]
 
 
@@ -88,7 +91,7 @@ class TgisModelSpec(C.Structure):
         ("n_layers", C.c_int32), ("dtype", C.c_int32), ("embed_scale", C.c_float), ("residual_mult", C.c_float),
         ("norm_eps", C.c_float), ("style", C.c_int32), ("layers", C.POINTER(TgisLayerSpec)),
         ("logit_scale", C.c_float), ("side_dim", C.c_int32),
-        ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("reserved", C.c_int32),
+        ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("loop_add_embed", C.c_int32),
     ]
 
 
@@ -143,7 +146,7 @@ ENGINE_SYMBOLS = [
 KERNEL_SYMBOLS = [
     "tgis_k_last_error", "tgis_k_gemm_timeline", "tgis_k_step_timeline_enable", "tgis_k_step_timeline_read", "tgis_k_gemm", "tgis_k_rmsnorm", "tgis_k_opt_layernorm", "tgis_k_opt_bias_act", "tgis_k_opt_embed", "tgis_k_silu_mul", "tgis_k_rope_kv", "tgis_k_gemm_rope", "tgis_k_gemm_norm_chain", "tgis_k_attention",
     "tgis_k_attention_bench", "tgis_k_decode_items", "tgis_k_gemm_plan", "tgis_k_gemm_unit_rows",
-    "tgis_k_sampler", "tgis_k_sampler_ex", "tgis_k_sampler_masked", "tgis_k_lora", "tgis_k_lora_bench", "tgis_k_silu_mul_interleaved", "tgis_k_gemm_any", "tgis_k_rmsnorm_f32", "tgis_k_resid_tail", "tgis_k_latent_prep", "tgis_k_latent_q_rope", "tgis_k_latent_attn", "tgis_k_moe_route", "tgis_k_moe_align", "tgis_k_capattn_prep", "tgis_k_capattn", "tgis_k_sigattn_prep", "tgis_k_sigattn", "tgis_k_poolattn_prep", "tgis_k_poolattn", "tgis_k_delta_scan", "tgis_k_ssd_scan", "tgis_k_token_shift", "tgis_k_short_conv", "tgis_k_selective_scan", "tgis_k_outer_scan", "tgis_k_head_norm_gate", "tgis_k_resid_tail_pair", "tgis_k_sizeof_sample_row", "tgis_k_sizeof_sample_out", "tgis_k_kv_block",
+    "tgis_k_sampler", "tgis_k_sampler_ex", "tgis_k_sampler_masked", "tgis_k_lora", "tgis_k_lora_bench", "tgis_k_silu_mul_interleaved", "tgis_k_gemm_any", "tgis_k_rmsnorm_f32", "tgis_k_resid_tail", "tgis_k_latent_prep", "tgis_k_latent_q_rope", "tgis_k_latent_attn", "tgis_k_moe_route", "tgis_k_moe_align", "tgis_k_moe_route_grouped", "tgis_k_dyt_tail", "tgis_k_lightning_scan", "tgis_k_capattn_prep", "tgis_k_capattn", "tgis_k_sigattn_prep", "tgis_k_sigattn", "tgis_k_poolattn_prep", "tgis_k_poolattn", "tgis_k_delta_scan", "tgis_k_ssd_scan", "tgis_k_token_shift", "tgis_k_short_conv", "tgis_k_selective_scan", "tgis_k_outer_scan", "tgis_k_head_norm_gate", "tgis_k_resid_tail_pair", "tgis_k_sizeof_sample_row", "tgis_k_sizeof_sample_out", "tgis_k_kv_block",
 ]
 
 _LIB: C.CDLL | None = None
@@ -221,6 +224,8 @@ def load_library() -> C.CDLL:
     lib.tgis_k_latent_attn.argtypes = [vp, vp, i32, C.POINTER(i32), i32, C.POINTER(i32), i32, i32, vp, i32, gp]
     lib.tgis_k_moe_route.argtypes = [vp, i32, vp, i32, i32, vp, vp, vp, i32]
     lib.tgis_k_moe_align.argtypes = [vp, i32, i32, i32, vp, vp, vp]
+    lib.tgis_k_moe_route_grouped.argtypes = [vp, i32, vp, i32, i32, i32, i32, vp, vp, i32]
+    lib.tgis_k_dyt_tail.argtypes = [vp, vp, vp, vp, vp, f32, vp, vp, vp, vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, f32, vp, i32, i32, i32]
     cg, ip = C.POINTER(TgisKCapAttnGeom), C.POINTER(i32)
     lib.tgis_k_capattn_prep.argtypes = [vp, i32, i32, i32, i32, cg, vp, vp, f32, vp, vp, vp, vp, vp, i32, i32]
     lib.tgis_k_capattn.argtypes = [vp, vp, vp, i32, ip, i32, ip, i32, i32, vp, i32, vp, cg]
@@ -237,6 +242,7 @@ def load_library() -> C.CDLL:
     lib.tgis_k_selective_scan.argtypes = [vp, vp, i32, vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp]
     lib.tgis_k_outer_scan.argtypes = [i32, vp, vp, vp, i32, i32, i32, f32, vp, i32, vp, vp, vp, vp, i32, vp, vp, f32, vp, vp, vp,
                                       vp, i32, i32, i32, i32, vp, vp, i32, ip, i32, vp]
+    lib.tgis_k_lightning_scan.argtypes = [vp, vp, vp, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp]
     lib.tgis_k_head_norm_gate.argtypes = [vp, i32, i32, i32, vp, vp, i32, i32, f32, vp, i32, i32]
     lib.tgis_k_resid_tail_pair.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, f32, i32, i32]
     _LIB = lib

@@ -3,6 +3,7 @@ from __future__ import annotations
 
 import ctypes as C
 import dataclasses
+import importlib
 from typing import Iterable
 
 from . import _lib
@@ -30,18 +31,19 @@ class ModelConfig:
     rms_eps: float = 1e-5
     max_model_len: int = 2048
     arch: str = "llama"
-    # arch "ponenex" (engine/ponenex.py), "falerax" (engine/falerax.py), "revepel" (engine/revepel.py) and "sikazen" (engine/sikazen.py): the layers are described one by one;
+    # arch "ponenex" (engine/ponenex.py), "falerax" (engine/falerax.py), "revepel" (engine/revepel.py), "sikazen" (engine/sikazen.py) and
+    # "bisuzen" (engine/bisuzen.py): the layers are described one by one;
     # n_q_heads / n_kv_heads / ffn are unused
-    layers: list | None = None          # list[ponenex.LayerSpec] / list[falerax.LayerSpec] / list[revepel.LayerSpec] / list[sikazen.LayerSpec]
+    layers: list | None = None          # list of the family module's LayerSpec
     embed_scale: float = 1.0
     logit_scale: float = 1.0            # logits = head x * logit_scale
     residual_mult: float = 1.0
     dtype: str = "bfloat16"             # "bfloat16" | "float32" (layer-list architectures only)
     side_dim: int = 0                   # arch "sikazen": columns of the side table one layer reads (0: no per-layer token input)
-    loop: tuple = (0, 0, 1)             # arch "sikazen": layers [start, stop) run `times` passes in a row
+    loop: tuple = (0, 0, 1)             # arch "sikazen" / "bisuzen": layers [start, stop) run `times` passes in a row
 
 
-LAYER_LIST_ARCHS = ("ponenex", "falerax", "revepel", "sikazen")   # created with tgis_engine_create_spec; bfloat16 or float32
+LAYER_LIST_ARCHS = ("ponenex", "falerax", "revepel", "sikazen", "bisuzen")   # created with tgis_engine_create_spec; bfloat16 or float32
 
 
 # Named architectures (real dims; this offline build runs them on synthetic weights — SURVEY.md §0)
@@ -77,9 +79,11 @@ def cache_block_bytes(mc: ModelConfig) -> int:
         from .sikazen import cache_block_elems
 
         return max((4 if mc.dtype == "float32" else 2) * cache_block_elems(mc, KV_BLOCK_TOKENS), 1)
-    if mc.arch in ("falerax", "revepel"):
+    if mc.arch in ("falerax", "revepel", "bisuzen"):
         if mc.arch == "falerax":
             from .falerax import cache_row_elems
+        elif mc.arch == "bisuzen":
+            from .bisuzen import cache_row_elems
         else:
             from .revepel import cache_row_elems
 
@@ -170,23 +174,15 @@ class NativeEngine:
         cfg.use_cuda_graphs, cfg.debug_gemm_ref, cfg.seed = int(use_cuda_graphs), 1 if debug_gemm_ref else 0, seed
         cfg.max_loras, cfg.max_lora_rank = int(max_loras), int(max_lora_rank) if max_loras else 0
         archs = {"llama": _lib.ARCH_LLAMA, "opt": _lib.ARCH_OPT, "ponenex": _lib.ARCH_PONENEX, "falerax": _lib.ARCH_FALERAX,
-                 "revepel": _lib.ARCH_REVEPEL, "sikazen": _lib.ARCH_SIKAZEN}
+                 "revepel": _lib.ARCH_REVEPEL, "sikazen": _lib.ARCH_SIKAZEN, "bisuzen": _lib.ARCH_BISUZEN}
         if model.arch not in archs:
             raise EngineError(f"unknown architecture {model.arch!r}")
         cfg.arch = archs[model.arch]
         self.max_loras, self.max_lora_rank = int(max_loras), int(max_lora_rank)
         self._h = C.c_void_p()
         if model.arch in LAYER_LIST_ARCHS:
-            if model.arch == "ponenex":
-                from .ponenex import model_spec
-            elif model.arch == "falerax":
-                from .falerax import model_spec
-            elif model.arch == "sikazen":
-                from .sikazen import model_spec
-            else:
-                from .revepel import model_spec
-
-            spec, _keep = model_spec(model)   # _keep: the ctypes layer array the spec points into
+            family = importlib.import_module("." + model.arch, __package__)   # one module per layer-list family
+            spec, _keep = family.model_spec(model)   # _keep: the ctypes arrays the spec points into
             if self.lib.tgis_engine_create_spec(C.byref(cfg), C.byref(spec), C.byref(self._h)) != 0:
                 raise EngineError(f"tgis_engine_create_spec failed: {_lib.last_error(self.lib)}")
         elif self.lib.tgis_engine_create(C.byref(cfg), C.byref(self._h)) != 0:

@@ -7,6 +7,7 @@ weights of the named architecture on the device instead."""
 from __future__ import annotations
 
 import dataclasses
+import importlib
 import json
 import logging
 from pathlib import Path
@@ -34,6 +35,10 @@ def model_config_from_hf(path: Path, max_model_len: int | None, dtype: str = "bf
         return model_config_from_json(cfg, max_model_len, dtype, checkpoint_shapes(path))
     if cfg.get("architecture") == "Sikazen":
         from .sikazen import model_config_from_json
+
+        return model_config_from_json(cfg, max_model_len, dtype)
+    if cfg.get("architecture") == "Bisuzen":
+        from .bisuzen import model_config_from_json
 
         return model_config_from_json(cfg, max_model_len, dtype)
     archs = cfg.get("architectures") or []
@@ -104,16 +109,8 @@ def load_synthetic_weights(eng: NativeEngine, mc: ModelConfig, seed: int, device
         return (torch.randn(r, c, generator=gen, device=f"cuda:{device}", dtype=torch.float32) * 0.02).to(torch.bfloat16)
 
     if mc.arch in LAYER_LIST_ARCHS:
-        if mc.arch == "ponenex":
-            from .ponenex import iter_synthetic_weights
-        elif mc.arch == "falerax":
-            from .falerax import iter_synthetic_weights
-        elif mc.arch == "sikazen":
-            from .sikazen import iter_synthetic_weights
-        else:
-            from .revepel import iter_synthetic_weights
-
-        for name, t in iter_synthetic_weights(mc, seed, f"cuda:{device}"):
+        family = importlib.import_module("." + mc.arch, __package__)
+        for name, t in family.iter_synthetic_weights(mc, seed, f"cuda:{device}"):
             eng.load_weight(name, t)
         return
 
@@ -194,12 +191,14 @@ def _resolve_model(args):
         if dtype == "float32" and mc.arch not in LAYER_LIST_ARCHS:
             raise ValueError(f"--dtype float32 is not available for the {mc.arch} architecture (bfloat16 only)")
         return mc, path
+    from .bisuzen import PRESETS as BISUZEN_PRESETS
     from .falerax import PRESETS as FALERAX_PRESETS
     from .ponenex import PRESETS as PONENEX_PRESETS
     from .revepel import PRESETS as REVEPEL_PRESETS
     from .sikazen import PRESETS as SIKAZEN_PRESETS
 
-    PONENEX_PRESETS = {**PONENEX_PRESETS, **FALERAX_PRESETS, **REVEPEL_PRESETS, **SIKAZEN_PRESETS}   # the presets of the layer-list architectures
+    PONENEX_PRESETS = {**PONENEX_PRESETS, **FALERAX_PRESETS, **REVEPEL_PRESETS, **SIKAZEN_PRESETS,
+                       **BISUZEN_PRESETS}   # the presets of the layer-list architectures
     if args.model in PRESETS or args.model in PONENEX_PRESETS:
         if not args.synthetic_weights:
             raise ValueError(f"--model {args.model} is a preset name: pass --synthetic-weights or a model directory")

@@ -148,6 +148,7 @@ def model_spec(mc: ModelConfig):
     spec.style = _lib.STYLE_PARALLEL_PAIR
     spec.side_dim = mc.side_dim
     spec.loop_start, spec.loop_stop, spec.loop_times = mc.loop
+    spec.loop_add_embed = 1
     spec.layers = C.cast(arr, C.POINTER(_lib.TgisLayerSpec))
     return spec, arr
 
