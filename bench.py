@@ -770,12 +770,13 @@ def run_ours(args) -> dict | None:
 
 
 # ------------------------------------------------------------------------------------------------ --arch-compare
-# Prefill and decode throughput of the layer-list families (Ponenex, Falerax, Revepel, Sikazen) beside the closest existing family (Llama) at equal hidden size, layer
+# Prefill and decode throughput of the layer-list families (Ponenex, Falerax, Revepel, Sikazen, Bisuzen) beside the closest existing family (Llama) at equal hidden size, layer
 # count and active feed-forward width, random weights, device-timed (the engine's CUDA events around every step).  Not the
 # default workload: `python bench.py --arch-compare` prints its own JSON line; the default JSON line is untouched.
 ARCH_COMPARE = [("ponenex-1k", "llama-cmp-1k"), ("ponenex-2k", "llama-cmp-2k"), ("falerax-1k", "llama-cmp-1k"),
                 ("falerax-2k", "llama-cmp-2k"), ("revepel-1k", "llama-cmp-1k"), ("revepel-2k", "llama-cmp-2k"),
-                ("sikazen-1k", "llama-cmp-1k"), ("sikazen-2k", "llama-cmp-2k")]
+                ("sikazen-1k", "llama-cmp-1k"), ("sikazen-2k", "llama-cmp-2k"),
+                ("bisuzen-1k", "llama-cmp-1k"), ("bisuzen-2k", "llama-cmp-2k")]
 
 
 def _arch_work(mc, B: int, ctx: float) -> tuple[float, float]:
@@ -863,6 +864,29 @@ def _arch_work(mc, B: int, ctx: float) -> tuple[float, float]:
             # behind it, latent rows), and reads + writes its fp32 state
             bytes_ += 2.0 * dense + B * (2.0 * cache + 8.0 * state)
         return flops + 2.0 * h * v, bytes_ + 2.0 * h * v
+    if mc.arch == "bisuzen":
+        from vllm_tgis_adapter_b200.engine.bisuzen import layer_runs
+
+        flops = bytes_ = 0.0
+        for i in layer_runs(mc):   # a looped layer runs (and streams its weights) once per pass
+            l = mc.layers[i]
+            keys = min(ctx, l.window + l.keep_first) if l.window else min(ctx, l.chunk or ctx)
+            dense = h * (l.heads * l.dim + l.kv_heads * (l.dim + l.vdim)) + l.heads * l.vdim * h
+            scan, state, cache = l.heads * keys * (l.dim + l.vdim), 0, keys * l.kv_heads * (l.dim + l.vdim)
+            if l.kind == "parallel":
+                dense += 2 * h * l.lin_heads * l.lin_dim + 3 * h * l.lin_heads * l.lin_vdim
+                state = l.lin_heads * l.lin_dim * l.lin_vdim
+                scan += 2 * state
+            ff = ff_step = 3 * h * l.ff
+            if l.moe:   # identity experts take their share of the choices and multiply nothing
+                n_out = l.experts + l.identity
+                ff = h * n_out + 2 * h * l.top * l.expert_ff * l.experts / n_out
+                ff_step = h * n_out + 2 * h * min(l.experts, B * l.top) * l.expert_ff
+            flops += 2.0 * (dense + ff + scan)
+            # a decode step streams the run's weights (every expert the batch touches), every sequence's visible cache rows,
+            # and reads + writes its fp32 state
+            bytes_ += 2.0 * (dense + ff_step) + B * (2.0 * cache + 8.0 * state)
+        return flops + 2.0 * h * v, bytes_ + 2.0 * h * v
     qd, kvd = mc.n_q_heads * 128, mc.n_kv_heads * 128
     per_layer = h * (qd + 2 * kvd) + qd * h + 3 * h * mc.ffn
     flops = mc.n_layers * 2.0 * (per_layer + mc.n_q_heads * ctx * 2 * 128) + 2.0 * h * v
@@ -884,7 +908,9 @@ def run_arch_compare(args) -> None:
 
     from vllm_tgis_adapter_b200.engine.sikazen import PRESETS as SKZ
 
-    PNX = {**PNX, **FLX, **RVP, **SKZ}   # the presets of the layer-list families
+    from vllm_tgis_adapter_b200.engine.bisuzen import PRESETS as BSZ
+
+    PNX = {**PNX, **FLX, **RVP, **SKZ, **BSZ}   # the presets of the layer-list families
 
     torch.cuda.set_device(0)
     hbm_gbs, _ = peaks()
