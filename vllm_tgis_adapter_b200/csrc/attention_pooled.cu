@@ -25,7 +25,9 @@
 // token, p = b * pool / KV_BLOCK, at index b - ceil(p * KV_BLOCK / pool); a page owns ceil(KV_BLOCK / pool) of them.
 #include <cmath>
 #include <cstdint>
+#include <algorithm>
 #include <cstdlib>
+#include <type_traits>
 
 #include "kernels.h"
 #include "launch.cuh"
@@ -326,22 +328,27 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
 }
 
 // ---------------------------------------------------------------------------------------------------------------- tensor cores
-// bf16 queries and cache rows, dim a multiple of 16 (<= 16 MMA_KS), vdim a multiple of 8 (<= 32 MMA_NT per warp).  Both products
-// on mma.sync m16n8k16 with fp32 accumulators: the tile's 16 queries are the M rows; for the scores each of the four warps owns
-// 8 of a chunk's 32 keys (the query's A fragments stay in registers for the whole walk, key rows are B fragments as they lie;
-// the chunk after the current one lands in a second buffer through cp.async meanwhile), for the weighted sum each warp owns
-// every fourth group of 8 value columns (value rows through ldmatrix.trans).  Scale, mask and the running softmax are fp32 on
-// the accumulator fragments; the weights are rounded to bf16 once and the SAME rounded numbers are summed for the normaliser.
-// Pooled chunks and token chunks differ only in where a row comes from and in which queries see it.
-constexpr int MMA_KS = 8, MMA_NT = 8, PA_NST = 4;
+// bf16 queries and cache rows, dim a multiple of 16 (<= 16 MMA_KS), vdim a multiple of 8 (<= 8 NT).  Both products on mma.sync
+// m16n8k16 with fp32 accumulators.  A warp owns 16 rows -- (token, query head) pairs of ONE key/value head -- from their scores to
+// their outputs: the query's A fragments stay in registers for the whole walk, a chunk's 32 scores per row, the running maximum and
+// sum and the accumulators never leave the warp, and the softmax weights become the A fragments of the second product as they lie.
+// Scale, mask and the running softmax are fp32 on the accumulator fragments; the weights are rounded to bf16 once and the SAME
+// rounded numbers are summed for the normaliser.  Pooled chunks and token chunks differ only in where a row comes from and in
+// which queries see it; a warp passes over a chunk that none of its rows sees.
+//
+// Two shapes of the same walk, four warps each; chunks arrive in a ring through 16-byte asynchronous copies:
+//   SPLIT = false  64 rows per CTA, 16 per warp: a chunk's rows are fetched once for all four warps (prompts and portions)
+//   SPLIT = true   16 rows per CTA, and every warp walks every fourth chunk on its own, without any CTA-wide barrier; the four
+//                  (maximum, sum, accumulator) states meet once at the end (decoded tokens: few rows, long walks)
+constexpr int MMA_KS = 8, MMA_MAX_NT = 32;
+template <bool SPLIT>
+struct PaShape {
+  static constexpr int ROWS = SPLIT ? 16 : 64, CPS = SPLIT ? 4 : 1, NST = SPLIT ? 2 : 4;   // rows per CTA, chunks per ring stage, stages
+};
 __device__ __forceinline__ void pa_ldsm_x4(uint32_t (&r)[4], const void* smem) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];\n"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(a));
-}
-__device__ __forceinline__ void pa_ldsm_x2(uint32_t (&r)[2], const void* smem) {
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];\n" : "=r"(r[0]), "=r"(r[1]) : "r"(a));
 }
 __device__ __forceinline__ void pa_ldsm_x4_trans(uint32_t (&r)[4], const void* smem) {
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(smem);
@@ -358,200 +365,261 @@ __device__ __forceinline__ void pa_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
+template <int NT, bool SPLIT>
 __global__ void __launch_bounds__(PA_THREADS)
 poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                     const __nv_bfloat16* __restrict__ v_cache, const __nv_bfloat16* __restrict__ pk,
                     const __nv_bfloat16* __restrict__ pv, const AttnSeq* __restrict__ seqs, const LatentTile* __restrict__ tiles,
                     const int32_t* __restrict__ block_table, int bt_stride, __nv_bfloat16* __restrict__ out, PoolAttnGeom g, int gs) {
-  // gs: query heads per tile.  1: the 16 rows are 16 tokens of head blockIdx.y; grid (tiles, heads).  heads / kv_heads (2, 4, 8 or
-  // 16): the rows are (token, head of key/value head blockIdx.y) pairs, 16 / gs tokens x gs heads, so a chunk's rows are fetched
-  // once for the whole group and a decoded token fills gs rows instead of one; grid (tiles, kv_heads, gs), CTA z takes the
-  // tile's tokens [z * 16 / gs, (z + 1) * 16 / gs) and leaves at once when the tile has none there.
+  // gs: query heads of a key/value head that share a CTA's rows (1, 2, 4, 8 or 16).  Row r: token r / gs of the CTA's ROWS / gs,
+  // head h_base + r % gs.  Grid (tiles, heads / gs, max(1, 16 gs / ROWS)): CTA z takes every ROWS / gs tokens of a 16-token tile; where
+  // a CTA takes more than a tile's 16 tokens, the tiles in between have nothing to do.
   using bf = __nv_bfloat16;
+  using SH = PaShape<SPLIT>;
   extern __shared__ __align__(16) uint8_t pam_smem[];
-  const int d = g.dim, dv = g.vdim, LDK = d + 8, LDV = dv + 8, LDP = KV_BLOCK + 8;
-  bf* Qs = reinterpret_cast<bf*>(pam_smem);            // [16][LDK]
-  bf* Ks2 = Qs + PA_QT * LDK;                          // [PA_NST][32][LDK]   a ring of chunks: one in use, the next ones landing
-  bf* Vs2 = Ks2 + PA_NST * KV_BLOCK * LDK;             // [PA_NST][32][LDV]
-  bf* Ps = Vs2 + PA_NST * KV_BLOCK * LDV;              // [16][LDP]
-  float* smax = reinterpret_cast<float*>(Ps + PA_QT * LDP);   // [4][16]; reused for the final row sums
+  const int d = g.dim, dv = g.vdim, LDK = d + 8, LDV = dv + 8;
+  bf* Ks2 = reinterpret_cast<bf*>(pam_smem);                     // [NST * CPS][32][LDK]   (first the queries: [ROWS][LDK])
+  bf* Vs2 = Ks2 + (size_t)SH::NST * SH::CPS * KV_BLOCK * LDK;    // [NST * CPS][32][LDV]
   griddep_launch();
   griddep_wait();
   const LatentTile tl = tiles[blockIdx.x];
   const AttnSeq sq = seqs[tl.seq];
-  const int kvh = gs > 1 ? blockIdx.y : blockIdx.y / (g.heads / g.kv_heads);
-  const int h_base = gs > 1 ? kvh * gs : blockIdx.y;     // head of row r: h_base + r % gs
-  const int tpt = PA_QT / gs;                             // tokens of this CTA's rows; token of row r: r / gs
-  const int tok0 = gs > 1 ? blockIdx.z * tpt : 0;
-  if (tok0 >= tl.nq) return;
+  const int tpt = SH::ROWS / gs;   // tokens per CTA
+  int tok0 = tl.q0, nq;
+  if (tpt > PA_QT) {
+    if (tl.q0 % tpt != 0) return;
+    nq = min(tpt, sq.q_len - tok0);
+  } else {
+    const int off = blockIdx.z * tpt;
+    if (off >= tl.nq) return;
+    tok0 += off;
+    nq = min(tpt, tl.nq - off);
+  }
+  const int h_base = blockIdx.y * gs, kvh = h_base / (g.heads / g.kv_heads);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t2 = (lane & 3) * 2;
-  const int row0 = sq.q_start + tl.q0 + tok0, pos0 = sq.kv_len - sq.q_len + tl.q0 + tok0, nq = min(tpt, tl.nq - tok0);
-  const int pos_last = pos0 + nq - 1;
-  const int dch = d / 8, vch = dv / 8;   // 16-byte chunks per row
-  for (int i = tid; i < PA_QT * dch; i += PA_THREADS) {
+  const int row0 = sq.q_start + tok0, pos0 = sq.kv_len - sq.q_len + tok0, pos_last = pos0 + nq - 1;
+  const int dch = d / 8, vch = dv / 8;   // 16-byte pieces per row
+  for (int i = tid; i < SH::ROWS * dch; i += PA_THREADS) {
     const int r = i / dch, ch = i % dch, tq = r / gs;
     uint4 v = make_uint4(0, 0, 0, 0);
     if (tq < nq) v = *reinterpret_cast<const uint4*>(q + ((size_t)(row0 + tq) * g.heads + h_base + r % gs) * d + ch * 8);
-    *reinterpret_cast<uint4*>(Qs + r * LDK + ch * 8) = v;
+    *reinterpret_cast<uint4*>(Ks2 + r * LDK + ch * 8) = v;
   }
   __syncthreads();
-  const int nks = d / 16;
+  const int nks = d / 16, wr0 = SPLIT ? 0 : warp * 16;   // the warp's first row
   uint32_t qa[MMA_KS][4];
 #pragma unroll
   for (int ks = 0; ks < MMA_KS; ++ks)
-    if (ks < nks) pa_ldsm_x4(qa[ks], Qs + (size_t)(lane & 15) * LDK + ks * 16 + (lane >> 4) * 8);
-  float acc[MMA_NT][4];
+    if (ks < nks) pa_ldsm_x4(qa[ks], Ks2 + (size_t)(wr0 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
+  __syncthreads();   // the ring may overwrite the queries
+  float acc[NT][4];
 #pragma unroll
-  for (int j = 0; j < MMA_NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_part[2] = {0.f, 0.f};   // rows gq and gq + 8
+  for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_part[2] = {0.f, 0.f};   // rows gq and gq + 8 of the warp
   if (g.sink != nullptr) {
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      m_run[r] = g.sink[h_base + (gq + r * 8) % gs];
-      l_part[r] = (warp == 0 && (lane & 3) == 0) ? 1.f : 0.f;   // (the row's sum adds up the parts of all its threads)
+      m_run[r] = g.sink[h_base + (wr0 + gq + r * 8) % gs];
+      l_part[r] = ((!SPLIT || warp == 0) && (lane & 3) == 0) ? 1.f : 0.f;   // (the row's sum adds up the parts of all its threads)
     }
   }
-  const int tqr[2] = {gq / gs, (gq + 8) / gs};   // tokens of this thread's two rows
+  const int tqr[2] = {(wr0 + gq) / gs, (wr0 + gq + 8) / gs};   // tokens of this thread's two rows
   const Visible vis[2] = {visible_tokens(pos0 + tqr[0], g), visible_tokens(pos0 + tqr[1], g)};
   const int n_vis[2] = {pooled_visible(pos0 + tqr[0], g.window, g.pool), pooled_visible(pos0 + tqr[1], g.window, g.pool)};
+  // the warp's first and last token: which chunks concern it at all
+  const int tq_lo = wr0 / gs, tq_hi = min((wr0 + 15) / gs, nq - 1);
+  const Visible w_first = visible_tokens(pos0 + tq_lo, g);
+  const int w_pooled = pooled_visible(pos0 + tq_hi, g.window, g.pool);
   const int n_pooled = pooled_visible(pos_last, g.window, g.pool);
   const Visible first = visible_tokens(pos0, g);
   const int blk0 = first.lo / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
   // chunks in front of the window's blocks: pooled rows, or the blocks of the kept first tokens
   const int n_pc = g.pool > 0 ? (n_pooled + KV_BLOCK - 1) / KV_BLOCK : min((first.keep + KV_BLOCK - 1) / KV_BLOCK, blk0);
-  const int n_chunks = n_pc + blk1 - blk0 + 1;
+  const int n_chunks = n_pc + blk1 - blk0 + 1, n_it = (n_chunks + SH::CPS - 1) / SH::CPS;
   const int rpp = g.rows_per_page();
   const int32_t* bt = block_table + (size_t)sq.block_row * bt_stride;
-  // chunk c's K and V rows -> stage c % PA_NST of the ring, as 16-byte asynchronous copies: four threads share a row, every
-  // call is one commit group (an empty one past the last chunk, so that the group count tells which chunk has landed); pooled
-  // rows that do not exist yet are zeros
-  const int fj = tid >> 2, fl = tid & 3;
-  auto fetch = [&](int c) {
-    if (c < n_chunks) {
-      const bool pooled = g.pool > 0 && c < n_pc;
-      const int blk = c < n_pc ? c : blk0 + c - n_pc;   // pooled chunk, or cache block of the sequence
-      long long r;
-      if (pooled) {
-        const int b = blk * KV_BLOCK + fj;
-        r = b < n_pooled ? (long long)pooled_row(b, g.pool, rpp, bt) : -1;
-      } else {
-        r = (long long)bt[blk] * KV_BLOCK + fj;
-      }
-      bf* Kd = Ks2 + ((size_t)(c % PA_NST) * KV_BLOCK + fj) * LDK;
-      bf* Vd = Vs2 + ((size_t)(c % PA_NST) * KV_BLOCK + fj) * LDV;
-      if (r < 0) {
-        for (int ch = fl; ch < dch; ch += 4) *reinterpret_cast<uint4*>(Kd + ch * 8) = make_uint4(0, 0, 0, 0);
-        for (int ch = fl; ch < vch; ch += 4) *reinterpret_cast<uint4*>(Vd + ch * 8) = make_uint4(0, 0, 0, 0);
-      } else {
-        const bf* ks = (pooled ? pk : k_cache) + ((size_t)r * g.kv_heads + kvh) * d;
-        const bf* vs = (pooled ? pv : v_cache) + ((size_t)r * g.kv_heads + kvh) * dv;
-        for (int ch = fl; ch < dch; ch += 4) pa_cp_async16(Kd + ch * 8, ks + ch * 8);
-        for (int ch = fl; ch < vch; ch += 4) pa_cp_async16(Vd + ch * 8, vs + ch * 8);
-      }
+  // one row of chunk c -> row fj of ring buffer `buf`, four threads per row; pooled rows that do not exist yet are zeros
+  auto fetch_row = [&](int c, int buf, int fj, int fl) {
+    const bool pooled = g.pool > 0 && c < n_pc;
+    const int blk = c < n_pc ? c : blk0 + c - n_pc;   // pooled chunk, or cache block of the sequence
+    long long r;
+    if (pooled) {
+      const int b = blk * KV_BLOCK + fj;
+      r = b < n_pooled ? (long long)pooled_row(b, g.pool, rpp, bt) : -1;
+    } else {
+      r = (long long)bt[blk] * KV_BLOCK + fj;
+    }
+    bf* Kd = Ks2 + ((size_t)buf * KV_BLOCK + fj) * LDK;
+    bf* Vd = Vs2 + ((size_t)buf * KV_BLOCK + fj) * LDV;
+    if (r < 0) {
+      for (int ch = fl; ch < dch; ch += 4) *reinterpret_cast<uint4*>(Kd + ch * 8) = make_uint4(0, 0, 0, 0);
+      for (int ch = fl; ch < vch; ch += 4) *reinterpret_cast<uint4*>(Vd + ch * 8) = make_uint4(0, 0, 0, 0);
+    } else {
+      const bf* ks = (pooled ? pk : k_cache) + ((size_t)r * g.kv_heads + kvh) * d;
+      const bf* vs = (pooled ? pv : v_cache) + ((size_t)r * g.kv_heads + kvh) * dv;
+      for (int ch = fl; ch < dch; ch += 4) pa_cp_async16(Kd + ch * 8, ks + ch * 8);
+      for (int ch = fl; ch < vch; ch += 4) pa_cp_async16(Vd + ch * 8, vs + ch * 8);
+    }
+  };
+  // every call is one commit group (an empty one past the last chunk), so that the group count tells which chunk has landed
+  auto fetch = [&](int it) {
+    if (SPLIT) {   // the warp's own chunk of the stage
+      const int c = it * SH::CPS + warp;
+      if (c < n_chunks)
+        for (int p = 0; p < 4; ++p) fetch_row(c, (it % SH::NST) * SH::CPS + warp, p * 8 + (lane >> 2), lane & 3);
+    } else if (it < n_chunks) {
+      fetch_row(it, it % SH::NST, tid >> 2, tid & 3);
     }
     asm volatile("cp.async.commit_group;\n" ::: "memory");
   };
 #pragma unroll
-  for (int c = 0; c < PA_NST - 1; ++c) fetch(c);
-  for (int c = 0; c < n_chunks; ++c) {
+  for (int it = 0; it < SH::NST - 1; ++it) fetch(it);
+  for (int it = 0; it < n_it; ++it) {
+    asm volatile("cp.async.wait_group %0;\n" ::"n"(SH::NST - 2) : "memory");
+    // this pass's chunk has landed for every thread that reads it, and the stage fetched into next is consumed
+    if (SPLIT) __syncwarp();
+    else __syncthreads();
+    fetch(it + SH::NST - 1);
+    const int c = SPLIT ? it * SH::CPS + warp : it, buf = SPLIT ? (it % SH::NST) * SH::CPS + warp : it % SH::NST;
     const bool pooled = g.pool > 0 && c < n_pc;
-    const int blk = c < n_pc ? c : blk0 + c - n_pc;
-    // the stage that chunk c + PA_NST - 1 goes to was last read in the previous pass, which ended with a barrier
-    fetch(c + PA_NST - 1);
-    asm volatile("cp.async.wait_group %0;\n" ::"n"(PA_NST - 1) : "memory");
-    __syncthreads();   // every thread's copies of chunk c have landed
-    const bf* Ks = Ks2 + (size_t)(c % PA_NST) * KV_BLOCK * LDK;
-    const bf* Vs = Vs2 + (size_t)(c % PA_NST) * KV_BLOCK * LDV;
-    // ---- scores of this warp's 8 keys
-    float sc[4] = {0.f, 0.f, 0.f, 0.f};
+    const int blk = c < n_pc ? c : blk0 + c - n_pc, key0 = blk * KV_BLOCK;   // first pooled block number, or token position
+    const bool idle = c >= n_chunks || tq_lo >= nq ||
+                      (pooled ? key0 >= w_pooled : key0 > pos0 + tq_hi || (key0 + KV_BLOCK <= w_first.lo && key0 >= w_first.keep));
+    if (!idle) {   // (the same for the whole warp)
+      const bf* Ks = Ks2 + (size_t)buf * KV_BLOCK * LDK;
+      const bf* Vs = Vs2 + (size_t)buf * KV_BLOCK * LDV;
+      float sc[4][4];   // keys 8 j + t2, 8 j + t2 + 1 of rows gq and gq + 8
 #pragma unroll
-    for (int ks = 0; ks < MMA_KS; ++ks)
-      if (ks < nks) {
-        uint32_t kb2[2];
-        pa_ldsm_x2(kb2, Ks + (size_t)(warp * 8 + (lane & 7)) * LDK + ks * 16 + ((lane >> 3) & 1) * 8);
-        pa_mma(sc, qa[ks], kb2[0], kb2[1]);
+      for (int j = 0; j < 4; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+#pragma unroll
+      for (int ks = 0; ks < MMA_KS; ++ks)
+        if (ks < nks) {
+#pragma unroll
+          for (int jj = 0; jj < 2; ++jj) {
+            uint32_t kb[4];
+            pa_ldsm_x4(kb, Ks + (size_t)(jj * 16 + (lane >> 4) * 8 + (lane & 7)) * LDK + ks * 16 + ((lane >> 3) & 1) * 8);
+            pa_mma(sc[2 * jj], qa[ks], kb[0], kb[1]);
+            pa_mma(sc[2 * jj + 1], qa[ks], kb[2], kb[3]);
+          }
+        }
+      float al[2];
+      uint32_t pa[2][4];   // the weights as A fragments of the two 16-key steps of the second product
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int pi = pos0 + tqr[r];
+        float mx = -INFINITY;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int kidx = key0 + j * 8 + t2 + e;
+            const bool ok = tqr[r] < nq && (pooled ? kidx < n_vis[r] : (kidx <= pi && (kidx >= vis[r].lo || kidx < vis[r].keep)));
+            const float v = ok ? sc[j][2 * r + e] * g.scale : -INFINITY;
+            sc[j][2 * r + e] = v;
+            mx = fmaxf(mx, v);
+          }
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+        const float m_new = fmaxf(m_run[r], mx), m_ref = m_new == -INFINITY ? 0.f : m_new;   // (-inf: nothing seen yet)
+        al[r] = m_new == -INFINITY ? 1.f : expf(m_run[r] - m_new);
+        float sum = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          __nv_bfloat162 pp;
+          pp.x = __float2bfloat16_rn(expf(sc[j][2 * r] - m_ref));        // exactly zero for a key that is not seen
+          pp.y = __float2bfloat16_rn(expf(sc[j][2 * r + 1] - m_ref));
+          sum += __bfloat162float(pp.x) + __bfloat162float(pp.y);
+          pa[j >> 1][(j & 1) * 2 + r] = *reinterpret_cast<uint32_t*>(&pp);
+        }
+        l_part[r] = fmaf(l_part[r], al[r], sum);
+        m_run[r] = m_new;
       }
-    bool ok[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = e >> 1, pi = pos0 + tqr[r];
-      const int kidx = blk * KV_BLOCK + warp * 8 + t2 + (e & 1);   // pooled block number, or token position
-      ok[e] = tqr[r] < nq && (pooled ? kidx < n_vis[r] : (kidx <= pi && (kidx >= vis[r].lo || kidx < vis[r].keep)));
-      sc[e] = ok[e] ? sc[e] * g.scale : -INFINITY;
+      for (int j = 0; j < NT; ++j)
+        if (j * 8 < dv) {
+          acc[j][0] *= al[0]; acc[j][1] *= al[0]; acc[j][2] *= al[1]; acc[j][3] *= al[1];
+          uint32_t vb[4];
+          pa_ldsm_x4_trans(vb, Vs + (size_t)lane * LDV + j * 8);
+          pa_mma(acc[j], pa[0], vb[0], vb[1]);
+          pa_mma(acc[j], pa[1], vb[2], vb[3]);
+        }
     }
-    float mx[2] = {fmaxf(sc[0], sc[1]), fmaxf(sc[2], sc[3])};
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-    }
-    if ((lane & 3) == 0) {
-      smax[warp * PA_QT + gq] = mx[0];
-      smax[warp * PA_QT + gq + 8] = mx[1];
-    }
-    __syncthreads();
-    float al[2];
-#pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      const int qi = gq + r * 8;
-      const float bm = fmaxf(fmaxf(smax[qi], smax[PA_QT + qi]), fmaxf(smax[2 * PA_QT + qi], smax[3 * PA_QT + qi]));
-      const float m_new = fmaxf(m_run[r], bm);
-      al[r] = m_new == -INFINITY ? 1.f : expf(m_run[r] - m_new);
-      const bf p0 = __float2bfloat16_rn(ok[2 * r] ? expf(sc[2 * r] - m_new) : 0.f);
-      const bf p1 = __float2bfloat16_rn(ok[2 * r + 1] ? expf(sc[2 * r + 1] - m_new) : 0.f);
-      l_part[r] = fmaf(l_part[r], al[r], __bfloat162float(p0) + __bfloat162float(p1));
-      m_run[r] = m_new;
-      __nv_bfloat162 pp;
-      pp.x = p0; pp.y = p1;
-      *reinterpret_cast<__nv_bfloat162*>(Ps + qi * LDP + warp * 8 + t2) = pp;
-    }
-    __syncthreads();
-    // ---- weighted sum of the values: this warp's groups of 8 columns
-    uint32_t a0[4], a1[4];
-    pa_ldsm_x4(a0, Ps + (size_t)(lane & 15) * LDP + (lane >> 4) * 8);
-    pa_ldsm_x4(a1, Ps + (size_t)(lane & 15) * LDP + 16 + (lane >> 4) * 8);
-#pragma unroll
-    for (int j = 0; j < MMA_NT; ++j) {
-      const int n0 = (warp + 4 * j) * 8;
-      if (n0 < dv) {
-        acc[j][0] *= al[0]; acc[j][1] *= al[0]; acc[j][2] *= al[1]; acc[j][3] *= al[1];
-        uint32_t vb2[4];
-        pa_ldsm_x4_trans(vb2, Vs + (size_t)lane * LDV + n0);
-        pa_mma(acc[j], a0, vb2[0], vb2[1]);
-        pa_mma(acc[j], a1, vb2[2], vb2[3]);
-      }
-    }
-    __syncthreads();   // this pass's buffers, maxima and weights are consumed
   }
-  // ---- row sums: over the quad, then over the warps
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     l_part[r] += __shfl_xor_sync(0xffffffffu, l_part[r], 1);
     l_part[r] += __shfl_xor_sync(0xffffffffu, l_part[r], 2);
   }
-  __syncthreads();
-  if ((lane & 3) == 0) {
-    smax[warp * PA_QT + gq] = l_part[0];
-    smax[warp * PA_QT + gq + 8] = l_part[1];
+  if (!SPLIT) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      if (tqr[r] >= nq) continue;
+      const float inv_l = 1.f / l_part[r];
+      bf* dst = out + ((size_t)(row0 + tqr[r]) * g.heads + h_base + (wr0 + gq + r * 8) % gs) * dv + t2;
+#pragma unroll
+      for (int j = 0; j < NT; ++j)
+        if (j * 8 < dv) *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(acc[j][2 * r] * inv_l, acc[j][2 * r + 1] * inv_l);
+    }
+    return;
   }
-  __syncthreads();
+  // ---- the four warps' states of the same rows meet, in warp order
+  __syncthreads();   // the ring is consumed
+  float* ms = reinterpret_cast<float*>(pam_smem);   // [4][16] maxima, [4][16] sums, [4][16][dv] accumulators
+  float* ls = ms + 4 * 16;
+  float* as = ls + 4 * 16;
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
-    const int qi = gq + r * 8;
-    if (tqr[r] >= nq) continue;
-    const float inv_l = 1.f / (smax[qi] + smax[PA_QT + qi] + smax[2 * PA_QT + qi] + smax[3 * PA_QT + qi]);
-    const size_t row = (size_t)(row0 + tqr[r]);
-    const int h = h_base + qi % gs;
-#pragma unroll
-    for (int j = 0; j < MMA_NT; ++j) {
-      const int n = (warp + 4 * j) * 8 + t2;
-      if (n < dv) {
-        __nv_bfloat162 pp;
-        pp.x = __float2bfloat16_rn(acc[j][2 * r] * inv_l); pp.y = __float2bfloat16_rn(acc[j][2 * r + 1] * inv_l);
-        *reinterpret_cast<__nv_bfloat162*>(out + (row * g.heads + h) * dv + n) = pp;
-      }
+    const int row = gq + r * 8;
+    if ((lane & 3) == 0) {
+      ms[warp * 16 + row] = m_run[r];
+      ls[warp * 16 + row] = l_part[r];
     }
+#pragma unroll
+    for (int j = 0; j < NT; ++j)
+      if (j * 8 < dv) *reinterpret_cast<float2*>(as + ((size_t)warp * 16 + row) * dv + j * 8 + t2) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
   }
+  __syncthreads();
+  for (int i = tid; i < nq * gs * (dv / 2); i += PA_THREADS) {
+    const int row = i / (dv / 2), col = (i % (dv / 2)) * 2;
+    const float m = fmaxf(fmaxf(ms[row], ms[16 + row]), fmaxf(ms[32 + row], ms[48 + row]));
+    float l = 0.f, o0 = 0.f, o1 = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = expf(ms[w * 16 + row] - m);   // zero for a warp that saw nothing (m is finite: every query sees itself)
+      const float2 a2 = *reinterpret_cast<const float2*>(as + ((size_t)w * 16 + row) * dv + col);
+      l = fmaf(f, ls[w * 16 + row], l);
+      o0 = fmaf(f, a2.x, o0);
+      o1 = fmaf(f, a2.y, o1);
+    }
+    *reinterpret_cast<__nv_bfloat162*>(out + ((size_t)(row0 + row / gs) * g.heads + h_base + row % gs) * dv + col) = __floats2bfloat162_rn(o0 / l, o1 / l);
+  }
+}
+
+template <int NT, bool SPLIT>
+cudaError_t launch_mma(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, const AttnSeq* seqs,
+                       const LatentTile* tiles, int n_tiles, const int32_t* block_table, int bt_stride, void* out, const PoolAttnGeom& g,
+                       cudaStream_t stream) {
+  using bf = __nv_bfloat16;
+  using SH = PaShape<SPLIT>;
+  // the ring; the queries staged before it and the states merged after it are smaller
+  const size_t smem = (size_t)SH::NST * SH::CPS * KV_BLOCK * (g.dim + 8 + g.vdim + 8) * sizeof(bf);   // <= 205 KB
+  static bool attr_set = false;
+  if (!attr_set) {
+    const cudaError_t e = cudaFuncSetAttribute(poolattn_mma_kernel<NT, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024);
+    if (e != cudaSuccess) return e;
+    attr_set = true;
+  }
+  static int group_on = -1;
+  if (group_on < 0) {
+    const char* e = getenv("TGIS_POOLATTN_GROUP");
+    group_on = (e && e[0] == '0') ? 0 : 1;
+  }
+  const int per_kv = g.heads / g.kv_heads;
+  const int gs = (group_on && per_kv <= 16 && 16 % per_kv == 0) ? per_kv : 1;
+  const dim3 grid(n_tiles, g.heads / gs, std::max(1, PA_QT * gs / SH::ROWS));
+  return launch_k(poolattn_mma_kernel<NT, SPLIT>, grid, dim3(PA_THREADS), smem, stream, reinterpret_cast<const bf*>(q),
+                  reinterpret_cast<const bf*>(k_cache), reinterpret_cast<const bf*>(v_cache), reinterpret_cast<const bf*>(pk),
+                  reinterpret_cast<const bf*>(pv), seqs, tiles, block_table, bt_stride, reinterpret_cast<bf*>(out), g, gs);
 }
 
 bool mma_eligible(const PoolAttnGeom& g, const void* q, const void* k, const void* v, const void* pk, const void* pv, const void* out) {
@@ -561,7 +629,7 @@ bool mma_eligible(const PoolAttnGeom& g, const void* q, const void* k, const voi
     on = (e && e[0] == '0') ? 0 : 1;
   }
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-  return on && g.dim % 16 == 0 && g.dim <= 16 * MMA_KS && g.vdim % 8 == 0 && g.vdim <= 32 * MMA_NT && al16(q) && al16(k) && al16(v) &&
+  return on && g.dim % 16 == 0 && g.dim <= 16 * MMA_KS && g.vdim % 8 == 0 && g.vdim <= 8 * MMA_MAX_NT && al16(q) && al16(k) && al16(v) &&
          al16(pk) && al16(pv) && al16(out);
 }
 
@@ -626,31 +694,18 @@ cudaError_t poolattn_pool_launch(const void* k_cache, const void* v_cache, void*
 }
 
 cudaError_t poolattn_launch(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, int dtype,
-                            const AttnSeq* seqs, const LatentTile* tiles, int n_tiles, const int32_t* block_table,
+                            const AttnSeq* seqs, const LatentTile* tiles, int n_tiles, int n_tokens, const int32_t* block_table,
                             int bt_stride, void* out, int out_dtype, const PoolAttnGeom& g, cudaStream_t stream) {
   if (n_tiles <= 0) return cudaSuccess;
   if (!geom_ok(g) || out_dtype != dtype) return cudaErrorInvalidValue;
   if (dtype == DT_BF16 && mma_eligible(g, q, k_cache, v_cache, pk, pv, out)) {
-    using bf = __nv_bfloat16;
-    const size_t smem = ((size_t)(PA_QT + PA_NST * KV_BLOCK) * (g.dim + 8) + (size_t)PA_NST * KV_BLOCK * (g.vdim + 8) + PA_QT * (KV_BLOCK + 8)) * sizeof(bf) +
-                        4 * PA_QT * sizeof(float);   // <= 108 KB
-    static bool attr_set = false;
-    if (!attr_set) {
-      const cudaError_t e = cudaFuncSetAttribute(poolattn_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 112 * 1024);
-      if (e != cudaSuccess) return e;
-      attr_set = true;
-    }
-    static int group_on = -1;
-    if (group_on < 0) {
-      const char* e = getenv("TGIS_POOLATTN_GROUP");
-      group_on = (e && e[0] == '0') ? 0 : 1;
-    }
-    const int per_kv = g.heads / g.kv_heads;
-    const int gs = (group_on && per_kv >= 2 && per_kv <= PA_QT && PA_QT % per_kv == 0) ? per_kv : 1;
-    const dim3 grid = gs > 1 ? dim3(n_tiles, g.kv_heads, gs) : dim3(n_tiles, g.heads, 1);
-    return launch_k(poolattn_mma_kernel, grid, dim3(PA_THREADS), smem, stream, reinterpret_cast<const bf*>(q),
-                    reinterpret_cast<const bf*>(k_cache), reinterpret_cast<const bf*>(v_cache), reinterpret_cast<const bf*>(pk),
-                    reinterpret_cast<const bf*>(pv), seqs, tiles, block_table, bt_stride, reinterpret_cast<bf*>(out), g, gs);
+    const bool split = n_tokens < 4 * n_tiles;   // mostly single tokens
+    auto run = [&](auto nt) {
+      constexpr int NT = decltype(nt)::value;
+      return split ? launch_mma<NT, true>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream)
+                   : launch_mma<NT, false>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream);
+    };
+    return g.vdim <= 128 ? run(std::integral_constant<int, 16>{}) : run(std::integral_constant<int, MMA_MAX_NT>{});
   }
   if (dtype == DT_BF16)
     return launch_fma<__nv_bfloat16>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream);

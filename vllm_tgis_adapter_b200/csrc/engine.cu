@@ -2404,7 +2404,7 @@ struct tgis_engine {
       CK(poolattn_prep_launch(pnx_y1, ld, l.c_q, l.c_k, l.c_v, l.in_bias, l.pa, l.cos_sin, eps, d_pos, d_slot, pnx_q, l.k_cache,
                               l.v_cache, A, T, stream));
       CK(poolattn_pool_launch(l.k_cache, l.v_cache, l.pk_cache, l.pv_cache, A, d_seqs, S, d_bt, bt_stride, l.pa, step_max_q, stream));
-      CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, l.pk_cache, l.pv_cache, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16,
+      CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, l.pk_cache, l.pv_cache, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16, T,
                          d_bt, bt_stride, pnx_oA, A, l.pa, stream));
       n_launches += l.pa.pool > 0 ? 3 : 2;
       pnx_gemm(pnx_oA, A, H * s.vdim, l.w_o, pnx_o, DT_F32, W, T, W, H * s.vdim);
@@ -2533,7 +2533,7 @@ struct tgis_engine {
     }
     CK(poolattn_prep_launch(pnx_y1, ld, l.c_q, l.c_k, l.c_v, l.in_bias, l.pa, l.cos_sin, eps, d_pos, d_slot, pnx_q, l.k_cache, l.v_cache,
                             A, T, stream));
-    CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, nullptr, nullptr, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16, d_bt,
+    CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, nullptr, nullptr, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16, T, d_bt,
                        bt_stride, pnx_oA, A, l.pa, stream));
     n_launches += 2;
     pnx_gemm(pnx_oA, A, H * s.vdim, l.w_o, pnx_o, DT_F32, W, T, W, H * s.vdim);

@@ -459,9 +459,9 @@ cudaError_t poolattn_prep_launch(const float* y, int ldy, int q_off, int k_off, 
 cudaError_t poolattn_pool_launch(const void* k_cache, const void* v_cache, void* pk, void* pv, int dtype,
                                  const AttnSeq* seqs, int n_seqs, const int32_t* block_table, int bt_stride,
                                  const PoolAttnGeom& g, int max_q_len, cudaStream_t stream);
-// out DT_* [T, heads * vdim]
+// out DT_* [T, heads * vdim]; n_tokens: the tiles' tokens together
 cudaError_t poolattn_launch(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, int dtype,
-                            const AttnSeq* seqs, const LatentTile* tiles, int n_tiles, const int32_t* block_table,
+                            const AttnSeq* seqs, const LatentTile* tiles, int n_tiles, int n_tokens, const int32_t* block_table,
                             int bt_stride, void* out, int out_dtype, const PoolAttnGeom& g, cudaStream_t stream);
 
 // ---- recurrent.cu: mixers that carry a state from token to token ----------------------------------------------------

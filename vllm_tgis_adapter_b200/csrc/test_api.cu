@@ -714,9 +714,10 @@ int tgis_k_poolattn(const void* q, const void* k_cache, const void* v_cache, voi
   std::vector<AttnSeq> seqs;
   host_seqs(seqs_host, n_seqs, seqs);
   std::vector<LatentTile> tiles;
-  int max_q = 0;
+  int max_q = 0, n_tok = 0;
   for (int i = 0; i < n_seqs; ++i) {
     max_q = std::max(max_q, seqs[i].q_len);
+    n_tok += seqs[i].q_len;
     for (int q0 = 0; q0 < seqs[i].q_len; q0 += POOLATTN_TILE) tiles.push_back(LatentTile{i, q0, std::min(POOLATTN_TILE, seqs[i].q_len - q0), 0});
   }
   Tmp<AttnSeq> d_seqs;
@@ -726,7 +727,7 @@ int tgis_k_poolattn(const void* q, const void* k_cache, const void* v_cache, voi
   KCK(d_tiles.upload(tiles.data(), tiles.size()));
   KCK(d_bt.upload(block_table_host, (size_t)bt_rows * bt_stride));
   KCK(poolattn_pool_launch(k_cache, v_cache, pk, pv, dt, d_seqs.p, n_seqs, d_bt.p, bt_stride, to_pool(g), max_q, 0));
-  KCK(poolattn_launch(q, k_cache, v_cache, pk, pv, dt, d_seqs.p, d_tiles.p, (int)tiles.size(), d_bt.p, bt_stride, out, dt, to_pool(g), 0));
+  KCK(poolattn_launch(q, k_cache, v_cache, pk, pv, dt, d_seqs.p, d_tiles.p, (int)tiles.size(), n_tok, d_bt.p, bt_stride, out, dt, to_pool(g), 0));
   KCK(cudaDeviceSynchronize());
   return 0;
 }
