@@ -365,8 +365,16 @@ __device__ __forceinline__ void pa_mma(float (&c)[4], const uint32_t (&a)[4], ui
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-template <int NT, bool SPLIT>
-__global__ void __launch_bounds__(PA_THREADS)
+// 2^x of the special function unit (relative error of a few 2^-23; results below 2^-126 become zero)
+__device__ __forceinline__ float pa_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// KS > 0: the sizes are compile-time constants, dim = 16 KS and vdim = 8 NT; KS = 0: any sizes with dim <= 16 MMA_KS, vdim <= 8 NT
+template <int KS, int NT, bool SPLIT>
+__global__ void __launch_bounds__(PA_THREADS, !SPLIT && NT <= 16 ? 3 : 1)
 poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
                     const __nv_bfloat16* __restrict__ v_cache, const __nv_bfloat16* __restrict__ pk,
                     const __nv_bfloat16* __restrict__ pv, const AttnSeq* __restrict__ seqs, const LatentTile* __restrict__ tiles,
@@ -377,7 +385,9 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   using bf = __nv_bfloat16;
   using SH = PaShape<SPLIT>;
   extern __shared__ __align__(16) uint8_t pam_smem[];
-  const int d = g.dim, dv = g.vdim, LDK = d + 8, LDV = dv + 8;
+  constexpr int KSM = KS > 0 ? KS : MMA_KS;
+  constexpr bool EXACT = KS > 0;
+  const int d = EXACT ? 16 * KS : g.dim, dv = EXACT ? 8 * NT : g.vdim, LDK = d + 8, LDV = dv + 8;
   bf* Ks2 = reinterpret_cast<bf*>(pam_smem);                     // [NST * CPS][32][LDK]   (first the queries: [ROWS][LDK])
   bf* Vs2 = Ks2 + (size_t)SH::NST * SH::CPS * KV_BLOCK * LDK;    // [NST * CPS][32][LDV]
   griddep_launch();
@@ -407,19 +417,22 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
   __syncthreads();
   const int nks = d / 16, wr0 = SPLIT ? 0 : warp * 16;   // the warp's first row
-  uint32_t qa[MMA_KS][4];
+  uint32_t qa[KSM][4];
 #pragma unroll
-  for (int ks = 0; ks < MMA_KS; ++ks)
-    if (ks < nks) pa_ldsm_x4(qa[ks], Ks2 + (size_t)(wr0 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
+  for (int ks = 0; ks < KSM; ++ks)
+    if (EXACT || ks < nks) pa_ldsm_x4(qa[ks], Ks2 + (size_t)(wr0 + (lane & 15)) * LDK + ks * 16 + (lane >> 4) * 8);
   __syncthreads();   // the ring may overwrite the queries
   float acc[NT][4];
 #pragma unroll
   for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+  // scores and maxima in units of ln 2: weights are powers of two
+  constexpr float LOG2E = 1.4426950408889634f;
+  const float scale2 = g.scale * LOG2E;
   float m_run[2] = {-INFINITY, -INFINITY}, l_part[2] = {0.f, 0.f};   // rows gq and gq + 8 of the warp
   if (g.sink != nullptr) {
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-      m_run[r] = g.sink[h_base + (wr0 + gq + r * 8) % gs];
+      m_run[r] = g.sink[h_base + (wr0 + gq + r * 8) % gs] * LOG2E;
       l_part[r] = ((!SPLIT || warp == 0) && (lane & 3) == 0) ? 1.f : 0.f;   // (the row's sum adds up the parts of all its threads)
     }
   }
@@ -428,8 +441,9 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   const int n_vis[2] = {pooled_visible(pos0 + tqr[0], g.window, g.pool), pooled_visible(pos0 + tqr[1], g.window, g.pool)};
   // the warp's first and last token: which chunks concern it at all
   const int tq_lo = wr0 / gs, tq_hi = min((wr0 + 15) / gs, nq - 1);
-  const Visible w_first = visible_tokens(pos0 + tq_lo, g);
-  const int w_pooled = pooled_visible(pos0 + tq_hi, g.window, g.pool);
+  const Visible w_first = visible_tokens(pos0 + tq_lo, g), w_last = visible_tokens(pos0 + tq_hi, g);
+  const int w_pooled = pooled_visible(pos0 + tq_hi, g.window, g.pool), w_pooled_all = pooled_visible(pos0 + tq_lo, g.window, g.pool);
+  const bool w_rows_all = (wr0 + 15) / gs < nq;
   const int n_pooled = pooled_visible(pos_last, g.window, g.pool);
   const Visible first = visible_tokens(pos0, g);
   const int blk0 = first.lo / KV_BLOCK, blk1 = pos_last / KV_BLOCK;
@@ -447,7 +461,7 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       const int b = blk * KV_BLOCK + fj;
       r = b < n_pooled ? (long long)pooled_row(b, g.pool, rpp, bt) : -1;
     } else {
-      r = (long long)bt[blk] * KV_BLOCK + fj;
+      r = (long long)__ldg(bt + blk) * KV_BLOCK + fj;
     }
     bf* Kd = Ks2 + ((size_t)buf * KV_BLOCK + fj) * LDK;
     bf* Vd = Vs2 + ((size_t)buf * KV_BLOCK + fj) * LDV;
@@ -492,8 +506,8 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
       for (int j = 0; j < 4; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
 #pragma unroll
-      for (int ks = 0; ks < MMA_KS; ++ks)
-        if (ks < nks) {
+      for (int ks = 0; ks < KSM; ++ks)
+        if (EXACT || ks < nks) {
 #pragma unroll
           for (int jj = 0; jj < 2; ++jj) {
             uint32_t kb[4];
@@ -502,42 +516,55 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
             pa_mma(sc[2 * jj + 1], qa[ks], kb[2], kb[3]);
           }
         }
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sc[j][e] *= scale2;
+      // a chunk that every row of the warp sees whole needs no mask
+      const bool whole = w_rows_all && (pooled ? key0 + KV_BLOCK <= w_pooled_all
+                                               : key0 + KV_BLOCK - 1 <= pos0 + tq_lo && (key0 >= w_last.lo || key0 + KV_BLOCK <= w_last.keep));
+      if (!whole) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int pi = tqr[r] < nq ? pos0 + tqr[r] : -1;
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              const int kidx = key0 + j * 8 + t2 + e;
+              const bool ok = pooled ? (pi >= 0 && kidx < n_vis[r]) : (kidx <= pi && (kidx >= vis[r].lo || kidx < vis[r].keep));
+              if (!ok) sc[j][2 * r + e] = -INFINITY;
+            }
+        }
+      }
       float al[2];
       uint32_t pa[2][4];   // the weights as A fragments of the two 16-key steps of the second product
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
-        const int pi = pos0 + tqr[r];
-        float mx = -INFINITY;
-#pragma unroll
-        for (int j = 0; j < 4; ++j)
-#pragma unroll
-          for (int e = 0; e < 2; ++e) {
-            const int kidx = key0 + j * 8 + t2 + e;
-            const bool ok = tqr[r] < nq && (pooled ? kidx < n_vis[r] : (kidx <= pi && (kidx >= vis[r].lo || kidx < vis[r].keep)));
-            const float v = ok ? sc[j][2 * r + e] * g.scale : -INFINITY;
-            sc[j][2 * r + e] = v;
-            mx = fmaxf(mx, v);
-          }
+        float mx = fmaxf(fmaxf(fmaxf(sc[0][2 * r], sc[0][2 * r + 1]), fmaxf(sc[1][2 * r], sc[1][2 * r + 1])),
+                         fmaxf(fmaxf(sc[2][2 * r], sc[2][2 * r + 1]), fmaxf(sc[3][2 * r], sc[3][2 * r + 1])));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
         const float m_new = fmaxf(m_run[r], mx), m_ref = m_new == -INFINITY ? 0.f : m_new;   // (-inf: nothing seen yet)
-        al[r] = m_new == -INFINITY ? 1.f : expf(m_run[r] - m_new);
+        al[r] = m_new == -INFINITY ? 1.f : pa_exp2(m_run[r] - m_new);
         float sum = 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          __nv_bfloat162 pp;
-          pp.x = __float2bfloat16_rn(expf(sc[j][2 * r] - m_ref));        // exactly zero for a key that is not seen
-          pp.y = __float2bfloat16_rn(expf(sc[j][2 * r + 1] - m_ref));
-          sum += __bfloat162float(pp.x) + __bfloat162float(pp.y);
-          pa[j >> 1][(j & 1) * 2 + r] = *reinterpret_cast<uint32_t*>(&pp);
+        for (int j = 0; j < 4; ++j) {   // exactly zero for a key that is not seen
+          const __nv_bfloat162 pp = __floats2bfloat162_rn(pa_exp2(sc[j][2 * r] - m_ref), pa_exp2(sc[j][2 * r + 1] - m_ref));
+          const float2 pf = __bfloat1622float2(pp);
+          sum += pf.x + pf.y;
+          pa[j >> 1][(j & 1) * 2 + r] = *reinterpret_cast<const uint32_t*>(&pp);
         }
         l_part[r] = fmaf(l_part[r], al[r], sum);
         m_run[r] = m_new;
       }
+      if (__any_sync(0xffffffffu, al[0] != 1.f || al[1] != 1.f)) {   // some row's maximum moved
+#pragma unroll
+        for (int j = 0; j < NT; ++j) { acc[j][0] *= al[0]; acc[j][1] *= al[0]; acc[j][2] *= al[1]; acc[j][3] *= al[1]; }
+      }
 #pragma unroll
       for (int j = 0; j < NT; ++j)
-        if (j * 8 < dv) {
-          acc[j][0] *= al[0]; acc[j][1] *= al[0]; acc[j][2] *= al[1]; acc[j][3] *= al[1];
+        if (EXACT || j * 8 < dv) {
           uint32_t vb[4];
           pa_ldsm_x4_trans(vb, Vs + (size_t)lane * LDV + j * 8);
           pa_mma(acc[j], pa[0], vb[0], vb[1]);
@@ -558,7 +585,7 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       bf* dst = out + ((size_t)(row0 + tqr[r]) * g.heads + h_base + (wr0 + gq + r * 8) % gs) * dv + t2;
 #pragma unroll
       for (int j = 0; j < NT; ++j)
-        if (j * 8 < dv) *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(acc[j][2 * r] * inv_l, acc[j][2 * r + 1] * inv_l);
+        if (EXACT || j * 8 < dv) *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(acc[j][2 * r] * inv_l, acc[j][2 * r + 1] * inv_l);
     }
     return;
   }
@@ -576,7 +603,7 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     }
 #pragma unroll
     for (int j = 0; j < NT; ++j)
-      if (j * 8 < dv) *reinterpret_cast<float2*>(as + ((size_t)warp * 16 + row) * dv + j * 8 + t2) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
+      if (EXACT || j * 8 < dv) *reinterpret_cast<float2*>(as + ((size_t)warp * 16 + row) * dv + j * 8 + t2) = make_float2(acc[j][2 * r], acc[j][2 * r + 1]);
   }
   __syncthreads();
   for (int i = tid; i < nq * gs * (dv / 2); i += PA_THREADS) {
@@ -585,7 +612,7 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     float l = 0.f, o0 = 0.f, o1 = 0.f;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float f = expf(ms[w * 16 + row] - m);   // zero for a warp that saw nothing (m is finite: every query sees itself)
+      const float f = pa_exp2(ms[w * 16 + row] - m);   // zero for a warp that saw nothing (m is finite: every query sees itself)
       const float2 a2 = *reinterpret_cast<const float2*>(as + ((size_t)w * 16 + row) * dv + col);
       l = fmaf(f, ls[w * 16 + row], l);
       o0 = fmaf(f, a2.x, o0);
@@ -595,7 +622,7 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   }
 }
 
-template <int NT, bool SPLIT>
+template <int KS, int NT, bool SPLIT>
 cudaError_t launch_mma(const void* q, const void* k_cache, const void* v_cache, const void* pk, const void* pv, const AttnSeq* seqs,
                        const LatentTile* tiles, int n_tiles, const int32_t* block_table, int bt_stride, void* out, const PoolAttnGeom& g,
                        cudaStream_t stream) {
@@ -605,7 +632,7 @@ cudaError_t launch_mma(const void* q, const void* k_cache, const void* v_cache, 
   const size_t smem = (size_t)SH::NST * SH::CPS * KV_BLOCK * (g.dim + 8 + g.vdim + 8) * sizeof(bf);   // <= 205 KB
   static bool attr_set = false;
   if (!attr_set) {
-    const cudaError_t e = cudaFuncSetAttribute(poolattn_mma_kernel<NT, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024);
+    const cudaError_t e = cudaFuncSetAttribute(poolattn_mma_kernel<KS, NT, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 208 * 1024);
     if (e != cudaSuccess) return e;
     attr_set = true;
   }
@@ -617,7 +644,7 @@ cudaError_t launch_mma(const void* q, const void* k_cache, const void* v_cache, 
   const int per_kv = g.heads / g.kv_heads;
   const int gs = (group_on && per_kv <= 16 && 16 % per_kv == 0) ? per_kv : 1;
   const dim3 grid(n_tiles, g.heads / gs, std::max(1, PA_QT * gs / SH::ROWS));
-  return launch_k(poolattn_mma_kernel<NT, SPLIT>, grid, dim3(PA_THREADS), smem, stream, reinterpret_cast<const bf*>(q),
+  return launch_k(poolattn_mma_kernel<KS, NT, SPLIT>, grid, dim3(PA_THREADS), smem, stream, reinterpret_cast<const bf*>(q),
                   reinterpret_cast<const bf*>(k_cache), reinterpret_cast<const bf*>(v_cache), reinterpret_cast<const bf*>(pk),
                   reinterpret_cast<const bf*>(pv), seqs, tiles, block_table, bt_stride, reinterpret_cast<bf*>(out), g, gs);
 }
@@ -700,12 +727,16 @@ cudaError_t poolattn_launch(const void* q, const void* k_cache, const void* v_ca
   if (!geom_ok(g) || out_dtype != dtype) return cudaErrorInvalidValue;
   if (dtype == DT_BF16 && mma_eligible(g, q, k_cache, v_cache, pk, pv, out)) {
     const bool split = n_tokens < 4 * n_tiles;   // mostly single tokens
-    auto run = [&](auto nt) {
-      constexpr int NT = decltype(nt)::value;
-      return split ? launch_mma<NT, true>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream)
-                   : launch_mma<NT, false>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream);
+    auto run = [&](auto ks, auto nt) {
+      constexpr int KS = decltype(ks)::value, NT = decltype(nt)::value;
+      return split ? launch_mma<KS, NT, true>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream)
+                   : launch_mma<KS, NT, false>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream);
     };
-    return g.vdim <= 128 ? run(std::integral_constant<int, 16>{}) : run(std::integral_constant<int, MMA_MAX_NT>{});
+    using std::integral_constant;
+    if (g.dim == 128 && g.vdim == 128) return run(integral_constant<int, 8>{}, integral_constant<int, 16>{});
+    if (g.dim == 64 && g.vdim == 64) return run(integral_constant<int, 4>{}, integral_constant<int, 8>{});
+    return g.vdim <= 128 ? run(integral_constant<int, 0>{}, integral_constant<int, 16>{})
+                         : run(integral_constant<int, 0>{}, integral_constant<int, MMA_MAX_NT>{});
   }
   if (dtype == DT_BF16)
     return launch_fma<__nv_bfloat16>(q, k_cache, v_cache, pk, pv, seqs, tiles, n_tiles, block_table, bt_stride, out, g, stream);
