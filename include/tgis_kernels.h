@@ -227,11 +227,12 @@ int tgis_k_outer_scan(int32_t mode, const float* q, const float* k, const float*
                       const float* fg, int32_t ldg, const float* ig_b, const float* fg_b, float gate_cap, float* S, float* n,
                       float* m, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const float* x, float* x_last,
                       int32_t width, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot);
-/* lightning attention: S <- decay_h S + silu(k) silu(v)^T, o = S^T silu(q); q, k [T, heads * dim], v [T, heads * vdim], decay device
+/* chunked != 0: csrc/lightning.cu (64 tokens at a time on the tensor cores, q / k / v in bf16); 0: outer_scan_kernel (fp32).
+ * lightning attention: S <- decay_h S + silu(k) silu(v)^T, o = S^T silu(q); q, k [T, heads * dim], v [T, heads * vdim], decay device
  * [heads], S [slots][heads][dim][vdim] */
 int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_t ldq, int32_t ldk, int32_t ldv, const float* decay,
                           float* S, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const int32_t* seqs_host,
-                          int32_t n_seqs, const int32_t* tok_slot);
+                          int32_t n_seqs, const int32_t* tok_slot, int32_t chunked);
 int tgis_k_head_norm_gate(const float* o, int32_t ldo, int32_t heads, int32_t vdim, const float* w, const float* gate, int32_t ldg,
                           int32_t act, float eps, void* out, int32_t out_dt, int32_t T);
 /* resid += rmsnorm((rmsnorm(y_main) * w_main + rmsnorm(y_pair) * w_pair) / 2) * w_post; out = rmsnorm(resid) * w_pre, or the

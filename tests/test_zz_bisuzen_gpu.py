@@ -230,8 +230,11 @@ def test_sink_of_each_head_takes_its_weight():
 
 
 # ====================================================================================================== lightning attention
-@pytest.mark.parametrize("H,d,dv", [(3, 6, 5), (2, 70, 40), (1, 1, 1), (2, 130, 33), (4, 48, 64), (2, 128, 128), (1, 64, 200)])
-def test_lightning_scan_in_portions_and_two_slots_matches_oracle(H, d, dv):
+@pytest.mark.parametrize("chunked,H,d,dv", [(1, 2, 16, 8), (1, 3, 48, 72), (1, 2, 128, 128), (1, 4, 64, 64), (1, 1, 80, 136), (1, 1, 32, 200)] + [
+    (0, *s) for s in [(3, 6, 5), (2, 70, 40), (1, 1, 1), (2, 130, 33), (4, 48, 64), (2, 128, 128), (1, 64, 200)]])
+def test_lightning_scan_in_portions_and_two_slots_matches_oracle(chunked, H, d, dv):
+    """chunked: the tensor-core form rounds q, k and v to bf16 after silu, and so does the reference here; everything the recurrence
+    adds stays fp32-like, so the bound is far below bf16's."""
     from oracle import bisuzen_oracle as O
 
     g = torch.Generator().manual_seed(3)
@@ -242,6 +245,8 @@ def test_lightning_scan_in_portions_and_two_slots_matches_oracle(H, d, dv):
     for h in seqs:
         h = h.double()
         q, k, v = O.silu(h[:, :H * d]).view(-1, H, d), O.silu(h[:, H * d:2 * H * d]).view(-1, H, d), O.silu(h[:, 2 * H * d:]).view(-1, H, dv)
+        if chunked:
+            q, k, v = (x.float().to(torch.bfloat16).double() for x in (q, k, v))
         S = torch.zeros(H, d, dv, dtype=F64)
         o = []
         for t in range(h.shape[0]):
@@ -268,7 +273,7 @@ def test_lightning_scan_in_portions_and_two_slots_matches_oracle(H, d, dv):
             _KEEP.append(y)
             out = torch.zeros(y.shape[0], H * dv, device="cuda")
             _ok(_lib().tgis_k_lightning_scan(_p(y), _p(y[:, H * d:]), _p(y[:, 2 * H * d:]), width, width, width, _p(dec), _p(S_dev), _p(out),
-                                             H * dv, H, d, dv, _ints(meta), len(meta) // 4, _p(_i32(tok_slot))))
+                                             H * dv, H, d, dv, _ints(meta), len(meta) // 4, _p(_i32(tok_slot)), chunked))
             o = 0
             for s, a, n in dst:
                 outs[s][a:a + n] = out[o:o + n]
@@ -276,7 +281,8 @@ def test_lightning_scan_in_portions_and_two_slots_matches_oracle(H, d, dv):
             step += 1
         for s in (0, 1):
             err = (outs[s].double().cpu() - refs[s]).abs().max()
-            assert float(err) < 2e-5 * max(1.0, float(refs[s].abs().max())), (sizes, s)
+            # (a value that sits on a bf16 rounding boundary may round the other way than the reference's)
+            assert float(err) < (2e-4 if chunked else 2e-5) * max(1.0, float(refs[s].abs().max())), (sizes, s)
 
 
 # ====================================================================================================== router and tails

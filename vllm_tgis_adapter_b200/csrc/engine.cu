@@ -302,6 +302,7 @@ struct tgis_engine {
   void *pnx_side = nullptr, *pnx_hB = nullptr;       // side table [vocab, n_layers * side_dim]; norm2's rows (operand type)
   float* pnx_x0 = nullptr;                           // the embedding output, kept for the passes of a loop
   int step_max_q = 0;                                // longest portion of the step
+  int step_n_lead1 = 0;                              // single-token sequences at the front of the step (before its portions)
   // the feed-forward of a parallel pair layer reads the same stream as the mixer: its two products run on a second stream
   // beside the mixer's kernels (fork after the tail that leaves both normed inputs, join before the tail that adds both
   // outputs), with a product workspace of their own.  TGIS_PAIR_OVERLAP=0: one stream
@@ -1431,6 +1432,7 @@ struct tgis_engine {
           CK(cudaMemcpy(l.decay, pnx_decays[i].data(), sizeof(float) * s.mm_heads, cudaMemcpyHostToDevice));
           pnx_expected_tensors += 8;  // right.{q, k, v, g, norm, o, out}, left.out
           m_f1 = std::max(m_f1, mv);
+          m_mix = std::max(m_mix, (size_t)2 * s.mm_heads * s.mm_dim + mv);
         }
         m_q = std::max<size_t>(m_q, (size_t)H * s.dim);
         m_ov = std::max<size_t>(m_ov, (size_t)H * s.vdim);
@@ -2517,7 +2519,18 @@ struct tgis_engine {
       os.S = l.st_S;
       os.out = flx_f1; os.ldo = mv;
       os.heads = mH; os.dim = s.mm_dim; os.vdim = s.mm_vdim;
-      CK(outer_scan_launch(os, d_seqs, S, d_tokslot, st));
+      // bf16 portions: chunk by chunk on the tensor cores; single tokens (the step's first sequences) and fp32: token by token
+      const int qkv = 2 * mH * s.mm_dim + mv;   // q' | k' | v' are neighbours in the projection
+      const int lead = step_n_lead1;
+      if (A == DT_BF16 && lead < S && lightning_chunk_eligible(s.mm_dim, s.mm_vdim) && l.c_mq % 4 == 0) {
+        CK(silu_cast_launch(pnx_y1 + l.c_mq, ld, flx_mix, qkv, qkv, T, st));
+        const LightningChunk lc{flx_mix, qkv, 0, l.c_mk - l.c_mq, l.c_mv - l.c_mq, l.decay, l.st_S, flx_f1, mv, mH, s.mm_dim, s.mm_vdim};
+        CK(lightning_chunk_launch(lc, d_seqs + lead, S - lead, d_tokslot, st));
+        if (lead > 0) CK(outer_scan_launch(os, d_seqs, lead, d_tokslot, st));
+        n_launches += lead > 0 ? 2 : 1;
+      } else {
+        CK(outer_scan_launch(os, d_seqs, S, d_tokslot, st));
+      }
       CK(head_norm_gate_launch(flx_f1, mv, 1, mv, l.mm_norm, pnx_y1 + l.c_mg, ld, /*sigmoid*/ 0, eps, flx_op2, A, T, st));
       n_launches += 2;
       pnx_gemm(flx_op2, A, mv, l.w_o2, pnx_yS, DT_F32, W, T, W, mv);
@@ -3152,6 +3165,7 @@ struct tgis_engine {
     step_n_ltiles = 0;
     step_n_ltiles16 = 0;
     step_max_q = 0;
+    step_n_lead1 = 0;
     step_max_kv = 0;
     for (int s = 0; s < S; ++s) {
       Request& r = *batch[s].r;
@@ -3185,6 +3199,7 @@ struct tgis_engine {
           for (int q0 = 0; q0 < q_len; q0 += POOLATTN_TILE)
             lt16[step_n_ltiles16++] = LatentTile{s, q0, std::min(POOLATTN_TILE, q_len - q0), 0};
           step_max_q = std::max(step_max_q, q_len);
+          if (q_len == 1 && step_n_lead1 == s) ++step_n_lead1;
         }
       }
       if (q_len == 1) {

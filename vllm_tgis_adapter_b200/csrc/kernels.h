@@ -523,6 +523,19 @@ struct OuterScan {
 };
 cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot,
                               cudaStream_t stream);
+// lightning.cu: the recurrence of OUTER_SCAN_LIGHTNING over whole portions, 64 tokens at a time on the tensor cores, from q, k, v in
+// bf16 after silu (outer_scan_launch keeps them fp32).  For steps that carry prompts.
+struct LightningChunk {
+  const void* qkv; int ld, q_off, k_off, v_off;   // bf16 [T, ld]: q and k [heads * dim], v [heads * vdim] at the given columns
+  const float* decay;                             // [heads]
+  float* S;                                       // [slots][heads][dim][vdim]
+  float* out; int ldo;                            // fp32 [T, heads * vdim]
+  int heads, dim, vdim;
+};
+bool lightning_chunk_eligible(int dim, int vdim);
+// out[t, i] = silu(x[t, i]) in bf16, i < n (n, ldx, ldo multiples of 4)
+cudaError_t silu_cast_launch(const float* x, int ldx, void* out, int ldo, int n, int T, cudaStream_t stream);
+cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot, cudaStream_t stream);
 // out[t, h, :] = rmsnorm(o[t, h, :]) * w[h, :] * act(gate[t, h, :])    act: 0 sigmoid, 1 silu, 2 none (gate may be nullptr)
 // gate_first != 0: out[t, h, :] = rmsnorm(o[t, h, :] * act(gate[t, h, :])) * w[h, :]   (the gate enters the norm)
 cudaError_t head_norm_gate_launch(const float* o, int ldo, int heads, int vdim, const float* w, const float* gate,

@@ -822,7 +822,7 @@ int tgis_k_outer_scan(int32_t mode, const float* q, const float* k, const float*
 
 int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_t ldq, int32_t ldk, int32_t ldv, const float* decay,
                           float* S, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const int32_t* seqs_host,
-                          int32_t n_seqs, const int32_t* tok_slot) {
+                          int32_t n_seqs, const int32_t* tok_slot, int32_t chunked) {
   std::vector<AttnSeq> seqs;
   host_seqs(seqs_host, n_seqs, seqs);
   Tmp<AttnSeq> d_seqs;
@@ -831,6 +831,19 @@ int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_
   a.mode = OUTER_SCAN_LIGHTNING;
   a.q = q; a.k = k; a.v = v; a.ldq = ldq; a.ldk = ldk; a.ldv = ldv; a.q_scale = 1.f;
   a.decay = decay; a.S = S; a.out = out; a.ldo = ldo; a.heads = heads; a.dim = dim; a.vdim = vdim;
+  if (chunked) {
+    int T = 0;
+    for (const AttnSeq& s : seqs) T += s.q_len;
+    const int hd = heads * dim, hv = heads * vdim, n = 2 * hd + hv;
+    Tmp<__nv_bfloat16> qkv;
+    KCK(qkv.alloc((size_t)T * n));
+    KCK(silu_cast_launch(q, ldq, qkv.p, n, hd, T, 0));
+    KCK(silu_cast_launch(k, ldk, qkv.p + hd, n, hd, T, 0));
+    KCK(silu_cast_launch(v, ldv, qkv.p + 2 * hd, n, hv, T, 0));
+    KCK(lightning_chunk_launch(LightningChunk{qkv.p, n, 0, hd, 2 * hd, decay, S, out, ldo, heads, dim, vdim}, d_seqs.p, n_seqs, tok_slot, 0));
+    KCK(cudaDeviceSynchronize());
+    return 0;
+  }
   KCK(outer_scan_launch(a, d_seqs.p, n_seqs, tok_slot, 0));
   KCK(cudaDeviceSynchronize());
   return 0;

@@ -242,7 +242,7 @@ def load_library() -> C.CDLL:
     lib.tgis_k_selective_scan.argtypes = [vp, vp, i32, vp, i32, i32, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp]
     lib.tgis_k_outer_scan.argtypes = [i32, vp, vp, vp, i32, i32, i32, f32, vp, i32, vp, vp, vp, vp, i32, vp, vp, f32, vp, vp, vp,
                                       vp, i32, i32, i32, i32, vp, vp, i32, ip, i32, vp]
-    lib.tgis_k_lightning_scan.argtypes = [vp, vp, vp, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp]
+    lib.tgis_k_lightning_scan.argtypes = [vp, vp, vp, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp, i32]
     lib.tgis_k_head_norm_gate.argtypes = [vp, i32, i32, i32, vp, vp, i32, i32, f32, vp, i32, i32]
     lib.tgis_k_resid_tail_pair.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, f32, i32, i32]
     _LIB = lib
