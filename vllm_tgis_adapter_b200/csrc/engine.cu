@@ -292,6 +292,7 @@ struct tgis_engine {
     // k_cache / v_cache; lightning side: c_mq .. c_mg, w_o2, mm_norm, st_S, out_l / out_r; experts: w_router, router_b (correction),
     // w_gu_e (up-projections), w_d_e
     DytNorm dyt1{}, dyt2{};
+    int router_cols = 0;                             // rows of w_router: the router's outputs and zero rows
     float *o_bias = nullptr, *decay = nullptr;       // [width] output bias of the attention; [mm_heads] decays
     int c_f = 0;                      // TGIS_MIXER_HGRN (w_in: q | f | v): column of the gate logits
   };
@@ -1386,12 +1387,14 @@ struct tgis_engine {
           m_ffs = std::max<size_t>(m_ffs, s.ff);
         } else if (s.mlp == TGIS_MLP_MOE_GROUPED) {
           const size_t E = s.experts, n_out = E + s.identity, ff = s.expert_ff;
-          l.w_router = pnx_alloc_dt(n_out * W);
+          // zero rows up to a full weight tile: prompts take the router's product through the tcgen05 kernel
+          l.router_cols = (int)std::max<size_t>((n_out + 7) / 8 * 8, 128);
+          l.w_router = pnx_alloc_dt((size_t)l.router_cols * W, true);
           l.router_b = pnx_alloc<float>(n_out);
           l.w_gu_e = pnx_alloc_dt(E * ff * W);     // up-projections, one [ff, width] matrix per expert
           l.w_d_e = pnx_alloc_dt(E * W * ff);
           pnx_expected_tensors += 2 + 2 * E;       // router, correction, e<j>.{up, down}
-          m_E = std::max(m_E, n_out); m_top = std::max<size_t>(m_top, s.top); m_ff = std::max(m_ff, ff);
+          m_E = std::max<size_t>(m_E, l.router_cols); m_top = std::max<size_t>(m_top, s.top); m_ff = std::max(m_ff, ff);
         }
         const int H = s.heads, G = s.kv_heads;
         const bool par = s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
@@ -2570,8 +2573,9 @@ struct tgis_engine {
         ft.y_main = pnx_o;
       } else {  // TGIS_MLP_MOE_GROUPED
         const int E = s.experts, n_out = E + s.identity, top = s.top, ff = s.expert_ff;
-        pnx_gemm(pnx_hA, A, W, l.w_router, pnx_rl, DT_F32, n_out, T, n_out, W);
-        CK(moe_route_launch(pnx_rl, n_out, l.router_b, n_out, top, pnx_ids, pnx_mixw, nullptr, T, stream, MOE_W_SHARE, s.expert_groups,
+        const int n_rl = A == DT_BF16 && T > 256 && W % 64 == 0 ? l.router_cols : n_out;
+        pnx_gemm(pnx_hA, A, W, l.w_router, pnx_rl, DT_F32, n_rl, T, n_rl, W);
+        CK(moe_route_launch(pnx_rl, n_rl, l.router_b, n_out, top, pnx_ids, pnx_mixw, nullptr, T, stream, MOE_W_SHARE, s.expert_groups,
                             s.expert_groups_keep));
         // one row segment per output; those of the identity experts come last and enter no product
         CK(moe_align_launch(pnx_ids, T, top, n_out, pnx_segoff, pnx_order, pnx_inv, stream));
