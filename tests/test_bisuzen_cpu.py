@@ -59,6 +59,8 @@ def test_config_json_to_specs():
             model_config_from_json({**CFG, "layers": [{**CFG["layers"][0], **bad}]}, None)
     with pytest.raises(ValueError):   # one decay per head
         model_config_from_json({**CFG, "layers": [{**CFG["layers"][1], "mixer": {"left": LEFT, "right": {**RIGHT, "heads": 3}}}]}, None)
+    empty, _ = model_spec(model_config_from_json({**CFG, "loop": {"start": 2, "stop": 2, "times": 4}}, None))
+    assert (empty.loop_start, empty.loop_stop, empty.loop_times) == (0, 0, 1)
     plain = model_config_from_json({k: v for k, v in CFG.items() if k not in ("loop", "logit_scale")}, None)
     assert (plain.loop[2], plain.logit_scale) == (1, 1.0)
 

@@ -160,7 +160,7 @@ def model_spec(mc: ModelConfig):
     spec.embed_scale, spec.residual_mult, spec.norm_eps = 1.0, 1.0, mc.rms_eps
     spec.logit_scale = mc.logit_scale
     spec.style = _lib.STYLE_PRE_DYT
-    spec.loop_start, spec.loop_stop, spec.loop_times = mc.loop
+    spec.loop_start, spec.loop_stop, spec.loop_times = mc.loop if mc.loop[1] > mc.loop[0] else (0, 0, 1)   # (an empty span: no loop)
     spec.layers = C.cast(arr, C.POINTER(_lib.TgisLayerSpec))
     return spec, keep
 
