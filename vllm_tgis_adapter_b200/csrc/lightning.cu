@@ -68,6 +68,7 @@ silu_cast_kernel(const float* __restrict__ x, int ldx, bf* __restrict__ out, int
   griddep_launch();
   griddep_wait();
   const int t = blockIdx.x;
+#pragma unroll 4
   for (int i = (blockIdx.y * 256 + threadIdx.x) * 4; i < n; i += gridDim.y * 1024) {
     const float4 v = *reinterpret_cast<const float4*>(x + (size_t)t * ldx + i);
     // (fast forms: their error is far below the rounding to bf16)
@@ -311,7 +312,7 @@ cudaError_t silu_cast_launch(const float* x, int ldx, void* out, int ldo, int n,
   if (T <= 0 || n <= 0) return cudaSuccess;
   if (n % 4 != 0 || ldx % 4 != 0 || ldo % 4 != 0 || (reinterpret_cast<uintptr_t>(x) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 7) != 0)
     return cudaErrorInvalidValue;
-  return launch_k(silu_cast_kernel, dim3(T, std::min((n + 1023) / 1024, 8)), dim3(256), 0, stream, x, ldx, reinterpret_cast<bf*>(out), ldo, n);
+  return launch_k(silu_cast_kernel, dim3(T, std::min((n + 1023) / 1024, 2)), dim3(256), 0, stream, x, ldx, reinterpret_cast<bf*>(out), ldo, n);
 }
 
 cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot, cudaStream_t stream) {
