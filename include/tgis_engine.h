@@ -39,7 +39,7 @@
 extern "C" {
 #endif
 
-#define TGIS_ABI_VERSION 12
+#define TGIS_ABI_VERSION 13
 #define TGIS_MAX_REQUEST_ID 96
 #define TGIS_MAX_TOPN 12 /* reference forces max_logprobs >= 11: tgis_utils/args.py:214-216 */
 #define TGIS_MAX_STOP_TOKEN_IDS 8
@@ -103,6 +103,15 @@ typedef struct tgis_engine tgis_engine;
  *          (TGIS_MLP_MOE_GROUPED).  Logits times logit_scale.  bf16 or fp32 operands.  Single GPU, no LoRA slots. */
 #define TGIS_ARCH_BISUZEN 6
 
+/*   LUDELIX: a layer list as well (tgis_engine_create_spec), fp32 residual stream.  Sublayers are pre-normed with plain RMS weights,
+ *          x += mixer(rms(x) w1); x += ff(rms(x) w2) (TGIS_STYLE_PRE_RMS), logits from the embedding table (TGIS_STYLE_TIED_HEAD).
+ *          Mixers: chunked attention with a gate per head beside retention, their outputs weighed by two constants
+ *          (TGIS_MIXER_CHUNK_RETENTION); windowed attention with a sink whose values are the projected keys
+ *          (TGIS_MIXER_POOLED_ATTENTION + flags); gated linear attention (TGIS_MIXER_GLA).  Feed-forward: squared relu
+ *          (TGIS_MLP_DENSE_RELU2) or experts chosen by a table of the token id (TGIS_MLP_MOE_TABLE).  bf16 or fp32 operands.
+ *          Single GPU, no LoRA slots. */
+#define TGIS_ARCH_LUDELIX 7
+
 /* Model + runtime configuration (bf16 decoder-only transformer; see TGIS_ARCH_*). */
 typedef struct tgis_config {
   int32_t abi_version; /* must be TGIS_ABI_VERSION */
@@ -156,6 +165,11 @@ typedef struct tgis_config {
 #define TGIS_MIXER_WINDOW_LIGHTNING 10 /* left: grouped-query attention as TGIS_MIXER_POOLED_ATTENTION; right: lightning attention (an
                                        * outer-product memory with one fixed decay per head); both outputs rms-normed over the
                                        * width with a plain weight, averaged */
+#define TGIS_MIXER_CHUNK_RETENTION 11 /* left: grouped-query attention as TGIS_MIXER_POOLED_ATTENTION; right: retention (an outer-product
+                                      * memory with one fixed decay per head on rotated queries and keys, every head's output divided
+                                      * by its root mean square, silu gate); left_scale * left + right_scale * right */
+#define TGIS_MIXER_GLA 12            /* gated linear attention: outer-product memory whose key channels decay by
+                                      * sigmoid(low-rank map + bias)^(1 / tau), head norm, silu gate */
 #define TGIS_MLP_NONE 0
 #define TGIS_MLP_MOE 1
 #define TGIS_MLP_DENSE_GELU 2        /* down(gelu_tanh(gate h) * (up h)), width `ff` */
@@ -166,6 +180,9 @@ typedef struct tgis_config {
                                       * softmax over all of them, choice by score + correction among the best expert_groups_keep of
                                       * expert_groups equal groups (a group counts as its best choice score), weights: the chosen
                                       * scores divided by their sum */
+#define TGIS_MLP_DENSE_RELU2 6       /* down(relu(up h)^2), width `ff` */
+#define TGIS_MLP_MOE_TABLE 7         /* experts down(silu(gate h) * (up h)); "l<i>.mlp.table" (int32 [vocab, top]) names each token id's
+                                      * experts, each of weight 1 / top; shared expert of width shared_ff (0: none) under a sigmoid gate */
 /* tgis_layer_spec.flags */
 #define TGIS_LAYER_ROT_INTERLEAVED 1 /* rotary pairs are (2i, 2i + 1) instead of (i, i + rot_dims / 2) */
 #define TGIS_LAYER_SINK 2            /* the softmax denominator of head h also holds exp(sink_h): "l<i>.mix.sink" */
@@ -173,6 +190,9 @@ typedef struct tgis_config {
 #define TGIS_LAYER_QKV_BIAS 8        /* "l<i>.mix.q.b|k.b|v.b" are added to the projections */
 #define TGIS_LAYER_UNIT_QK 16        /* queries and keys are divided by their root mean square per head after the rotation */
 #define TGIS_LAYER_OUT_BIAS 32       /* the attention's output projection has a bias: "o.b" */
+#define TGIS_LAYER_SHARED_KV 64      /* no value projection: values are the keys as projected (bias included, before norm and rotation) */
+#define TGIS_LAYER_FULL_QK_NORM 128  /* queries and keys are rms-normed over all heads at once before the rotation ("q.norm", "k.norm") */
+#define TGIS_LAYER_HEAD_GATE 256     /* head h's output times sigmoid(W_g h)_h ("g": [heads, width]) */
 typedef struct tgis_layer_spec {
   int32_t mixer;        /* TGIS_MIXER_* */
   int32_t heads, dim, rot_dim, vdim, kv_rank, q_rank; /* per head: dim unrotated + rot_dim rotated query/key dims, vdim values */
@@ -224,7 +244,16 @@ typedef struct tgis_layer_spec {
   int32_t reserved2;
   /* TGIS_MIXER_WINDOW_LIGHTNING, right side: mm_heads heads, queries / keys of mm_dim, values of mm_vdim; decay [mm_heads] (host
    * memory, read by tgis_engine_create_spec) */
-  const float* decay;
+  const float* decay;   /* TGIS_MIXER_CHUNK_RETENTION reads mm_heads / mm_dim / mm_vdim / decay alike */
+  /* rotary frequencies by wavelength l = 2 pi / f (band_factor > 0): f where l < band_original / band_high, f / band_factor where
+   * l > band_original / band_low, between them (1 - s) f / band_factor + s f with s = (band_original / l - band_low) / (band_high - band_low) */
+  float band_factor, band_original, band_low, band_high;
+  /* TGIS_MIXER_CHUNK_RETENTION: rotation of the right side (the left side: rot_dims / rot_base / yarn_*), weights of both outputs */
+  float mm_rot_base;
+  int32_t mm_rot_dims;
+  float left_scale, right_scale;
+  float tau;            /* TGIS_MIXER_GLA: heads x dim queries / keys, heads x vdim values, decay_rank the low-rank map's inner size */
+  int32_t reserved3;
 } tgis_layer_spec;
 #define TGIS_STYLE_POST_NORM 1 /* x += rmsnorm(sublayer(x)) * w with a plain weight; unset: pre- and post-norm, weights stored
                                 * as deviations from one */
@@ -234,6 +263,7 @@ typedef struct tgis_layer_spec {
                                      * input (side_dim > 0): x += rms(side.proj (gelu_tanh(side.gate x) * e)) * side.norm */
 #define TGIS_STYLE_PRE_DYT 16       /* every norm is tanh(alpha x) * w + b ("<norm>", "<norm>.b", "<norm>.alpha"); x += mixer(dyt1(x)), then
                                      * x += ff(dyt2(x)) */
+#define TGIS_STYLE_PRE_RMS 32       /* x += mixer(rms(x) * norm1), then x += ff(rms(x) * norm2), plain weights */
 #define TGIS_DTYPE_BF16 0 /* bf16 operands, fp32 accumulation; norms, softmax, routers and the residual sum in fp32 */
 #define TGIS_DTYPE_F32 1  /* everything in true fp32 (no TF32) */
 typedef struct tgis_model_spec {
@@ -371,11 +401,15 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
 /* cfg->arch == TGIS_ARCH_BISUZEN; parameter names: "embed", "head", every norm as "<norm>|<norm>.b|<norm>.alpha" (alpha: one number):
  * "final.norm", "l<i>.norm1|norm2"; "l<i>.mlp.gate|up|down" or "l<i>.mlp.router|correction|e<j>.up|e<j>.down"; TGIS_MIXER_POOLED_ATTENTION
  * "l<i>.mix.q|k|v|o"; TGIS_MIXER_WINDOW_LIGHTNING "l<i>.mix.left.q|q.b|k|k.b|v|v.b|sink|o|o.b|out", "l<i>.mix.right.q|k|v|g|norm|o|out". */
+/* cfg->arch == TGIS_ARCH_LUDELIX; parameter names: "embed", "final.norm", "l<i>.norm1|norm2", "l<i>.mlp.up|down" or "l<i>.mlp.table
+ * (dtype 1)|e<j>.gate|e<j>.up|e<j>.down|shared.gate|shared.up|shared.down|shared.sg"; TGIS_MIXER_POOLED_ATTENTION "l<i>.mix.q|q.b|q.norm|k|
+ * k.b|k.norm|sink|o"; TGIS_MIXER_CHUNK_RETENTION "l<i>.mix.left.q|k|v|g|o", "l<i>.mix.right.q|k|v|g|o"; TGIS_MIXER_GLA "l<i>.mix.q|k|v|g|
+ * o|norm|a1|a2|a2.b". */
 /* name: HF Llama parameter name ("model.layers.3.self_attn.q_proj.weight", "lm_head.weight", ...) or
  * "tgis.rope_cos_sin" ([max_model_len,128] bf16 = cos|sin); arch OPT: HF OPT parameter names
  * ("model.decoder.layers.3.self_attn.q_proj.bias", "model.decoder.embed_positions.weight" with >= max_model_len + 2 rows,
  * ...; a 1-D tensor is passed as rows = n, cols = 1).  ptr may be host or device memory (cudaMemcpyDefault);
- * dtype 0 = bf16.  rows/cols describe the full (unsharded) tensor. */
+ * dtype 0 = bf16, 1 = int32 (tables of the layer-list architectures).  rows/cols describe the full (unsharded) tensor. */
 int tgis_engine_load_weight(tgis_engine* e, const char* name, const void* ptr, int64_t rows, int64_t cols, int32_t dtype);
 int tgis_engine_start(tgis_engine* e);
 int tgis_engine_add_request(tgis_engine* e, const char* request_id, const int32_t* prompt_ids, int32_t n_prompt,

@@ -9,6 +9,7 @@
 // weight but without a value had been seen.
 //
 //   poolattn_prep_kernel   per token and head: bias, rotary turn (fp32 table), unit RMS norm of queries and keys, cache write
+//   poolattn_prep_full_kernel  the same with queries and keys normed over all heads at once, values optionally the projected keys
 //   poolattn_pool_kernel   the blocks that this step's tokens complete: mean of the block's cache rows -> the pooled cache
 //   poolattn_mma_kernel    bf16 rows whose sizes fit the MMA tiles: both products on mma.sync with fp32 accumulators
 //   poolattn_kernel        any sizes and fp32 rows (FMA pipe)
@@ -66,6 +67,11 @@ __device__ __forceinline__ Visible visible_tokens(int pos, const PoolAttnGeom& g
   const int wl = g.window > 0 ? max(0, pos - g.window + 1) : 0;
   return {max(cl, wl), cl > 0 ? 0 : g.keep_first};
 }
+// factor on the outputs of head h at token row t
+__device__ __forceinline__ float out_factor(const PoolAttnGeom& g, int t, int h) {
+  return g.head_gate != nullptr ? g.out_mul / (1.f + expf(-g.head_gate[(size_t)t * g.gate_ld + h])) : g.out_mul;
+}
+__device__ __forceinline__ size_t out_row(const PoolAttnGeom& g, int t) { return (size_t)t * (g.out_ld > 0 ? g.out_ld : g.heads * g.vdim); }
 // row of pooled block b inside the pooled cache (page table bt of the sequence)
 __device__ __forceinline__ size_t pooled_row(int b, int pool, int rpp, const int32_t* bt) {
   const int page = (int)(((long long)b * pool) / KV_BLOCK);
@@ -124,9 +130,74 @@ poolattn_prep_kernel(const float* __restrict__ y, int ldy, int q_off, int k_off,
   } else if (slot >= 0) {
     const int h = hh - g.heads - g.kv_heads;
     const float* src = y + (size_t)t * ldy + v_off + (size_t)h * g.vdim;
-    const float* b = bias != nullptr ? bias + nq + nk + (size_t)h * g.vdim : nullptr;
+    const float* b = bias != nullptr ? bias + nq + (v_off == k_off ? 0 : nk) + (size_t)h * g.vdim : nullptr;
     CT* dst = v_cache + ((size_t)slot * g.kv_heads + h) * g.vdim;
     for (int i = lane; i < g.vdim; i += 32) stf(dst + i, src[i] + (b ? b[i] : 0.f));
+  }
+}
+
+// Queries and keys normed over ALL heads of the token (kernels.h: q_norm / k_norm), optionally with values that are the keys as
+// projected: grid (T), 256 threads, one token per CTA.  The row [q | k] (bias added) is staged in shared memory once; its two sums
+// of squares are reduced over the CTA, then every pair is normed, turned and stored.
+constexpr int PREPF_THREADS = 256;
+template <class CT>
+__global__ void __launch_bounds__(PREPF_THREADS)
+poolattn_prep_full_kernel(const float* __restrict__ y, int ldy, int q_off, int k_off, int v_off, const float* __restrict__ bias,
+                          PoolAttnGeom g, const float* __restrict__ cos_sin, float eps, const int32_t* __restrict__ positions,
+                          const int32_t* __restrict__ slot_mapping, CT* __restrict__ q_out, CT* __restrict__ k_cache,
+                          CT* __restrict__ v_cache) {
+  extern __shared__ float prow[];   // [heads * dim | kv_heads * dim]
+  __shared__ float red[2][PREPF_THREADS / 32];
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, slot = slot_mapping[t];
+  const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim, nv = g.kv_heads * g.vdim;
+  const float* src = y + (size_t)t * ldy;
+  const bool shared_kv = v_off == k_off;
+  float sq = 0.f, sk = 0.f;
+  for (int i = tid; i < nq + nk; i += PREPF_THREADS) {
+    const bool is_q = i < nq;
+    const float v = src[is_q ? q_off + i : k_off + i - nq] + (bias != nullptr ? bias[i] : 0.f);
+    prow[i] = v;
+    if (is_q) sq = fmaf(v, v, sq);
+    else sk = fmaf(v, v, sk);
+  }
+  sq = warp_sum_f(sq);
+  sk = warp_sum_f(sk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = sq;
+    red[1][tid >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < PREPF_THREADS / 32; ++w) {   // the same order in every thread
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float rq = 1.f / sqrtf(sq / (float)nq + eps), rk = 1.f / sqrtf(sk / (float)nk + eps);
+  const float* cs = cos_sin != nullptr ? cos_sin + (size_t)positions[t] * g.rot_dims : nullptr;
+  const int half = g.rot_dims / 2;
+  for (int i = tid; i < nq + nk; i += PREPF_THREADS) {
+    const bool is_q = i < nq;
+    if (!is_q && slot < 0) break;
+    const float* w = is_q ? g.q_norm : g.k_norm - nq;
+    const float rs = is_q ? rq : rk;
+    const int d = (is_q ? i : i - nq) % g.dim;
+    float v = prow[i] * rs * w[i];
+    if (d < g.rot_dims) {
+      const bool first = g.rot_interleaved ? (d & 1) == 0 : d < half;
+      const int j = i + (g.rot_interleaved ? (first ? 1 : -1) : (first ? half : -half));
+      const int f = g.rot_interleaved ? d >> 1 : (first ? d : d - half);
+      const float p = prow[j] * rs * w[j];
+      v = first ? v * cs[f] - p * cs[half + f] : v * cs[f] + p * cs[half + f];
+    }
+    if (is_q) stf(q_out + (size_t)t * nq + i, v);
+    else stf(k_cache + (size_t)slot * nk + i - nq, v);
+  }
+  if (slot >= 0) {
+    for (int i = tid; i < nv; i += PREPF_THREADS)
+      stf(v_cache + (size_t)slot * nv + i, shared_kv ? prow[nq + i] : src[v_off + i] + (bias != nullptr ? bias[nq + nk + i] : 0.f));
   }
 }
 
@@ -206,6 +277,7 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
   float* alpha = Ps + PA_QT * KV_BLOCK;       // [PA_QT]
   float* lsum = alpha + PA_QT;                // [PA_QT]
   __shared__ long long rowoff[KV_BLOCK];      // cache row of every key of the chunk (-1: none)
+  __shared__ float fac[PA_QT];                // factors of the tile's outputs
   griddep_launch();
   griddep_wait();
   const LatentTile tl = tiles[blockIdx.x];
@@ -315,6 +387,7 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
 #pragma unroll
     for (int i = 0; i < 4; ++i) lsum[warp * 4 + i] = l_run[i];
   }
+  if (tid < nq) fac[tid] = out_factor(g, row0 + tid, h);
   __syncthreads();
 #pragma unroll
   for (int cc = 0; cc < PA_CC; ++cc) {
@@ -322,7 +395,7 @@ poolattn_kernel(const CT* __restrict__ q, const CT* __restrict__ k_cache, const 
     if (col < dv) {
 #pragma unroll
       for (int qi = 0; qi < PA_QT; ++qi)
-        if (qi < nq) stf(out + ((size_t)(row0 + qi) * g.heads + h) * dv + col, acc[qi][cc] / lsum[qi]);
+        if (qi < nq) stf(out + out_row(g, row0 + qi) + (size_t)h * dv + col, acc[qi][cc] * (fac[qi] / lsum[qi]));
     }
   }
 }
@@ -581,8 +654,9 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       if (tqr[r] >= nq) continue;
-      const float inv_l = 1.f / l_part[r];
-      bf* dst = out + ((size_t)(row0 + tqr[r]) * g.heads + h_base + (wr0 + gq + r * 8) % gs) * dv + t2;
+      const int h = h_base + (wr0 + gq + r * 8) % gs;
+      const float inv_l = out_factor(g, row0 + tqr[r], h) / l_part[r];
+      bf* dst = out + out_row(g, row0 + tqr[r]) + (size_t)h * dv + t2;
 #pragma unroll
       for (int j = 0; j < NT; ++j)
         if (EXACT || j * 8 < dv) *reinterpret_cast<__nv_bfloat162*>(dst + j * 8) = __floats2bfloat162_rn(acc[j][2 * r] * inv_l, acc[j][2 * r + 1] * inv_l);
@@ -618,7 +692,8 @@ poolattn_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
       o0 = fmaf(f, a2.x, o0);
       o1 = fmaf(f, a2.y, o1);
     }
-    *reinterpret_cast<__nv_bfloat162*>(out + ((size_t)(row0 + row / gs) * g.heads + h_base + row % gs) * dv + col) = __floats2bfloat162_rn(o0 / l, o1 / l);
+    const float f = out_factor(g, row0 + row / gs, h_base + row % gs) / l;
+    *reinterpret_cast<__nv_bfloat162*>(out + out_row(g, row0 + row / gs) + (size_t)(h_base + row % gs) * dv + col) = __floats2bfloat162_rn(o0 * f, o1 * f);
   }
 }
 
@@ -657,7 +732,7 @@ bool mma_eligible(const PoolAttnGeom& g, const void* q, const void* k, const voi
   }
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   return on && g.dim % 16 == 0 && g.dim <= 16 * MMA_KS && g.vdim % 8 == 0 && g.vdim <= 8 * MMA_MAX_NT && al16(q) && al16(k) && al16(v) &&
-         al16(pk) && al16(pv) && al16(out);
+         al16(pk) && al16(pv) && al16(out) && g.out_ld % 2 == 0;
 }
 
 template <class CT>
@@ -693,8 +768,26 @@ cudaError_t poolattn_prep_launch(const float* y, int ldy, int q_off, int k_off, 
                                  cudaStream_t stream) {
   if (T <= 0) return cudaSuccess;
   if (!geom_ok(g) || (g.rot_dims > 0 && cos_sin == nullptr)) return cudaErrorInvalidValue;
+  if (v_off == k_off && g.dim != g.vdim) return cudaErrorInvalidValue;
   const dim3 grid(T, (g.heads + 2 * g.kv_heads + PREP_WARPS - 1) / PREP_WARPS);
   using bf = __nv_bfloat16;
+  if (g.q_norm != nullptr || g.k_norm != nullptr) {
+    if (g.q_norm == nullptr || g.k_norm == nullptr || g.unit_norm) return cudaErrorInvalidValue;
+    const size_t smem = (size_t)(g.heads + g.kv_heads) * g.dim * sizeof(float);
+    if (smem > 160 * 1024) return cudaErrorInvalidValue;
+    static bool attr_set = false;
+    if (smem > 40 * 1024 && !attr_set) {
+      cudaError_t e = cudaFuncSetAttribute(poolattn_prep_full_kernel<bf>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(poolattn_prep_full_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024);
+      if (e != cudaSuccess) return e;
+      attr_set = true;
+    }
+    if (dtype == DT_BF16)
+      return launch_k(poolattn_prep_full_kernel<bf>, dim3(T), dim3(PREPF_THREADS), smem, stream, y, ldy, q_off, k_off, v_off, bias, g, cos_sin,
+                      eps, positions, slot_mapping, reinterpret_cast<bf*>(q_out), reinterpret_cast<bf*>(k_cache), reinterpret_cast<bf*>(v_cache));
+    return launch_k(poolattn_prep_full_kernel<float>, dim3(T), dim3(PREPF_THREADS), smem, stream, y, ldy, q_off, k_off, v_off, bias, g, cos_sin,
+                    eps, positions, slot_mapping, reinterpret_cast<float*>(q_out), reinterpret_cast<float*>(k_cache), reinterpret_cast<float*>(v_cache));
+  }
   const bool small = g.dim <= 128;   // four entries per lane
   if (dtype == DT_BF16)
     return launch_k(small ? poolattn_prep_kernel<bf, 4> : poolattn_prep_kernel<bf, PREP_MAX_DIM / 32>, grid, dim3(PREP_WARPS * 32), 0,

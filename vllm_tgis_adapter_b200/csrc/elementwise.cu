@@ -705,6 +705,7 @@ __global__ void __launch_bounds__(NORM_THREADS) resid_tail_kernel(ResidTail a, i
   const int t = blockIdx.x;
   const size_t base = (size_t)t * hidden;
   float ss = 0.f;
+  float ss2 = 0.f;
   float rs_a = 1.f, rs_b = 1.f;
   if (a.y_pair != nullptr) {   // two mixers side by side: each output is normed by itself first
     float sa = 0.f, sb = 0.f;
@@ -733,7 +734,7 @@ __global__ void __launch_bounds__(NORM_THREADS) resid_tail_kernel(ResidTail a, i
     } else {
       if (a.y_rows != nullptr)
         for (int k = 0; k < a.top; ++k) {
-          const float w = a.mix_w[(size_t)t * a.top + k];
+          const float w = a.mix_w != nullptr ? a.mix_w[(size_t)t * a.top + k] : a.mix_const;
           const FV<VEC> r = ld_fv<VEC>(a.y_rows + (size_t)a.inv[(size_t)t * a.top + k] * hidden + i);
 #pragma unroll
           for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(w, r.v[e], y.v[e]);
@@ -745,13 +746,27 @@ __global__ void __launch_bounds__(NORM_THREADS) resid_tail_kernel(ResidTail a, i
         for (int e = 0; e < VEC; ++e) y.v[e] = fmaf(w, r.v[e], y.v[e]);
       }
     }
+    if (a.w_post == nullptr) {   // the output is added as it is: one pass over the row
+      FV<VEC> r = ld_fv<VEC>(a.resid + base + i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) r.v[e] = fmaf(a.mult, y.v[e], r.v[e]);
+      if (a.extra != nullptr) {
+        const FV<VEC> ex = ld_fv<VEC>(a.extra + base + i);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) r.v[e] += ex.v[e];
+      }
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) ss2 += r.v[e] * r.v[e];
+      st_fv<VEC>(a.resid + base + i, r);
+      st_fv<VEC>(row_buf + i, r);
+      continue;
+    }
     st_fv<VEC>(row_buf + i, y);
 #pragma unroll
     for (int e = 0; e < VEC; ++e) ss += y.v[e] * y.v[e];
   }
-  const float rs = 1.f / sqrtf(block_sum<NORM_THREADS>(ss, red) / (float)hidden + a.eps);
-  float ss2 = 0.f;
-  for (int i = threadIdx.x * VEC; i < hidden; i += NORM_THREADS * VEC) {
+  const float rs = a.w_post != nullptr ? 1.f / sqrtf(block_sum<NORM_THREADS>(ss, red) / (float)hidden + a.eps) : 0.f;
+  for (int i = threadIdx.x * VEC; a.w_post != nullptr && i < hidden; i += NORM_THREADS * VEC) {
     const FV<VEC> y = ld_fv<VEC>(row_buf + i), x = ld_fv<VEC>(a.resid + base + i), w = ld_fv<VEC>(a.w_post + i);
     FV<VEC> r;
 #pragma unroll
@@ -776,8 +791,14 @@ __global__ void __launch_bounds__(NORM_THREADS) resid_tail_kernel(ResidTail a, i
     return;
   }
   const float rs2 = 1.f / sqrtf(block_sum<NORM_THREADS>(ss2, red) / (float)hidden + a.eps);
+  float dot = 0.f;
   for (int i = threadIdx.x * VEC; i < hidden; i += NORM_THREADS * VEC) {
     const FV<VEC> r = ld_fv<VEC>(row_buf + i), w = ld_fv<VEC>(a.w_pre + i);
+    if (a.dot_out != nullptr) {
+      const FV<VEC> d = ld_fv<VEC>(a.w_dot + i);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) dot = fmaf(r.v[e] * rs2 * (a.w_off + w.v[e]), d.v[e], dot);
+    }
     if (VEC == 4 && a.out_dtype == DT_BF16) {
       __nv_bfloat162 lo = __floats2bfloat162_rn(r.v[0] * rs2 * (a.w_off + w.v[0]), r.v[1 % VEC] * rs2 * (a.w_off + w.v[1 % VEC]));
       __nv_bfloat162 hi = __floats2bfloat162_rn(r.v[2 % VEC] * rs2 * (a.w_off + w.v[2 % VEC]), r.v[3 % VEC] * rs2 * (a.w_off + w.v[3 % VEC]));
@@ -795,14 +816,19 @@ __global__ void __launch_bounds__(NORM_THREADS) resid_tail_kernel(ResidTail a, i
       for (int e = 0; e < VEC; ++e) st_dt(a.out2, a.out_dtype, base + i + e, r.v[e] * rs2 * (a.w_off + w2.v[e]));
     }
   }
+  if (a.dot_out != nullptr) {
+    const float z = block_sum<NORM_THREADS>(dot, red);
+    if (threadIdx.x == 0) a.dot_out[t] = 1.f / (1.f + expf(-z));
+  }
 }
 cudaError_t resid_tail_launch(const ResidTail& a, int T, int hidden, cudaStream_t stream) {
   if (T <= 0) return cudaSuccess;
-  if (a.w_post == nullptr || a.resid == nullptr || (size_t)hidden * 4 > 48 * 1024) return cudaErrorInvalidValue;
+  if (a.resid == nullptr || (size_t)hidden * 4 > 48 * 1024) return cudaErrorInvalidValue;
+  if (a.dot_out != nullptr && (a.w_pre == nullptr || a.w_dot == nullptr)) return cudaErrorInvalidValue;
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   if (a.y_pair != nullptr && (a.y_main == nullptr || a.w_main == nullptr || a.w_pair == nullptr)) return cudaErrorInvalidValue;
   if (a.w_pre2 != nullptr && (a.w_pre == nullptr || a.out2 == nullptr)) return cudaErrorInvalidValue;
-  const bool vec = hidden % 4 == 0 && al16(a.extra) && al16(a.w_pre2) && al16(a.out2) && al16(a.y_main) && al16(a.y_rows) && al16(a.y_side) && al16(a.resid) && al16(a.w_post) &&
+  const bool vec = hidden % 4 == 0 && al16(a.extra) && al16(a.w_pre2) && al16(a.out2) && al16(a.y_main) && al16(a.y_rows) && al16(a.y_side) && al16(a.resid) && al16(a.w_post) && al16(a.w_dot) &&
                    al16(a.w_pre) && al16(a.out) && al16(a.y_pair) && al16(a.w_main) && al16(a.w_pair);
   if (vec) return launch_k(resid_tail_kernel<4>, dim3(T), dim3(NORM_THREADS), (size_t)hidden * sizeof(float), stream, a, hidden);
   return launch_k(resid_tail_kernel<1>, dim3(T), dim3(NORM_THREADS), (size_t)hidden * sizeof(float), stream, a, hidden);

@@ -295,9 +295,23 @@ struct tgis_engine {
     int router_cols = 0;                             // rows of w_router: the router's outputs and zero rows
     float *o_bias = nullptr, *decay = nullptr;       // [width] output bias of the attention; [mm_heads] decays
     int c_f = 0;                      // TGIS_MIXER_HGRN (w_in: q | f | v): column of the gate logits
+    // ---- layers of the plain pre-norm style (TGIS_ARCH_LUDELIX): norm1 / norm2.  Attention: pa, w_in, in_bias, sink, k_cache / v_cache,
+    // c_g (head gate); retention: c_mq .. c_mg, decay, st_S; GLA: c_q, c_k, c_v, c_mg (gate), c_a1, w_w2, w0, mm_norm, st_S; experts:
+    // w_gu_e, w_d_e, w_gu_s, w_d_s
+    int o_cols = 0, c_o2 = 0;         // columns of w_o: the attention's heads, then (from c_o2) the retention's; zero columns between
+    float *q_norm = nullptr, *k_norm = nullptr;      // norms over all query / key heads at once
+    const float* cos_sin2 = nullptr;  // the retention's rotation
+    float* w_gate_s = nullptr;        // [width] the shared expert's gate row, fp32
+    MoeTable tab{};                   // the experts of every token id, and this step's row segments
   };
   std::vector<PnxLayer> layer_runs;    // styles with loops (pair, dyt): one entry per layer RUN (a looped span repeats), weights shared
   bool dyt_style = false;             // TGIS_STYLE_PRE_DYT
+  bool rms_style = false;             // TGIS_STYLE_PRE_RMS
+  bool run_style() const { return pair_style || dyt_style || rms_style; }   // layer runs own caches and states
+  MoeTable* moe_tables = nullptr;     // device copy of every table-routed layer's `tab` ([n_moe_tables]) for the one launch that
+  int n_moe_tables = 0, moe_tables_max_E = 0;   // makes all row segments of a step
+  cudaEvent_t ev_tables = nullptr;    // ... which runs on the second stream beside the first mixer
+  bool tables_pending = false;        // this step's segments are not yet waited for
   DytNorm pnx_final_dyt{};
   bool pair_style = false;            // TGIS_STYLE_PARALLEL_PAIR
   void *pnx_side = nullptr, *pnx_hB = nullptr;       // side table [vocab, n_layers * side_dim]; norm2's rows (operand type)
@@ -493,6 +507,7 @@ struct tgis_engine {
     if (stream2) cudaStreamSynchronize(stream2);
     if (ev_fork) cudaEventDestroy(ev_fork);
     if (ev_join) cudaEventDestroy(ev_join);
+    if (ev_tables) cudaEventDestroy(ev_tables);
     if (stream2) cudaStreamDestroy(stream2);
     if (h_stage) cudaFreeHost(h_stage);
     if (h_samp_out) cudaFreeHost(h_samp_out);
@@ -539,7 +554,7 @@ struct tgis_engine {
     Vl = c.vocab / tp;
     opt = c.arch == TGIS_ARCH_OPT;
     pnx_on = c.arch == TGIS_ARCH_PONENEX || c.arch == TGIS_ARCH_FALERAX || c.arch == TGIS_ARCH_REVEPEL || c.arch == TGIS_ARCH_SIKAZEN ||
-             c.arch == TGIS_ARCH_BISUZEN;  // the layer-list architectures
+             c.arch == TGIS_ARCH_BISUZEN || c.arch == TGIS_ARCH_LUDELIX;  // the layer-list architectures
     if (pnx_on) logits_bf16 = false;  // fp32 logits straight from the accumulators
     model_head_dim = opt ? c.head_dim : HEAD_DIM;
     attn_scale = 1.0f / std::sqrt((float)model_head_dim);  // zero-padded head dims add nothing to q . k
@@ -1055,7 +1070,11 @@ struct tgis_engine {
     return fail("unknown layer weight " + full_name);
   }
 
-  int load_weight(const std::string& name, const void* ptr, int64_t rows, int64_t cols) {
+  int load_weight(const std::string& name, const void* ptr, int64_t rows, int64_t cols, int dtype) {
+    if (dtype != 0) {
+      if (pnx_on && dtype == 1) return pnx_load_table(name, static_cast<const int32_t*>(ptr), rows, cols);
+      return fail("only bf16 (dtype 0) weights are supported, int32 (dtype 1) for the tables of layer-list architectures");
+    }
     if (opt) return load_weight_opt(name, ptr, rows, cols);
     if (pnx_on) return pnx_load_weight(name, ptr, rows, cols);
     const tgis_config& c = cfg;
@@ -1227,18 +1246,31 @@ struct tgis_engine {
   // YaRN scaling (factor > 0): with dim(t) = dims ln(original / (2 pi t)) / (2 ln base) the dimension whose wave makes t turns
   // over `original` positions, lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)), dims - 1) and the ramp
   // r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1):  f_i <- f_i / factor * r_i + f_i (1 - r_i), cos and sin times 0.1 ln(factor) + 1.
-  // linear > 0: every frequency is divided by it (linear position scaling).
+  // linear > 0: every frequency is divided by it (linear position scaling).  band (factor > 0): scaling by wavelength
+  // (tgis_layer_spec.band_*).
+  struct Band { float factor, original, low, high; };
   const float* pnx_rope_table(float base, int dims, float factor = 0.f, float original = 0.f, float fast = 0.f, float slow = 0.f,
-                              float linear = 1.f) {
-    const std::vector<float> key = {base, (float)dims, factor, original, fast, slow, linear};
+                              float linear = 1.f, Band band = Band()) {
+    const std::vector<float> key = {base, (float)dims, factor, original, fast, slow, linear, band.factor, band.original, band.low, band.high};
     for (auto& kv : pnx_rope_tables)
       if (kv.first == key) return kv.second;
     const int half = dims / 2;
     std::vector<double> freq(std::max(half, 1));
     double mag = 1.0;
     for (int i = 0; i < half; ++i) freq[i] = std::pow((double)base, -2.0 * i / dims) / (linear > 0.f ? (double)linear : 1.0);
+    const double pi = 3.14159265358979323846;
+    if (band.factor > 0.f)
+      for (int i = 0; i < half; ++i) {
+        const double wave = 2.0 * pi / freq[i], f = freq[i], orig = band.original;
+        if (wave < orig / band.high) continue;
+        if (wave > orig / band.low) {
+          freq[i] = f / band.factor;
+        } else {
+          const double t = (orig / wave - band.low) / ((double)band.high - band.low);
+          freq[i] = (1.0 - t) * f / band.factor + t * f;
+        }
+      }
     if (factor > 0.f) {
-      const double pi = 3.14159265358979323846;
       auto turn_dim = [&](double turns) { return dims * std::log((double)original / (2.0 * pi * turns)) / (2.0 * std::log((double)base)); };
       const double lo = std::max(std::floor(turn_dim(fast)), 0.0), hi = std::min(std::ceil(turn_dim(slow)), (double)dims - 1.0);
       for (int i = 0; i < half; ++i) {
@@ -1263,7 +1295,7 @@ struct tgis_engine {
   DytNorm alloc_dyt(size_t W) { return DytNorm{pnx_alloc<float>(W), pnx_alloc<float>(W), pnx_alloc<float>(1)}; }
   // mixers whose attention keeps paged keys and values per layer run
   static bool run_has_kv(const tgis_layer_spec& s) {
-    return s.mixer == TGIS_MIXER_POOLED_ATTENTION || s.mixer == TGIS_MIXER_WINDOW_LIGHTNING;
+    return s.mixer == TGIS_MIXER_POOLED_ATTENTION || s.mixer == TGIS_MIXER_WINDOW_LIGHTNING || s.mixer == TGIS_MIXER_CHUNK_RETENTION;
   }
 
   void init_pnx() {
@@ -1278,6 +1310,7 @@ struct tgis_engine {
     gated_style = (pnx_spec.style & TGIS_STYLE_PARALLEL_GATED) != 0;
     pair_style = (pnx_spec.style & TGIS_STYLE_PARALLEL_PAIR) != 0;
     dyt_style = (pnx_spec.style & TGIS_STYLE_PRE_DYT) != 0;
+    rms_style = (pnx_spec.style & TGIS_STYLE_PRE_RMS) != 0;
     pnx_embed = pnx_alloc_dt(V * W);
     pnx_head = tied_head ? pnx_embed : pnx_alloc_dt(V * W);
     pnx_final_norm = pnx_alloc<float>(W);
@@ -1370,6 +1403,99 @@ struct tgis_engine {
           m_heads = std::max<size_t>(m_heads, s.heads);
           pnx_tile_tokens = std::min(pnx_tile_tokens, latent_tile_tokens(s.heads));
         }
+        continue;
+      }
+      if (rms_style) {   // weights only, as above
+        l.weights_of = (int)i;
+        l.norm1 = pnx_alloc<float>(W);
+        pnx_expected_tensors += 1;
+        if (s.mlp != TGIS_MLP_NONE) {
+          l.norm2 = pnx_alloc<float>(W);
+          pnx_expected_tensors += 1;
+        }
+        if (s.mlp == TGIS_MLP_DENSE_RELU2) {
+          l.w_gu = pnx_alloc_dt((size_t)s.ff * W);
+          l.w_d = pnx_alloc_dt(W * s.ff);
+          pnx_expected_tensors += 2;  // mlp.up, mlp.down
+          m_ffs = std::max<size_t>(m_ffs, s.ff);
+        } else if (s.mlp == TGIS_MLP_MOE_TABLE) {
+          const size_t E = s.experts, ff = s.expert_ff, ffs = s.shared_ff;
+          l.w_gu_e = pnx_alloc_dt(E * 2 * ff * W);
+          l.w_d_e = pnx_alloc_dt(E * W * ff);
+          l.tab = MoeTable{pnx_alloc<int32_t>(V * s.top, true), pnx_alloc<int32_t>(E + 1), pnx_alloc<int32_t>(T * s.top),
+                           pnx_alloc<int32_t>(T * s.top), s.experts, s.top};
+          pnx_expected_tensors += 1 + 3 * E;   // table, e<j>.{gate, up, down}
+          if (ffs > 0) {
+            l.w_gu_s = pnx_alloc_dt(2 * ffs * W);
+            l.w_d_s = pnx_alloc_dt(W * ffs);
+            l.w_gate_s = pnx_alloc<float>(W);
+            pnx_expected_tensors += 4;  // shared.{gate, up, down, sg}
+          }
+          m_top = std::max<size_t>(m_top, s.top); m_ff = std::max(m_ff, ff); m_ffs = std::max(m_ffs, ffs);
+        }
+        const int H = s.heads, G = s.kv_heads;
+        int col = 0;
+        auto cols = [&](int n) { const int r = col; col += n; return r; };
+        auto up8 = [](int n) { return (n + 7) / 8 * 8; };
+        if (s.mixer == TGIS_MIXER_GLA) {
+          const size_t hd = (size_t)H * s.dim, hv = (size_t)H * s.vdim;
+          l.c_q = cols((int)hd); l.c_k = cols((int)hd); l.c_v = cols((int)hv); l.c_mg = cols((int)hv); l.c_a1 = cols(s.decay_rank);
+          l.w_w2 = pnx_alloc_dt(hd * s.decay_rank);
+          l.w0 = pnx_alloc<float>(hd);
+          l.mm_norm = pnx_alloc<float>(hv);   // the per-head weight, repeated for every head
+          l.o_cols = up8((int)hv);
+          pnx_expected_tensors += 9;  // q, k, v, g, o, norm, a1, a2, a2.b
+          m_f1 = std::max(m_f1, hv); m_f2 = std::max(m_f2, hd);
+          m_mix = std::max(m_mix, 2 * hd + hv);
+        } else {
+          const bool par = s.mixer == TGIS_MIXER_CHUNK_RETENTION, shared_kv = (s.flags & TGIS_LAYER_SHARED_KV) != 0;
+          l.c_q = cols(H * s.dim); l.c_k = cols(G * s.dim);
+          l.c_v = shared_kv ? l.c_k : cols(G * s.vdim);
+          pnx_expected_tensors += shared_kv ? 3 : 4;  // q, k, o (+ v)
+          l.c_o2 = l.o_cols = up8(H * s.vdim);
+          if (par) {
+            const size_t md = (size_t)s.mm_heads * s.mm_dim, mv = (size_t)s.mm_heads * s.mm_vdim;
+            l.c_mq = cols((int)md); l.c_mk = cols((int)md); l.c_mv = cols((int)mv); l.c_mg = cols((int)mv);
+            l.o_cols = l.c_o2 + up8((int)mv);
+            l.decay = pnx_alloc<float>(s.mm_heads);
+            CK(cudaMemcpy(l.decay, pnx_decays[i].data(), sizeof(float) * s.mm_heads, cudaMemcpyHostToDevice));
+            l.cos_sin2 = s.mm_rot_dims > 0 ? pnx_rope_table(s.mm_rot_base, s.mm_rot_dims) : nullptr;
+            pnx_expected_tensors += 5;  // right.{q, k, v, g, o}
+            m_f1 = std::max(m_f1, mv);
+            m_mix = std::max(m_mix, 2 * md + mv);
+          }
+          if ((s.flags & TGIS_LAYER_HEAD_GATE) != 0) {
+            l.c_g = cols(H);
+            pnx_expected_tensors += 1;
+          }
+          if ((s.flags & TGIS_LAYER_SINK) != 0) {
+            l.sink = pnx_alloc<float>(H);
+            pnx_expected_tensors += 1;
+          }
+          if ((s.flags & TGIS_LAYER_FULL_QK_NORM) != 0) {
+            l.q_norm = pnx_alloc<float>((size_t)H * s.dim);
+            l.k_norm = pnx_alloc<float>((size_t)G * s.dim);
+            pnx_expected_tensors += 2;
+          }
+          if ((s.flags & TGIS_LAYER_QKV_BIAS) != 0) {
+            l.in_bias = pnx_alloc<float>((size_t)H * s.dim + (size_t)G * (s.dim + s.vdim), true);
+            pnx_expected_tensors += shared_kv ? 2 : 3;  // q.b, k.b (+ v.b)
+          }
+          l.pa = PoolAttnGeom{H, G, s.dim, s.vdim, s.window, s.window > 0 ? s.pool : 0, s.rot_dims, s.scale,
+                              (s.flags & TGIS_LAYER_UNIT_QK) != 0 ? 1 : 0, s.window > 0 ? s.keep_first : 0, s.chunk,
+                              (s.flags & TGIS_LAYER_ROT_INTERLEAVED) != 0 ? 1 : 0, l.sink};
+          l.pa.out_ld = l.o_cols;
+          l.pa.q_norm = l.q_norm; l.pa.k_norm = l.k_norm;
+          l.pa.out_mul = par ? s.left_scale : 1.f;
+          l.cos_sin = s.rot_dims > 0 ? pnx_rope_table(s.rot_base, s.rot_dims, s.yarn_factor, s.yarn_original, s.yarn_fast, s.yarn_slow, 1.f,
+                                                      Band{s.band_factor, s.band_original, s.band_low, s.band_high}) : nullptr;
+          m_q = std::max<size_t>(m_q, (size_t)H * s.dim);
+        }
+        l.in_cols = up8(col);
+        l.w_in = pnx_alloc_dt((size_t)l.in_cols * W, true);
+        l.w_o = pnx_alloc_dt(W * l.o_cols, true);
+        m_ov = std::max<size_t>(m_ov, l.o_cols);
+        m_down = std::max<size_t>(m_down, l.in_cols);
         continue;
       }
       if (dyt_style) {   // weights only, as above
@@ -1627,7 +1753,7 @@ struct tgis_engine {
       cache_row_bytes += row * dt_size(pnx_dt);
       pnx_tile_tokens = std::min(pnx_tile_tokens, latent_tile_tokens(s.heads));
     }
-    if (pair_style || dyt_style) {
+    if (run_style()) {
       // the layer runs: layers [loop_start, loop_stop) repeat loop_times passes in a row; every run owns cache rows and state
       const int L = (int)pnx_layers.size(), a = pnx_spec.loop_start, b = pnx_spec.loop_stop;
       const int passes = (pnx_spec.loop_times > 1 && b > a) ? pnx_spec.loop_times : 1;
@@ -1650,7 +1776,7 @@ struct tgis_engine {
           cache_row_bytes += (size_t)r.g.row() * dt_size(pnx_dt);
         else
           r.st_S = pnx_alloc<float>((size_t)S_max * s.heads * s.dim * s.vdim, true);
-        if (s.mixer == TGIS_MIXER_WINDOW_LIGHTNING) r.st_S = pnx_alloc<float>((size_t)S_max * s.mm_heads * s.mm_dim * s.mm_vdim, true);
+        if (s.mixer == TGIS_MIXER_WINDOW_LIGHTNING || s.mixer == TGIS_MIXER_CHUNK_RETENTION) r.st_S = pnx_alloc<float>((size_t)S_max * s.mm_heads * s.mm_dim * s.mm_vdim, true);
       }
       if (pnx_spec.side_dim > 0) {
         pnx_side = pnx_alloc_dt(V * pnx_layers.size() * pnx_spec.side_dim);
@@ -1665,6 +1791,18 @@ struct tgis_engine {
         gemm_ws2.alloc(gemm_workspace_bytes(num_sms) / sizeof(float));
         gemm_counters2.alloc(1 << 16);
         gemm_counters2.zero();
+      }
+      std::vector<MoeTable> tabs;
+      for (const PnxLayer& l : pnx_layers)
+        if (l.sp.mlp == TGIS_MLP_MOE_TABLE) {
+          tabs.push_back(l.tab);
+          moe_tables_max_E = std::max(moe_tables_max_E, l.sp.experts);
+        }
+      if (!tabs.empty()) {
+        n_moe_tables = (int)tabs.size();
+        moe_tables = pnx_alloc<MoeTable>(tabs.size());
+        CK(cudaMemcpy(moe_tables, tabs.data(), tabs.size() * sizeof(MoeTable), cudaMemcpyHostToDevice));
+        CK(cudaEventCreateWithFlags(&ev_tables, cudaEventDisableTiming));
       }
     }
     // activations
@@ -1718,7 +1856,7 @@ struct tgis_engine {
     if (nb < 1) throw CudaError("cache too small for one block");
     num_blocks = (int)nb;
     for (PnxLayer& l : pnx_layers) {  // finite everywhere
-      if (pair_style || dyt_style) break;   // (the layer runs own the caches)
+      if (run_style()) break;   // (the layer runs own the caches)
       if (l.sp.mixer == TGIS_MIXER_LATENT_ATTENTION) l.cache = pnx_alloc_dt(nb * KV_BLOCK * l.g.row(), true);
       if (l.sp.mixer == TGIS_MIXER_PARALLEL) {
         l.k_cache = pnx_alloc_dt(nb * KV_BLOCK * l.ca.kv_heads * l.ca.dim, true);
@@ -1747,6 +1885,25 @@ struct tgis_engine {
     }
     free_blocks.resize(num_blocks);
     for (int i = 0; i < num_blocks; ++i) free_blocks[i] = num_blocks - 1 - i;
+  }
+
+  // int32 tables: "l<i>.mlp.table" [vocab, top] -- the experts of every token id
+  int pnx_load_table(const std::string& name, const int32_t* ptr, int64_t rows, int64_t cols) {
+    const size_t dot = name.find('.');
+    const int li = (name.size() > 2 && name[0] == 'l' && dot != std::string::npos) ? atoi(name.substr(1, dot - 1).c_str()) : -1;
+    if (li < 0 || li >= (int)pnx_layers.size() || name.substr(dot + 1) != "mlp.table" || pnx_layers[li].sp.mlp != TGIS_MLP_MOE_TABLE)
+      return fail("unknown table " + name);
+    const PnxLayer& l = pnx_layers[li];
+    if (rows * cols != (int64_t)cfg.vocab * l.sp.top)
+      return fail("shape mismatch for " + name + ": got " + std::to_string(rows) + "x" + std::to_string(cols));
+    std::vector<int32_t> h((size_t)(rows * cols));
+    if (cudaMemcpy(h.data(), ptr, h.size() * sizeof(int32_t), cudaMemcpyDefault) != cudaSuccess) return fail("cudaMemcpy(table) failed");
+    for (int32_t e : h)   // the kernels index expert segments with these
+      if (e < 0 || e >= l.sp.experts) return fail("expert index out of range in " + name);
+    if (cudaMemcpy(const_cast<int32_t*>(l.tab.table), h.data(), h.size() * sizeof(int32_t), cudaMemcpyHostToDevice) != cudaSuccess)
+      return fail("cudaMemcpy(table) failed");
+    pnx_loaded.insert(name);
+    return 0;
   }
 
   int pnx_load_weight(const std::string& name, const void* ptr, int64_t rows, int64_t cols) {
@@ -1871,6 +2028,77 @@ struct tgis_engine {
         if (sub == "mix.uv") return mat(l.w_uv, (int64_t)s.heads * s.vdim, s.kv_rank);
         if (sub == "mix.sink" && l.sink != nullptr) return vec(l.sink, s.heads);
         if (sub == "mix.o") return mat(l.w_o, W, (int64_t)s.heads * s.vdim);
+      }
+      return fail("unknown layer weight " + name);
+    }
+    if (rms_style) {
+      auto in_rows = [&](int col, int64_t r) { return mat(at(l.w_in, (size_t)col * W), r, W); };
+      if (sub == "norm1") return vec(l.norm1, W);
+      if (sub == "norm2")   // (of a layer without a feed-forward: nothing reads it)
+        return s.mlp != TGIS_MLP_NONE ? vec(l.norm2, W) : n == W ? 0 : bad_shape();
+      if (s.mlp == TGIS_MLP_DENSE_RELU2) {
+        if (sub == "mlp.up") return mat(l.w_gu, s.ff, W);
+        if (sub == "mlp.down") return mat(l.w_d, W, s.ff);
+      } else if (s.mlp == TGIS_MLP_MOE_TABLE) {
+        const int64_t ff = s.expert_ff, ffs = s.shared_ff;
+        // gate / up rows interleave (row 2j = gate_j, row 2j + 1 = up_j): one product, the gated activation in its epilogue
+        if (ffs > 0) {
+          if (sub == "mlp.shared.sg") return vec(l.w_gate_s, W);
+          if (sub == "mlp.shared.gate") return place(l.w_gu_s, pnx_dt, ffs, W, 2 * W, 1);
+          if (sub == "mlp.shared.up") return place(at(l.w_gu_s, (size_t)W), pnx_dt, ffs, W, 2 * W, 1);
+          if (sub == "mlp.shared.down") return mat(l.w_d_s, W, ffs);
+        }
+        if (sub.rfind("mlp.e", 0) == 0) {
+          const size_t d2 = sub.find('.', 5);
+          if (d2 == std::string::npos) return fail("unknown layer weight " + name);
+          const int ei = atoi(sub.substr(5, d2 - 5).c_str());
+          if (ei < 0 || ei >= s.experts) return fail("expert index out of range in " + name);
+          const std::string which = sub.substr(d2 + 1);
+          if (which == "gate") return place(at(l.w_gu_e, (size_t)ei * 2 * ff * W), pnx_dt, ff, W, 2 * W, 1);
+          if (which == "up") return place(at(l.w_gu_e, (size_t)ei * 2 * ff * W + W), pnx_dt, ff, W, 2 * W, 1);
+          if (which == "down") return mat(at(l.w_d_e, (size_t)ei * W * ff), W, ff);
+        }
+      }
+      const int64_t H = s.heads, G = s.kv_heads, hv = H * s.vdim;
+      // output projections of the two mixers of a layer lie side by side in one matrix [width, o_cols]
+      auto out_proj = [&](int col, int64_t k) { return place(at(l.w_o, (size_t)col), pnx_dt, W, k, l.o_cols, 1); };
+      if (s.mixer == TGIS_MIXER_GLA) {
+        const int64_t hd = H * s.dim;
+        if (sub == "mix.q") return in_rows(l.c_q, hd);
+        if (sub == "mix.k") return in_rows(l.c_k, hd);
+        if (sub == "mix.v") return in_rows(l.c_v, hv);
+        if (sub == "mix.g") return in_rows(l.c_mg, hv);
+        if (sub == "mix.a1") return in_rows(l.c_a1, s.decay_rank);
+        if (sub == "mix.a2") return mat(l.w_w2, hd, s.decay_rank);
+        if (sub == "mix.a2.b") return vec(l.w0, hd);
+        if (sub == "mix.norm") return per_head(l.mm_norm, s.heads, s.vdim);
+        if (sub == "mix.o") return out_proj(0, hv);
+        return fail("unknown layer weight " + name);
+      }
+      const bool par = s.mixer == TGIS_MIXER_CHUNK_RETENTION, shared_kv = (s.flags & TGIS_LAYER_SHARED_KV) != 0;
+      const std::string left = par ? "mix.left." : "mix.", right = "mix.right.";
+      if (sub == left + "q") return in_rows(l.c_q, H * s.dim);
+      if (sub == left + "k") return in_rows(l.c_k, G * s.dim);
+      if (sub == left + "v" && !shared_kv) return in_rows(l.c_v, G * s.vdim);
+      if (sub == left + "g" && (s.flags & TGIS_LAYER_HEAD_GATE) != 0) return in_rows(l.c_g, H);
+      if (sub == left + "o") return out_proj(0, hv);
+      if (sub == left + "sink" && l.sink != nullptr) return vec(l.sink, H);
+      if (l.q_norm != nullptr) {
+        if (sub == left + "q.norm") return vec(l.q_norm, H * s.dim);
+        if (sub == left + "k.norm") return vec(l.k_norm, G * s.dim);
+      }
+      if (l.in_bias != nullptr) {   // q | k (| v)
+        if (sub == left + "q.b") return vec(l.in_bias, H * s.dim);
+        if (sub == left + "k.b") return vec(l.in_bias + H * s.dim, G * s.dim);
+        if (sub == left + "v.b" && !shared_kv) return vec(l.in_bias + (H + G) * s.dim, G * s.vdim);
+      }
+      if (par) {
+        const int64_t md = (int64_t)s.mm_heads * s.mm_dim, mv = (int64_t)s.mm_heads * s.mm_vdim;
+        if (sub == right + "q") return in_rows(l.c_mq, md);
+        if (sub == right + "k") return in_rows(l.c_mk, md);
+        if (sub == right + "v") return in_rows(l.c_mv, mv);
+        if (sub == right + "g") return in_rows(l.c_mg, mv);
+        if (sub == right + "o") return out_proj(l.c_o2, mv);
       }
       return fail("unknown layer weight " + name);
     }
@@ -2605,6 +2833,154 @@ struct tgis_engine {
     pnx_dump_resid(T);
   }
 
+  // One layer run of the plain pre-norm style (TGIS_STYLE_PRE_RMS).  On entry pnx_hA holds rms(x) * norm1 (operand type):
+  //   x += mixer(hA);   x += ff(rms(x) * norm2)
+  // and every tail leaves the next sublayer's input (after the last run: the final norm's output) behind.
+  void rms_layer(int ri, int T, int S) {
+    PnxLayer& l = layer_runs[ri];
+    const tgis_layer_spec& s = l.sp;
+    const int W = cfg.hidden, A = pnx_dt;
+    const float eps = pnx_spec.norm_eps;
+    const int32_t* d_pos = ds<int32_t>(off_pos);
+    const int32_t* d_slot = ds<int32_t>(off_slotmap);
+    const int32_t* d_tokslot = ds<int32_t>(off_tokslot);
+    const AttnSeq* d_seqs = ds<AttnSeq>(off_seqs);
+    const bool last = ri + 1 == (int)layer_runs.size(), has_ff = s.mlp != TGIS_MLP_NONE;
+    const float* next = last ? pnx_final_norm : layer_runs[ri + 1].norm1;
+    const int ld = l.in_cols, hv = s.heads * s.vdim;
+    auto fork = [&]() {
+      CK(cudaEventRecord(ev_fork, stream));
+      CK(cudaStreamWaitEvent(stream2, ev_fork, 0));
+      on_side_stream = true;
+    };
+    auto side_done = [&]() {
+      on_side_stream = false;
+      CK(cudaEventRecord(ev_join, stream2));
+    };
+    // ---- mixer: every projection that reads hA in one product, every head's output into pnx_oA, one output product
+    pnx_gemm(pnx_hA, A, W, l.w_in, pnx_y1, DT_F32, ld, T, ld, W);
+    if (s.mixer == TGIS_MIXER_GLA) {
+      const int hd = s.heads * s.dim;
+      pnx_gemm(pnx_y1 + l.c_a1, DT_F32, ld, l.w_w2, flx_f2, DT_F32, hd, T, hd, s.decay_rank);
+      OuterScan os{};
+      os.mode = OUTER_SCAN_GLA;
+      os.q = pnx_y1 + l.c_q; os.k = pnx_y1 + l.c_k; os.v = pnx_y1 + l.c_v; os.ldq = os.ldk = os.ldv = ld;
+      os.q_scale = 1.f / sqrtf((float)s.dim);
+      os.decay_raw = flx_f2; os.ldd = hd; os.w0 = l.w0; os.inv_tau = 1.f / s.tau;
+      os.S = l.st_S;
+      os.out = flx_f1; os.ldo = hv;
+      os.heads = s.heads; os.dim = s.dim; os.vdim = s.vdim;
+      CK(outer_scan_launch(os, d_seqs, S, d_tokslot, stream));
+      CK(head_norm_gate_launch(flx_f1, hv, s.heads, s.vdim, l.mm_norm, pnx_y1 + l.c_mg, ld, /*silu*/ 1, eps, pnx_oA, A, T, stream, 0, 1.f,
+                               l.o_cols));
+      n_launches += 2;
+    } else {
+      const bool par = s.mixer == TGIS_MIXER_CHUNK_RETENTION;
+      auto retention = [&](cudaStream_t st) {   // -> columns [c_o2, ..) of pnx_oA
+        const int mH = s.mm_heads, md = mH * s.mm_dim, mv = mH * s.mm_vdim;
+        // bf16 portions: chunk by chunk on the tensor cores; single tokens (the step's first sequences) and fp32: token by token
+        const int lead = step_n_lead1, qkv = 2 * md + mv;
+        const bool chunked = A == DT_BF16 && lead < S && lightning_chunk_eligible(s.mm_dim, s.mm_vdim);
+        RotaryRows rr{pnx_y1, ld, l.c_mq, l.c_mk, l.c_mv, mH, s.mm_dim, s.mm_vdim, s.mm_rot_dims, 1.f, 1.f / sqrtf((float)s.mm_dim),
+                      l.cos_sin2, d_pos, chunked ? flx_mix : nullptr, qkv, lead};
+        CK(rotary_rows_launch(rr, T, st));
+        OuterScan os{};
+        os.mode = OUTER_SCAN_RETENTION;
+        os.q = pnx_y1 + l.c_mq; os.k = pnx_y1 + l.c_mk; os.v = pnx_y1 + l.c_mv; os.ldq = os.ldk = os.ldv = ld;
+        os.q_scale = 1.f;
+        os.decay = l.decay;
+        os.S = l.st_S;
+        os.out = flx_f1; os.ldo = mv;
+        os.heads = mH; os.dim = s.mm_dim; os.vdim = s.mm_vdim;
+        if (chunked) {
+          const LightningChunk lc{flx_mix, qkv, 0, md, 2 * md, l.decay, l.st_S, flx_f1, mv, mH, s.mm_dim, s.mm_vdim};
+          CK(lightning_chunk_launch(lc, d_seqs + lead, S - lead, d_tokslot, st));
+          if (lead > 0) CK(outer_scan_launch(os, d_seqs, lead, d_tokslot, st));
+          n_launches += lead > 0 ? 1 : 0;
+        } else {
+          CK(outer_scan_launch(os, d_seqs, S, d_tokslot, st));
+        }
+        CK(head_norm_gate_launch(flx_f1, mv, mH, s.mm_vdim, nullptr, pnx_y1 + l.c_mg, ld, /*silu*/ 1, eps,
+                                 reinterpret_cast<uint8_t*>(pnx_oA) + (size_t)l.c_o2 * dt_size(A), A, T, st, 0, s.right_scale, l.o_cols));
+        n_launches += 3;
+      };
+      const bool forked = par && stream2 != nullptr;   // the two mixers side by side
+      if (forked) {
+        fork();
+        retention(stream2);
+        side_done();
+      }
+      PoolAttnGeom pa = l.pa;
+      if ((s.flags & TGIS_LAYER_HEAD_GATE) != 0) {
+        pa.head_gate = pnx_y1 + l.c_g;
+        pa.gate_ld = ld;
+      }
+      CK(poolattn_prep_launch(pnx_y1, ld, l.c_q, l.c_k, l.c_v, l.in_bias, pa, l.cos_sin, eps, d_pos, d_slot, pnx_q, l.k_cache, l.v_cache, A, T,
+                              stream));
+      CK(poolattn_launch(pnx_q, l.k_cache, l.v_cache, nullptr, nullptr, A, d_seqs, ds<LatentTile>(off_ltiles16), step_n_ltiles16, T,
+                         ds<int32_t>(off_bt), bt_stride, pnx_oA, A, pa, stream));
+      n_launches += 2;
+      if (forked) CK(cudaStreamWaitEvent(stream, ev_join, 0));
+      else if (par) retention(stream);
+    }
+    pnx_gemm(pnx_oA, A, l.o_cols, l.w_o, pnx_o, DT_F32, W, T, W, l.o_cols);
+    ResidTail rt{};
+    rt.resid = pnx_resid; rt.out = pnx_hA; rt.out_dtype = A; rt.mult = 1.f; rt.w_off = 0.f; rt.eps = eps;
+    ResidTail ft = rt;   // the feed-forward's
+    rt.y_main = pnx_o; rt.w_pre = has_ff ? l.norm2 : next;
+    const bool shared = s.mlp == TGIS_MLP_MOE_TABLE && s.shared_ff > 0;
+    if (shared) { rt.w_dot = l.w_gate_s; rt.dot_out = pnx_sgate; }   // the shared expert's gate reads the same normed row
+    CK(resid_tail_launch(rt, T, W, stream));
+    ++n_launches;
+    // ---- feed-forward
+    if (has_ff) {
+      ft.w_pre = next;
+      if (s.mlp == TGIS_MLP_DENSE_RELU2) {
+        pnx_gemm(pnx_hA, A, W, l.w_gu, pnx_actS, A, s.ff, T, s.ff, W, GEMM_ANY_RELU2);
+        pnx_gemm(pnx_actS, A, s.ff, l.w_d, pnx_o, DT_F32, W, T, W, s.ff);
+        ft.y_main = pnx_o;
+      } else {  // TGIS_MLP_MOE_TABLE
+        const int top = s.top, ff = s.expert_ff, ffs = s.shared_ff;
+        auto shared_expert = [&]() {
+          pnx_gemm(pnx_hA, A, W, l.w_gu_s, pnx_actS, A, ffs, T, 2 * ffs, W, GEMM_ANY_SWIGLU);
+          pnx_gemm(pnx_actS, A, ffs, l.w_d_s, pnx_yS, DT_F32, W, T, W, ffs);
+        };
+        const bool forked = shared && stream2 != nullptr;   // the shared expert beside the chosen ones
+        if (forked) {
+          fork();
+          shared_expert();
+          side_done();
+        } else if (shared) {
+          shared_expert();
+        }
+        if (tables_pending) {
+          CK(cudaStreamWaitEvent(stream, ev_tables, 0));
+          tables_pending = false;
+        }
+        GemmAny a{};
+        a.X = pnx_hA; a.W = l.w_gu_e; a.Y = pnx_actE;
+        a.x_dtype = A; a.w_dtype = A; a.y_dtype = A;
+        a.T = T * top; a.N = 2 * ff; a.K = W; a.ldx = W; a.ldw = W; a.ldy = ff;
+        a.batch = 1; a.seg_off = l.tab.seg_off; a.n_groups = s.experts; a.w_gs = (long long)2 * ff * W;
+        a.gather = l.tab.order; a.gather_div = top; a.mode = GEMM_ANY_SWIGLU;
+        CK(gemm_any_launch(a, stream));
+        GemmAny b{};
+        b.X = pnx_actE; b.W = l.w_d_e; b.Y = pnx_yE;
+        b.x_dtype = A; b.w_dtype = A; b.y_dtype = DT_F32;
+        b.T = T * top; b.N = W; b.K = ff; b.ldx = ff; b.ldw = ff; b.ldy = W;
+        b.batch = 1; b.seg_off = l.tab.seg_off; b.n_groups = s.experts; b.w_gs = (long long)W * ff;
+        CK(gemm_any_launch(b, stream));
+        n_launches += 2;
+        if (forked) CK(cudaStreamWaitEvent(stream, ev_join, 0));
+        ft.y_rows = pnx_yE; ft.inv = l.tab.inv; ft.top = top; ft.mix_const = 1.f / (float)top;
+        ft.y_side = shared ? pnx_yS : nullptr; ft.side_gate = shared ? pnx_sgate : nullptr;
+      }
+      CK(resid_tail_launch(ft, T, W, stream));
+      ++n_launches;
+    }
+    pnx_dump_resid(T);
+  }
+
   // embeddings + layer stack + final norm -> pnx_hA [T, hidden] (operand type), fp32 residual stream in pnx_resid
   void pnx_forward(int T, int S) {
     const int W = cfg.hidden, A = pnx_dt;
@@ -2623,6 +2999,23 @@ struct tgis_engine {
       if (f.sp.mlp == TGIS_MLP_DENSE_SILU) CK(rmsnorm_f32_launch(pnx_resid, W, f.norm2, 0.f, pnx_hB, A, W, T, W, eps, stream));
       n_launches += 3;
       for (int ri = 0; ri < (int)layer_runs.size(); ++ri) pair_layer(ri, T, S);
+      return;
+    }
+    if (rms_style) {
+      if (n_moe_tables > 0) {   // the experts of every layer follow from the token ids alone
+        const bool forked = stream2 != nullptr;
+        if (forked) {
+          CK(cudaEventRecord(ev_fork, stream));
+          CK(cudaStreamWaitEvent(stream2, ev_fork, 0));
+        }
+        CK(moe_table_align_launch(moe_tables, n_moe_tables, moe_tables_max_E, d_tok, cfg.vocab, T, forked ? stream2 : stream));
+        if (forked) CK(cudaEventRecord(ev_tables, stream2));
+        tables_pending = forked;
+        ++n_launches;
+      }
+      CK(rmsnorm_f32_launch(pnx_resid, W, layer_runs[0].norm1, 0.f, pnx_hA, A, W, T, W, eps, stream));
+      n_launches += 2;
+      for (int ri = 0; ri < (int)layer_runs.size(); ++ri) rms_layer(ri, T, S);
       return;
     }
     if (dyt_style) {
@@ -3198,7 +3591,7 @@ struct tgis_engine {
         LatentTile* lt = hs<LatentTile>(off_ltiles);
         for (int q0 = 0; q0 < q_len; q0 += pnx_tile_tokens)
           lt[step_n_ltiles++] = LatentTile{s, q0, std::min(pnx_tile_tokens, q_len - q0), 0};
-        if (pair_style || dyt_style) {
+        if (run_style()) {
           LatentTile* lt16 = hs<LatentTile>(off_ltiles16);
           for (int q0 = 0; q0 < q_len; q0 += POOLATTN_TILE)
             lt16[step_n_ltiles16++] = LatentTile{s, q0, std::min(POOLATTN_TILE, q_len - q0), 0};
@@ -3754,7 +4147,7 @@ int tgis_engine_create(const tgis_config* cfg, tgis_engine** out) {
   if (!cfg || !out) return fail("null argument");
   if (cfg->abi_version != TGIS_ABI_VERSION) return fail("ABI version mismatch");
   if (cfg->arch == TGIS_ARCH_PONENEX || cfg->arch == TGIS_ARCH_FALERAX || cfg->arch == TGIS_ARCH_REVEPEL || cfg->arch == TGIS_ARCH_SIKAZEN ||
-      cfg->arch == TGIS_ARCH_BISUZEN)
+      cfg->arch == TGIS_ARCH_BISUZEN || cfg->arch == TGIS_ARCH_LUDELIX)
     return fail("this architecture is described layer by layer: use tgis_engine_create_spec");
   if (cfg->arch != TGIS_ARCH_LLAMA && cfg->arch != TGIS_ARCH_OPT) return fail("unknown arch");
   if (cfg->arch == TGIS_ARCH_OPT) {
@@ -3802,7 +4195,7 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
   if (!cfg || !spec || !out || !spec->layers) return fail("null argument");
   if (cfg->abi_version != TGIS_ABI_VERSION) return fail("ABI version mismatch");
   if (cfg->arch != TGIS_ARCH_PONENEX && cfg->arch != TGIS_ARCH_FALERAX && cfg->arch != TGIS_ARCH_REVEPEL && cfg->arch != TGIS_ARCH_SIKAZEN &&
-      cfg->arch != TGIS_ARCH_BISUZEN)
+      cfg->arch != TGIS_ARCH_BISUZEN && cfg->arch != TGIS_ARCH_LUDELIX)
     return fail("tgis_engine_create_spec: arch must be a layer-list architecture");
   if (spec->n_layers < 1 || spec->n_layers > 4096) return fail("bad n_layers");
   if (spec->dtype != TGIS_DTYPE_BF16 && spec->dtype != TGIS_DTYPE_F32) return fail("dtype must be bf16 or fp32");
@@ -3838,6 +4231,45 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
       } else {
         return fail("unknown mixer type" + at);
       }
+      continue;
+    }
+    if ((spec->style & TGIS_STYLE_PRE_RMS) != 0) {
+      if ((spec->style & ~TGIS_STYLE_TIED_HEAD) != TGIS_STYLE_PRE_RMS) return fail("the plain pre-norm style has its own norm placement");
+      if (spec->loop_times > 1 && (spec->loop_start < 0 || spec->loop_stop > spec->n_layers || spec->loop_start >= spec->loop_stop))
+        return fail("the looped span must lie inside the layer list");
+      if (spec->loop_times > 64) return fail("more than 64 passes of a loop");
+      if (spec->loop_add_embed != 0) return fail("the plain pre-norm style adds nothing between the passes of a loop");
+      if (spec->logit_scale != 0.f && spec->logit_scale != 1.f) return fail("the plain pre-norm style has no logit scale");
+      if (s.mlp == TGIS_MLP_MOE_TABLE) {
+        if (s.experts < 1 || s.experts > 4096 || s.top < 1 || s.top > s.experts || s.expert_ff < 1 || s.shared_ff < 0)
+          return fail("bad mixture-of-experts sizes" + at);
+      } else if (s.mlp == TGIS_MLP_DENSE_RELU2 ? s.ff < 1 : s.mlp != TGIS_MLP_NONE) {
+        return fail("bad feed-forward" + at);
+      }
+      if (s.mixer == TGIS_MIXER_GLA) {
+        if (s.heads < 1 || s.dim < 1 || s.dim > OUTER_SCAN_MAX_DIM || s.vdim < 1 || s.decay_rank < 1 || !(s.tau > 0.f))
+          return fail("bad gated-linear-attention sizes" + at);
+        continue;
+      }
+      if (s.mixer != TGIS_MIXER_POOLED_ATTENTION && s.mixer != TGIS_MIXER_CHUNK_RETENTION) return fail("unknown mixer type" + at);
+      if (s.heads < 1 || s.kv_heads < 1 || s.heads % s.kv_heads != 0 || s.dim < 1 || s.vdim < 1 || s.vdim > POOLATTN_MAX_VDIM || s.dim > 512)
+        return fail("bad attention sizes" + at);
+      if (s.rot_dims < 0 || s.rot_dims > s.dim || (s.rot_dims & 1) || (s.rot_dims > 0 && !(s.rot_base > 0.f)))
+        return fail("rot.dims must be even and <= dim, rot.base positive" + at);
+      if (s.yarn_factor > 0.f && !(s.yarn_original > 0.f && s.yarn_fast > 0.f && s.yarn_slow > 0.f && s.rot_base > 1.f))
+        return fail("bad rotary scaling" + at);
+      if (s.band_factor > 0.f && (s.yarn_factor > 0.f || !(s.band_original > 0.f && s.band_low > 0.f && s.band_high > s.band_low)))
+        return fail("bad rotary scaling" + at);
+      if (s.pool > 0) return fail("pooled blocks do not run in the plain pre-norm style" + at);
+      if (s.keep_first < 0 || s.chunk < 0) return fail("bad mask" + at);
+      if ((s.flags & TGIS_LAYER_SHARED_KV) != 0 && s.dim != s.vdim) return fail("values that are the keys must have their size" + at);
+      if ((s.flags & TGIS_LAYER_FULL_QK_NORM) != 0 && ((s.flags & TGIS_LAYER_UNIT_QK) != 0 || (s.heads + s.kv_heads) * s.dim > 40960))
+        return fail("bad query / key norm" + at);
+      if ((s.flags & TGIS_LAYER_OUT_BIAS) != 0) return fail("output biases do not run in the plain pre-norm style" + at);
+      if (s.mixer == TGIS_MIXER_CHUNK_RETENTION &&
+          (s.mm_heads < 1 || s.mm_dim < 1 || s.mm_dim > OUTER_SCAN_MAX_DIM || s.mm_vdim < 1 || s.decay == nullptr || s.mm_rot_dims < 0 ||
+           s.mm_rot_dims > s.mm_dim || (s.mm_rot_dims & 1) || (s.mm_rot_dims > 0 && !(s.mm_rot_base > 0.f))))
+        return fail("bad retention sizes" + at);
       continue;
     }
     if ((spec->style & TGIS_STYLE_PRE_DYT) != 0) {
@@ -3960,9 +4392,8 @@ int tgis_engine_create_spec(const tgis_config* cfg, const tgis_model_spec* spec,
 
 int tgis_engine_load_weight(tgis_engine* e, const char* name, const void* ptr, int64_t rows, int64_t cols, int32_t dtype) {
   if (!e || !name || !ptr) return fail("null argument");
-  if (dtype != 0) return fail("only bf16 (dtype 0) weights are supported");
   if (e->started) return fail("engine already started");
-  return e->load_weight(name, ptr, rows, cols);
+  return e->load_weight(name, ptr, rows, cols, dtype);
 }
 
 int tgis_engine_start(tgis_engine* e) {

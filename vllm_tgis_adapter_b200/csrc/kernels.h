@@ -277,6 +277,8 @@ cudaError_t embed_scale_f32_launch(const int32_t* token_ids, const void* table, 
 //                                                                                            side by side, plain weights)
 //   cast_out != 0 (and w_pre == nullptr): out[t] = resid[t] in the operand type -- the next sublayer reads the stream itself
 //   extra != nullptr: resid[t] += extra[t] after the update;  w_pre2 / out2: out2[t] = rmsnorm(resid[t]) * (w_off + w_pre2)
+//   w_post == nullptr: the sublayer's output is added as it is, resid[t] += mult * y[t];  mix_w == nullptr: every row of the mixture
+//   weighs mix_const;  dot_out != nullptr: dot_out[t] = sigmoid(sum_i n[t, i] * w_dot[i]) with n the fp32 rows that become out
 struct ResidTail {
   const float* y_main;
   const float* y_rows; const int32_t* inv; const float* mix_w; int top;
@@ -288,6 +290,8 @@ struct ResidTail {
   int cast_out;
   const float* extra;                 // optional fp32 [T, hidden]: added to resid after the sublayer's update, before the pre-norm
   const float* w_pre2; void* out2;    // optional second pre-norm of the same rows with another weight (two sublayers side by side)
+  float mix_const;                    // the mixture's weight when mix_w == nullptr
+  const float* w_dot; float* dot_out; // optional: a sigmoid gate computed from the pre-normed row ([hidden] -> one number per token)
 };
 cudaError_t resid_tail_launch(const ResidTail& a, int T, int hidden, cudaStream_t stream);
 // Tail of a layer whose mixer and feed-forward run side by side on ONE normed input and are gated per channel, row per CTA:
@@ -442,12 +446,20 @@ struct PoolAttnGeom {
   int keep_first, chunk;
   int rot_interleaved;   // != 0: rotary pairs are (2i, 2i + 1) instead of (i, i + rot_dims / 2)
   const float* sink;     // fp32 [heads] or nullptr
+  // head_gate != nullptr: the output of head h at token t is multiplied by sigmoid(head_gate[t * gate_ld + h]); all outputs by out_mul
+  const float* head_gate = nullptr; int gate_ld = 0;
+  float out_mul = 1.f;
+  int out_ld = 0;        // elements between output rows (0: heads * vdim)
+  // q_norm != nullptr: all heads of a token's queries are rms-normed as ONE row of heads * dim entries (weight q_norm), and its keys as one
+  // row of kv_heads * dim (k_norm), after the bias and before the rotation
+  const float *q_norm = nullptr, *k_norm = nullptr;
   __host__ __device__ int rows_per_page() const { return pool > 0 ? (KV_BLOCK + pool - 1) / pool : 0; }   // pooled rows a cache page owns
 };
 constexpr int POOLATTN_TILE = 16;      // query tokens per CTA
 constexpr int POOLATTN_MAX_VDIM = 512; // value columns per head the FMA kernel's accumulators cover
 // y fp32 [T, ldy] holds q at column q_off (heads * dim), k at k_off (kv_heads * dim), v at v_off (kv_heads * vdim); bias fp32
-// (q | k | v, in that order, or nullptr) is added first.  cos_sin fp32 [max_pos][rot_dims] = cos | sin.  q_out DT_* [T, heads * dim];
+// (q | k | v, in that order, or nullptr) is added first.  v_off == k_off: the values ARE the keys as projected (bias included, before
+// any norm and rotation; dim == vdim, bias holds q | k).  cos_sin fp32 [max_pos][rot_dims] = cos | sin.  q_out DT_* [T, heads * dim];
 // cache rows K [num_blocks][KV_BLOCK][kv_heads * dim], V [..][kv_heads * vdim] at slot[t].
 cudaError_t poolattn_prep_launch(const float* y, int ldy, int q_off, int k_off, int v_off, const float* bias,
                                  const PoolAttnGeom& g, const float* cos_sin, float eps, const int32_t* positions,
@@ -505,7 +517,11 @@ cudaError_t selective_scan_launch(const SelScan& a, const AttnSeq* seqs, int n_s
 //                      S <- diag(f) S + (1 - f) v^T;  o = S^T silu(q)   (no key: what the gate forgets is what it writes; the
 //                      query reads the state after the token's update)
 //   OUTER_SCAN_LIGHTNING:  S <- decay_h S + silu(k) silu(v)^T;  o = S^T silu(q)   (one fixed decay per head)
-constexpr int OUTER_SCAN_DECAY = 0, OUTER_SCAN_GATED = 1, OUTER_SCAN_SSD = 2, OUTER_SCAN_HGRN = 3, OUTER_SCAN_LIGHTNING = 4;
+//   OUTER_SCAN_RETENTION:  S <- decay_h S + k v^T;  o = S^T q   (the same without activations)
+//   OUTER_SCAN_GLA:    f = sigmoid(decay_raw + w0)^inv_tau (one decay per head and key channel);  S <- diag(f) S + k v^T;  o = S^T q
+//                      (the query reads the state after the token's update)
+constexpr int OUTER_SCAN_DECAY = 0, OUTER_SCAN_GATED = 1, OUTER_SCAN_SSD = 2, OUTER_SCAN_HGRN = 3, OUTER_SCAN_LIGHTNING = 4,
+              OUTER_SCAN_RETENTION = 5, OUTER_SCAN_GLA = 6;
 constexpr int OUTER_SCAN_MAX_DIM = 256;
 struct OuterScan {
   int mode;
@@ -519,12 +535,13 @@ struct OuterScan {
   const float* x; float* x_last; int width;   // optional: x_last[slot] = x[last row of the portion] (the token shift's state)
   int qk_heads;                                // q / k heads (head h reads h / (heads / qk_heads)); 0: one per head
   const float* step_raw; int lds; const float *step_b, *A_log, *D;   // SSD: [T, heads], [heads], [heads], [heads]
-  const float* decay;                          // LIGHTNING: [heads]
+  const float* decay;                          // LIGHTNING, RETENTION: [heads]
+  float inv_tau;                               // GLA
 };
 cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot,
                               cudaStream_t stream);
-// lightning.cu: the recurrence of OUTER_SCAN_LIGHTNING over whole portions, 64 tokens at a time on the tensor cores, from q, k, v in
-// bf16 after silu (outer_scan_launch keeps them fp32).  For steps that carry prompts.
+// lightning.cu: the recurrence of OUTER_SCAN_LIGHTNING / OUTER_SCAN_RETENTION over whole portions, 64 tokens at a time on the tensor
+// cores, from q, k, v in bf16 after their activation or rotation (outer_scan_launch keeps them fp32).  For steps that carry prompts.
 struct LightningChunk {
   const void* qkv; int ld, q_off, k_off, v_off;   // bf16 [T, ld]: q and k [heads * dim], v [heads * vdim] at the given columns
   const float* decay;                             // [heads]
@@ -535,12 +552,23 @@ struct LightningChunk {
 bool lightning_chunk_eligible(int dim, int vdim);
 // out[t, i] = silu(x[t, i]) in bf16, i < n (n, ldx, ldo multiples of 4)
 cudaError_t silu_cast_launch(const float* x, int ldx, void* out, int ldo, int n, int T, cudaStream_t stream);
+// Queries and keys of a recurrent mixer turned in place, x fp32 [T, ld]: heads * dim entries at column q_off (times q_mul) and at k_off
+// (times k_mul); the first rot_dims entries of a head turn as "rotate half" pairs by the table cos_sin (kernels above).  cast != nullptr:
+// q | k | v (v: heads * vdim entries at v_off) go to bf16 rows [T, cast_ld] instead and x stays as it is for tokens >= n_inplace.
+struct RotaryRows {
+  float* x; int ld, q_off, k_off, v_off, heads, dim, vdim, rot_dims;
+  float q_mul, k_mul;
+  const float* cos_sin; const int32_t* positions;
+  void* cast; int cast_ld, n_inplace;
+};
+cudaError_t rotary_rows_launch(const RotaryRows& a, int T, cudaStream_t stream);
 cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot, cudaStream_t stream);
 // out[t, h, :] = rmsnorm(o[t, h, :]) * w[h, :] * act(gate[t, h, :])    act: 0 sigmoid, 1 silu, 2 none (gate may be nullptr)
 // gate_first != 0: out[t, h, :] = rmsnorm(o[t, h, :] * act(gate[t, h, :])) * w[h, :]   (the gate enters the norm)
+// w == nullptr: no weight; mult multiplies every output; out rows are out_ld elements apart (0: heads * vdim)
 cudaError_t head_norm_gate_launch(const float* o, int ldo, int heads, int vdim, const float* w, const float* gate,
                                   int ldg, int act, float eps, void* out, int out_dtype, int T, cudaStream_t stream,
-                                  int gate_first = 0);
+                                  int gate_first = 0, float mult = 1.f, int out_ld = 0);
 // The short convolution's state after a step: conv_state[slot][e][c] = input at position end - (taps - 1) + e, taken from the
 // step's rows x [T, ld] (channels c < n) or, for positions before the portion, from the old state.  Runs after the
 // convolution that read the old state.
@@ -579,6 +607,14 @@ cudaError_t moe_route_launch(const float* logits, int ld, const float* bias, int
 // seg_off[E + 1]: rows per expert, prefix-summed; order[p] = t * top + k of the p-th row; inv[t * top + k] = p
 cudaError_t moe_align_launch(const int32_t* ids, int T, int top, int E, int32_t* seg_off, int32_t* order, int32_t* inv,
                              cudaStream_t stream);
+// Experts chosen by a table of the token id (ids[t, k] = table[tok[t], k], entries in [0, E)): seg_off / order / inv of every such
+// layer of the model in ONE launch at the start of a step -- the choice depends on no activation.
+struct MoeTable {
+  const int32_t* table;            // [vocab, top]
+  int32_t *seg_off, *order, *inv;  // as above
+  int E, top;
+};
+cudaError_t moe_table_align_launch(const MoeTable* layers_dev, int n_layers, int max_E, const int32_t* tok, int vocab, int T, cudaStream_t stream);
 
 // ---- sampler.cu --------------------------------------------------------------------------------------------------
 constexpr int MAX_TOPN = 12;  // reference forces max_logprobs >= 11 (tgis_utils/args.py:214-216)

@@ -1,5 +1,6 @@
 // Lightning attention over the portions of a step, chunk by chunk on the tensor cores (kernels.h: LightningChunk).
-// Per head  S_t = r S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t  with one fixed decay r and q, k, v = silu of their projections.  For the n <= 64
+// Per head  S_t = r S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t  with one fixed decay r and q, k, v = silu of their projections
+// (lightning attention), or q and k rotated by their position and v as projected (retention).  For the n <= 64
 // tokens i, j = 0 .. n-1 of a chunk and the state S that the tokens before it left, this is
 //     o_i = r^(i+1) S^T q_i + sum_{j <= i} r^(i-j) (q_i . k_j) v_j          S <- r^n S + sum_j r^(n-1-j) k_j v_j^T
 // so a portion of T tokens takes T / 64 dependent steps of matrix products instead of T dependent rank-one updates.
@@ -9,7 +10,7 @@
 // by lane, the B fragments of the read-out (Q S), so the state never passes through shared memory.  The decayed scores are computed
 // once per CTA (16 rows per warp) and shared.
 //
-// silu_cast_kernel makes q, k and v from the projections once for all CTAs; the chunk after the current one lands in the other half of
+// silu_cast_kernel (or rotary_rows_kernel) makes q, k and v from the projections once for all CTAs; the chunk after the current one lands in the other half of
 // a double buffer.
 //
 // Precision: q, k and v are rounded to bf16 after silu, as any product input.  Everything the recurrence adds is kept to 32 bits'
@@ -79,6 +80,38 @@ silu_cast_kernel(const float* __restrict__ x, int ldx, bf* __restrict__ out, int
     pk.y = *reinterpret_cast<const uint32_t*>(&hi);
     *reinterpret_cast<uint2*>(out + (size_t)t * ldo + i) = pk;
   }
+}
+
+// grid (T, y): one token per x; pairs / values of the row in strides of the CTA (kernels.h: RotaryRows)
+__global__ void __launch_bounds__(256)
+rotary_rows_kernel(RotaryRows a) {
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x, D = a.dim, half = a.rot_dims / 2, hd = a.heads * D;
+  float* row = a.x + (size_t)t * a.ld;
+  const float* cs = a.cos_sin != nullptr ? a.cos_sin + (size_t)a.positions[t] * a.rot_dims : nullptr;
+  bf* dst = (a.cast != nullptr && t >= a.n_inplace) ? reinterpret_cast<bf*>(a.cast) + (size_t)t * a.cast_ld : nullptr;
+  const int per = half + D - a.rot_dims;   // per head: the pairs, then the entries that pass
+  const int n_qk = 2 * a.heads * per;
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < n_qk; i += gridDim.y * 256) {
+    const bool is_k = i >= a.heads * per;
+    const int r = is_k ? i - a.heads * per : i, h = r / per, e = r % per;
+    const float mul = is_k ? a.k_mul : a.q_mul;
+    float* src = row + (is_k ? a.k_off : a.q_off) + h * D;
+    bf* out = dst != nullptr ? dst + (is_k ? hd : 0) + h * D : nullptr;
+    if (e < half) {
+      const float c = cs[e], s = cs[half + e], u = src[e], v = src[e + half];
+      const float u2 = (u * c - v * s) * mul, v2 = (v * c + u * s) * mul;
+      if (out != nullptr) { out[e] = __float2bfloat16_rn(u2); out[e + half] = __float2bfloat16_rn(v2); }
+      else { src[e] = u2; src[e + half] = v2; }
+    } else {
+      const int p = e - half + a.rot_dims;
+      if (out != nullptr) out[p] = __float2bfloat16_rn(src[p] * mul);
+      else src[p] *= mul;
+    }
+  }
+  if (dst != nullptr)
+    for (int i = blockIdx.y * 256 + threadIdx.x; i < a.heads * a.vdim; i += gridDim.y * 256) dst[2 * hd + i] = __float2bfloat16_rn(row[a.v_off + i]);
 }
 
 // DKS: k-steps of 16 over dim (dim <= 16 DKS, a multiple of 16)
@@ -313,6 +346,13 @@ cudaError_t silu_cast_launch(const float* x, int ldx, void* out, int ldo, int n,
   if (n % 4 != 0 || ldx % 4 != 0 || ldo % 4 != 0 || (reinterpret_cast<uintptr_t>(x) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 7) != 0)
     return cudaErrorInvalidValue;
   return launch_k(silu_cast_kernel, dim3(T, std::min((n + 1023) / 1024, 2)), dim3(256), 0, stream, x, ldx, reinterpret_cast<bf*>(out), ldo, n);
+}
+
+cudaError_t rotary_rows_launch(const RotaryRows& a, int T, cudaStream_t stream) {
+  if (T <= 0) return cudaSuccess;
+  if (a.heads < 1 || a.dim < 1 || a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1) || (a.rot_dims > 0 && a.cos_sin == nullptr))
+    return cudaErrorInvalidValue;
+  return launch_k(rotary_rows_kernel, dim3(T, std::min((a.heads * a.dim + 511) / 512, 8)), dim3(256), 0, stream, a);
 }
 
 cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot, cudaStream_t stream) {

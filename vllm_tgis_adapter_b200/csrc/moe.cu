@@ -135,7 +135,64 @@ moe_align_kernel(const int32_t* __restrict__ ids, int n, int E, int32_t* __restr
   }
 }
 
+// one CTA per layer; dynamic shared memory: 2 max_E ints
+__global__ void __launch_bounds__(1024)
+moe_table_align_kernel(const MoeTable* __restrict__ layers, const int32_t* __restrict__ tok, int vocab, int T) {
+  extern __shared__ int sm_i[];
+  griddep_launch();
+  griddep_wait();
+  const MoeTable a = layers[blockIdx.x];
+  const int E = a.E, top = a.top, n = T * top, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  int* cnt = sm_i;
+  int* cur = sm_i + E;
+  __shared__ int warp_tot[32];
+  auto expert = [&](int i) {
+    const int t = tok[i / top];
+    return a.table[(size_t)(t >= 0 && t < vocab ? t : 0) * top + i % top];   // (as the embedding reads ids outside the vocabulary)
+  };
+  for (int e = threadIdx.x; e < E; e += 1024) cnt[e] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < n; i += 1024) atomicAdd(&cnt[expert(i)], 1);
+  __syncthreads();
+  int base = 0;   // exclusive prefix sum, 1024 experts at a time
+  for (int e0 = 0; e0 < E; e0 += 1024) {
+    const int e = e0 + threadIdx.x, c = e < E ? cnt[e] : 0;
+    int run = c;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const int up = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += up;
+    }
+    if (lane == 31) warp_tot[warp] = run;
+    __syncthreads();
+    int before = base, all = 0;
+    for (int w = 0; w < 32; ++w) {
+      if (w < warp) before += warp_tot[w];
+      all += warp_tot[w];
+    }
+    if (e < E) {
+      cur[e] = before + run - c;
+      a.seg_off[e] = before + run - c;
+    }
+    base += all;
+    __syncthreads();
+  }
+  if (threadIdx.x == 0) a.seg_off[E] = base;
+  // the place of a row inside its segment does not enter any result (every row of a grouped product is computed alone)
+  for (int i = threadIdx.x; i < n; i += 1024) {
+    const int p = atomicAdd(&cur[expert(i)], 1);
+    a.order[p] = i;
+    a.inv[i] = p;
+  }
+}
+
 }  // namespace
+
+cudaError_t moe_table_align_launch(const MoeTable* layers_dev, int n_layers, int max_E, const int32_t* tok, int vocab, int T, cudaStream_t stream) {
+  if (T <= 0 || n_layers <= 0) return cudaSuccess;
+  if (max_E < 1 || (size_t)2 * max_E * 4 > 40 * 1024) return cudaErrorInvalidValue;
+  return launch_k(moe_table_align_kernel, dim3(n_layers), dim3(1024), (size_t)2 * max_E * sizeof(int), stream, layers_dev, tok, vocab, T);
+}
 
 cudaError_t moe_route_launch(const float* logits, int ld, const float* bias, int E, int top, int32_t* ids, float* w,
                              float* side_gate, int T, cudaStream_t stream, int weight_mode, int groups, int keep) {

@@ -246,8 +246,8 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
   float u_r[RPT];   // DECAY: the bonus u of this thread's rows; GATED: the normaliser n of its rows (the same in every lane)
   float m_run = 0.f;
   const float ssd_rate = MODE == OUTER_SCAN_SSD ? -expf(a.A_log[h]) : 0.f, ssd_skip = MODE == OUTER_SCAN_SSD ? a.D[h] : 0.f;
-  const float fixed_decay = MODE == OUTER_SCAN_LIGHTNING ? a.decay[h] : 0.f;
-  if (MODE == OUTER_SCAN_SSD || MODE == OUTER_SCAN_HGRN || MODE == OUTER_SCAN_LIGHTNING) {
+  const float fixed_decay = (MODE == OUTER_SCAN_LIGHTNING || MODE == OUTER_SCAN_RETENTION) ? a.decay[h] : 0.f;
+  if (MODE == OUTER_SCAN_SSD || MODE == OUTER_SCAN_HGRN || MODE == OUTER_SCAN_LIGHTNING || MODE == OUTER_SCAN_RETENTION || MODE == OUTER_SCAN_GLA) {
 #pragma unroll
     for (int j = 0; j < RPT; ++j) u_r[j] = 0.f;
   } else if (MODE == OUTER_SCAN_DECAY) {
@@ -284,7 +284,7 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
       const bool in = tok && i < D;
       pq[e] = in ? qr[i] : 0.f;
       pk[e] = in ? (MODE == OUTER_SCAN_HGRN ? a.u[(size_t)h * D + i] : kr[i]) : 0.f;   // HGRN: the gate's lower bound
-      if (MODE == OUTER_SCAN_DECAY || MODE == OUTER_SCAN_HGRN)
+      if (MODE == OUTER_SCAN_DECAY || MODE == OUTER_SCAN_HGRN || MODE == OUTER_SCAN_GLA)
         pd[e] = in ? a.decay_raw[row * a.ldd + (size_t)h * D + i] + a.w0[(size_t)h * D + i] : 0.f;
     }
 #pragma unroll
@@ -319,6 +319,7 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
             v3[i] = pq[e] * a.q_scale;
             v3[D + i] = pk[e];
             if (MODE == OUTER_SCAN_DECAY) v3[2 * D + i] = expf(-expf(pd[e]));
+            if (MODE == OUTER_SCAN_GLA) v3[2 * D + i] = expf(logsigmoid_f(pd[e]) * a.inv_tau);
           }
         }
       }
@@ -350,7 +351,7 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
             S[j] = fmaf(v3[2 * D + i], S[j], kv);
           }
         }
-      } else if (MODE == OUTER_SCAN_HGRN) {
+      } else if (MODE == OUTER_SCAN_HGRN || MODE == OUTER_SCAN_GLA) {
 #pragma unroll
         for (int j = 0; j < RPT; ++j) {
           const int i = g + j * OS_GROUPS;
@@ -359,7 +360,7 @@ outer_scan_kernel(OuterScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
             o = fmaf(v3[i], S[j], o);
           }
         }
-      } else if (MODE == OUTER_SCAN_LIGHTNING) {
+      } else if (MODE == OUTER_SCAN_LIGHTNING || MODE == OUTER_SCAN_RETENTION) {
 #pragma unroll
         for (int j = 0; j < RPT; ++j) {
           const int i = g + j * OS_GROUPS;
@@ -613,7 +614,7 @@ delta_scan_kernel(DeltaScan a, const AttnSeq* __restrict__ seqs, const int32_t* 
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ o, int ldo, int heads, int vdim, const float* __restrict__ w,
                       const float* __restrict__ gate, int ldg, int act, float eps, void* __restrict__ out, int out_dtype,
-                      int out_ld, int gate_first) {
+                      int out_ld, int gate_first, float mult) {
   griddep_launch();
   griddep_wait();
   const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -629,7 +630,7 @@ head_norm_gate_kernel(const float* __restrict__ o, int ldo, int heads, int vdim,
     const float rs = 1.f / sqrtf(warp_sum_f(ss) / (float)vdim + eps);
     for (int i = lane; i < vdim; i += 32) {
       const float v = orow[i] * (act == 1 ? silu_f(grow[i]) : sigmoid_f(grow[i]));
-      st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, v * rs * w[(size_t)h * vdim + i]);
+      st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, v * rs * (w != nullptr ? w[(size_t)h * vdim + i] : 1.f) * mult);
     }
     return;
   }
@@ -641,7 +642,7 @@ head_norm_gate_kernel(const float* __restrict__ o, int ldo, int heads, int vdim,
       const float gl = gate[(size_t)t * ldg + (size_t)h * vdim + i];
       gv = act == 1 ? silu_f(gl) : sigmoid_f(gl);
     }
-    st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, orow[i] * rs * w[(size_t)h * vdim + i] * gv);
+    st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, orow[i] * rs * (w != nullptr ? w[(size_t)h * vdim + i] : 1.f) * (gv * mult));
   }
 }
 
@@ -649,7 +650,7 @@ head_norm_gate_kernel(const float* __restrict__ o, int ldo, int heads, int vdim,
 __global__ void __launch_bounds__(256)
 head_norm_gate_wide_kernel(const float* __restrict__ o, int ldo, int heads, int vdim, const float* __restrict__ w,
                            const float* __restrict__ gate, int ldg, int act, float eps, void* __restrict__ out, int out_dtype,
-                           int out_ld, int gate_first) {
+                           int out_ld, int gate_first, float mult) {
   __shared__ float red[8];
   griddep_launch();
   griddep_wait();
@@ -671,7 +672,7 @@ head_norm_gate_wide_kernel(const float* __restrict__ o, int ldo, int heads, int 
   const float rs = 1.f / sqrtf(tot / (float)vdim + eps);
   for (int i = tid; i < vdim; i += 256) {
     const float gv = act == 2 ? 1.f : act == 1 ? silu_f(grow[i]) : sigmoid_f(grow[i]);
-    st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, orow[i] * gv * rs * w[(size_t)h * vdim + i]);
+    st_op(out, out_dtype, (size_t)t * out_ld + (size_t)h * vdim + i, orow[i] * gv * rs * (w != nullptr ? w[(size_t)h * vdim + i] : 1.f) * mult);
   }
 }
 
@@ -754,6 +755,14 @@ cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seq
     if (a.decay == nullptr) return cudaErrorInvalidValue;
     return outer_scan_mode<OUTER_SCAN_LIGHTNING>(a, seqs, n_seqs, tok_slot, stream);
   }
+  if (a.mode == OUTER_SCAN_RETENTION) {
+    if (a.decay == nullptr) return cudaErrorInvalidValue;
+    return outer_scan_mode<OUTER_SCAN_RETENTION>(a, seqs, n_seqs, tok_slot, stream);
+  }
+  if (a.mode == OUTER_SCAN_GLA) {
+    if (a.decay_raw == nullptr || a.w0 == nullptr || !(a.inv_tau > 0.f)) return cudaErrorInvalidValue;
+    return outer_scan_mode<OUTER_SCAN_GLA>(a, seqs, n_seqs, tok_slot, stream);
+  }
   if (a.mode == OUTER_SCAN_HGRN) {
     if (a.decay_raw == nullptr || a.w0 == nullptr || a.u == nullptr) return cudaErrorInvalidValue;
     return outer_scan_mode<OUTER_SCAN_HGRN>(a, seqs, n_seqs, tok_slot, stream);
@@ -764,15 +773,15 @@ cudaError_t outer_scan_launch(const OuterScan& a, const AttnSeq* seqs, int n_seq
 
 cudaError_t head_norm_gate_launch(const float* o, int ldo, int heads, int vdim, const float* w, const float* gate,
                                   int ldg, int act, float eps, void* out, int out_dtype, int T, cudaStream_t stream,
-                                  int gate_first) {
+                                  int gate_first, float mult, int out_ld) {
   if (T <= 0) return cudaSuccess;
   if (act == 2) gate_first = 0;
   else if (gate == nullptr) return cudaErrorInvalidValue;
   if (vdim >= 1024 && heads <= 65535)
     return launch_k(head_norm_gate_wide_kernel, dim3(T, heads), dim3(256), 0, stream, o, ldo, heads, vdim, w, gate, ldg, act, eps, out,
-                    out_dtype, heads * vdim, gate_first);
+                    out_dtype, out_ld > 0 ? out_ld : heads * vdim, gate_first, mult);
   return launch_k(head_norm_gate_kernel, dim3(T, (heads + 3) / 4), dim3(128), 0, stream, o, ldo, heads, vdim, w, gate, ldg, act,
-                  eps, out, out_dtype, heads * vdim, gate_first);
+                  eps, out, out_dtype, out_ld > 0 ? out_ld : heads * vdim, gate_first, mult);
 }
 
 cudaError_t conv_state_save_launch(const float* x, int ld, int n, int taps, const AttnSeq* seqs, int n_seqs,

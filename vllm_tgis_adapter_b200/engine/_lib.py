@@ -10,14 +10,15 @@ import ctypes as C
 import os
 from pathlib import Path
 
-ABI_VERSION = 12
-ARCH_LLAMA, ARCH_OPT, ARCH_PONENEX, ARCH_FALERAX, ARCH_REVEPEL, ARCH_SIKAZEN, ARCH_BISUZEN = 0, 1, 2, 3, 4, 5, 6
+ABI_VERSION = 13
+ARCH_LLAMA, ARCH_OPT, ARCH_PONENEX, ARCH_FALERAX, ARCH_REVEPEL, ARCH_SIKAZEN, ARCH_BISUZEN, ARCH_LUDELIX = 0, 1, 2, 3, 4, 5, 6, 7
 MIXER_LATENT_ATTENTION, MIXER_PARALLEL, MIXER_SELECTIVE_SCAN, MIXER_WKV = 1, 2, 3, 4
 MIXER_SIGMOID_ATTENTION, MIXER_SSD, MIXER_CHANNEL_DELTA = 5, 6, 7
-MIXER_POOLED_ATTENTION, MIXER_HGRN, MIXER_WINDOW_LIGHTNING = 8, 9, 10
-MLP_NONE, MLP_MOE, MLP_DENSE_GELU, MLP_MOE_SIGMOID, MLP_DENSE_SILU, MLP_MOE_GROUPED = 0, 1, 2, 3, 4, 5
+MIXER_POOLED_ATTENTION, MIXER_HGRN, MIXER_WINDOW_LIGHTNING, MIXER_CHUNK_RETENTION, MIXER_GLA = 8, 9, 10, 11, 12
+MLP_NONE, MLP_MOE, MLP_DENSE_GELU, MLP_MOE_SIGMOID, MLP_DENSE_SILU, MLP_MOE_GROUPED, MLP_DENSE_RELU2, MLP_MOE_TABLE = 0, 1, 2, 3, 4, 5, 6, 7
 LAYER_ROT_INTERLEAVED, LAYER_SINK, LAYER_NO_OUT_GATE, LAYER_QKV_BIAS, LAYER_UNIT_QK, LAYER_OUT_BIAS = 1, 2, 4, 8, 16, 32
-STYLE_POST_NORM, STYLE_TIED_HEAD, STYLE_PARALLEL_GATED, STYLE_PARALLEL_PAIR, STYLE_PRE_DYT = 1, 2, 4, 8, 16
+LAYER_SHARED_KV, LAYER_FULL_QK_NORM, LAYER_HEAD_GATE = 64, 128, 256
+STYLE_POST_NORM, STYLE_TIED_HEAD, STYLE_PARALLEL_GATED, STYLE_PARALLEL_PAIR, STYLE_PRE_DYT, STYLE_PRE_RMS = 1, 2, 4, 8, 16, 32
 DTYPE_BF16, DTYPE_F32 = 0, 1
 MAX_REQUEST_ID = 96
 MAX_TOPN = 12
@@ -54,6 +55,9 @@ class TgisLayerSpec(C.Structure):
         ("pool", C.c_int32), ("rot_linear", C.c_float), ("flags", C.c_int32), ("keep_first", C.c_int32),
         ("chunk", C.c_int32), ("identity", C.c_int32), ("expert_groups", C.c_int32), ("expert_groups_keep", C.c_int32),
         ("reserved2", C.c_int32), ("decay", C.POINTER(C.c_float)),
+        ("band_factor", C.c_float), ("band_original", C.c_float), ("band_low", C.c_float), ("band_high", C.c_float),
+        ("mm_rot_base", C.c_float), ("mm_rot_dims", C.c_int32), ("left_scale", C.c_float), ("right_scale", C.c_float),
+        ("tau", C.c_float), ("reserved3", C.c_int32),
     ]
 
 

@@ -31,8 +31,8 @@ class ModelConfig:
     rms_eps: float = 1e-5
     max_model_len: int = 2048
     arch: str = "llama"
-    # arch "ponenex" (engine/ponenex.py), "falerax" (engine/falerax.py), "revepel" (engine/revepel.py), "sikazen" (engine/sikazen.py) and
-    # "bisuzen" (engine/bisuzen.py): the layers are described one by one;
+    # arch "ponenex" (engine/ponenex.py), "falerax" (engine/falerax.py), "revepel" (engine/revepel.py), "sikazen" (engine/sikazen.py),
+    # "bisuzen" (engine/bisuzen.py) and "ludelix" (engine/ludelix.py): the layers are described one by one;
     # n_q_heads / n_kv_heads / ffn are unused
     layers: list | None = None          # list of the family module's LayerSpec
     embed_scale: float = 1.0
@@ -43,7 +43,7 @@ class ModelConfig:
     loop: tuple = (0, 0, 1)             # arch "sikazen" / "bisuzen": layers [start, stop) run `times` passes in a row
 
 
-LAYER_LIST_ARCHS = ("ponenex", "falerax", "revepel", "sikazen", "bisuzen")   # created with tgis_engine_create_spec; bfloat16 or float32
+LAYER_LIST_ARCHS = ("ponenex", "falerax", "revepel", "sikazen", "bisuzen", "ludelix")   # created with tgis_engine_create_spec; bfloat16 or float32
 
 
 # Named architectures (real dims; this offline build runs them on synthetic weights — SURVEY.md §0)
@@ -79,15 +79,9 @@ def cache_block_bytes(mc: ModelConfig) -> int:
         from .sikazen import cache_block_elems
 
         return max((4 if mc.dtype == "float32" else 2) * cache_block_elems(mc, KV_BLOCK_TOKENS), 1)
-    if mc.arch in ("falerax", "revepel", "bisuzen"):
-        if mc.arch == "falerax":
-            from .falerax import cache_row_elems
-        elif mc.arch == "bisuzen":
-            from .bisuzen import cache_row_elems
-        else:
-            from .revepel import cache_row_elems
-
-        return max(KV_BLOCK_TOKENS * (4 if mc.dtype == "float32" else 2) * cache_row_elems(mc), 1)
+    if mc.arch in ("falerax", "revepel", "bisuzen", "ludelix"):
+        family = importlib.import_module("." + mc.arch, __package__)
+        return max(KV_BLOCK_TOKENS * (4 if mc.dtype == "float32" else 2) * family.cache_row_elems(mc), 1)
     return 2 * mc.n_layers * mc.n_kv_heads * KV_BLOCK_TOKENS * 128 * 2
 
 
@@ -174,7 +168,8 @@ class NativeEngine:
         cfg.use_cuda_graphs, cfg.debug_gemm_ref, cfg.seed = int(use_cuda_graphs), 1 if debug_gemm_ref else 0, seed
         cfg.max_loras, cfg.max_lora_rank = int(max_loras), int(max_lora_rank) if max_loras else 0
         archs = {"llama": _lib.ARCH_LLAMA, "opt": _lib.ARCH_OPT, "ponenex": _lib.ARCH_PONENEX, "falerax": _lib.ARCH_FALERAX,
-                 "revepel": _lib.ARCH_REVEPEL, "sikazen": _lib.ARCH_SIKAZEN, "bisuzen": _lib.ARCH_BISUZEN}
+                 "revepel": _lib.ARCH_REVEPEL, "sikazen": _lib.ARCH_SIKAZEN, "bisuzen": _lib.ARCH_BISUZEN,
+                 "ludelix": _lib.ARCH_LUDELIX}
         if model.arch not in archs:
             raise EngineError(f"unknown architecture {model.arch!r}")
         cfg.arch = archs[model.arch]
@@ -191,18 +186,20 @@ class NativeEngine:
 
     # -- weights ------------------------------------------------------------------------------------------------
     def load_weight(self, name: str, tensor) -> None:
-        """tensor: contiguous torch bf16 tensor (host or device) — "PyTorch tensors for weights only"."""
+        """tensor: contiguous torch bf16 tensor (host or device) — "PyTorch tensors for weights only"; integer tensors are tables
+        and go over as int32."""
         import torch
 
         t = tensor.detach()
-        if t.dtype != torch.bfloat16:
-            t = t.to(torch.bfloat16)
+        table = not t.is_floating_point()
+        if t.dtype != (torch.int32 if table else torch.bfloat16):
+            t = t.to(torch.int32 if table else torch.bfloat16)
         if t.dim() == 0:
             t = t.reshape(1)   # a single number (norms that carry one weight for all channels)
         t = t.contiguous()
         rows = t.shape[0]
         cols = t.numel() // rows if rows else 0
-        if self.lib.tgis_engine_load_weight(self._h, name.encode(), C.c_void_p(t.data_ptr()), rows, cols, 0) != 0:
+        if self.lib.tgis_engine_load_weight(self._h, name.encode(), C.c_void_p(t.data_ptr()), rows, cols, 1 if table else 0) != 0:
             raise EngineError(f"load_weight({name}) failed: {_lib.last_error(self.lib)}")
 
     def load_weights(self, weights: dict) -> None:

@@ -41,6 +41,10 @@ def model_config_from_hf(path: Path, max_model_len: int | None, dtype: str = "bf
         from .bisuzen import model_config_from_json
 
         return model_config_from_json(cfg, max_model_len, dtype)
+    if cfg.get("architecture") == "Ludelix":
+        from .ludelix import checkpoint_shapes, model_config_from_json
+
+        return model_config_from_json(cfg, max_model_len, dtype, checkpoint_shapes(path))
     archs = cfg.get("architectures") or []
     if cfg.get("model_type") == "opt" or any("OPT" in a for a in archs):
         return _opt_model_config(cfg, max_model_len)
@@ -193,12 +197,13 @@ def _resolve_model(args):
         return mc, path
     from .bisuzen import PRESETS as BISUZEN_PRESETS
     from .falerax import PRESETS as FALERAX_PRESETS
+    from .ludelix import PRESETS as LUDELIX_PRESETS
     from .ponenex import PRESETS as PONENEX_PRESETS
     from .revepel import PRESETS as REVEPEL_PRESETS
     from .sikazen import PRESETS as SIKAZEN_PRESETS
 
     PONENEX_PRESETS = {**PONENEX_PRESETS, **FALERAX_PRESETS, **REVEPEL_PRESETS, **SIKAZEN_PRESETS,
-                       **BISUZEN_PRESETS}   # the presets of the layer-list architectures
+                       **BISUZEN_PRESETS, **LUDELIX_PRESETS}   # the presets of the layer-list architectures
     if args.model in PRESETS or args.model in PONENEX_PRESETS:
         if not args.synthetic_weights:
             raise ValueError(f"--model {args.model} is a preset name: pass --synthetic-weights or a model directory")
