@@ -770,13 +770,14 @@ def run_ours(args) -> dict | None:
 
 
 # ------------------------------------------------------------------------------------------------ --arch-compare
-# Prefill and decode throughput of the layer-list families (Ponenex, Falerax, Revepel, Sikazen, Bisuzen) beside the closest existing family (Llama) at equal hidden size, layer
+# Prefill and decode throughput of the layer-list families (Ponenex, Falerax, Revepel, Sikazen, Bisuzen, Ludelix) beside the closest existing family (Llama) at equal hidden size, layer
 # count and active feed-forward width, random weights, device-timed (the engine's CUDA events around every step).  Not the
 # default workload: `python bench.py --arch-compare` prints its own JSON line; the default JSON line is untouched.
 ARCH_COMPARE = [("ponenex-1k", "llama-cmp-1k"), ("ponenex-2k", "llama-cmp-2k"), ("falerax-1k", "llama-cmp-1k"),
                 ("falerax-2k", "llama-cmp-2k"), ("revepel-1k", "llama-cmp-1k"), ("revepel-2k", "llama-cmp-2k"),
                 ("sikazen-1k", "llama-cmp-1k"), ("sikazen-2k", "llama-cmp-2k"),
-                ("bisuzen-1k", "llama-cmp-1k"), ("bisuzen-2k", "llama-cmp-2k")]
+                ("bisuzen-1k", "llama-cmp-1k"), ("bisuzen-2k", "llama-cmp-2k"),
+                ("ludelix-1k", "llama-cmp-1k"), ("ludelix-2k", "llama-cmp-2k")]
 
 
 def _arch_work(mc, B: int, ctx: float) -> tuple[float, float]:
@@ -887,6 +888,32 @@ def _arch_work(mc, B: int, ctx: float) -> tuple[float, float]:
             # and reads + writes its fp32 state
             bytes_ += 2.0 * (dense + ff_step) + B * (2.0 * cache + 8.0 * state)
         return flops + 2.0 * h * v, bytes_ + 2.0 * h * v
+    if mc.arch == "ludelix":
+        flops = bytes_ = 0.0
+        for l in mc.layers:
+            hd, hv, scan, state, cache = l.heads * l.dim, l.heads * l.vdim, 0, 0, 0
+            if l.kind == "gla":
+                dense = h * (2 * hd + 2 * hv + l.rank) + l.rank * hd + hv * h
+                state = hd * l.vdim
+                scan = 2 * state
+            else:
+                keys = min(ctx, l.window or l.chunk or ctx)
+                own_v = l.kind == "parallel"   # the windowed attention's values are its keys
+                dense = h * (hd + l.kv_heads * (l.dim + (l.vdim if own_v else 0))) + hv * h
+                scan, cache = l.heads * keys * (l.dim + l.vdim), keys * l.kv_heads * (l.dim + l.vdim)
+                if own_v:
+                    dense += h * l.heads + 2 * h * l.ret_heads * l.ret_dim + 3 * h * l.ret_heads * l.ret_vdim
+                    state = l.ret_heads * l.ret_dim * l.ret_vdim
+                    scan += 2 * state
+            ff = ff_step = 2 * h * l.ff
+            if l.moe:
+                ff = 3 * h * (l.top * l.expert_ff + l.shared_ff) + h
+                ff_step = 3 * h * (min(l.experts, B * l.top) * l.expert_ff + l.shared_ff) + h
+            flops += 2.0 * (dense + ff + scan)
+            # a decode step streams the weights once (every expert the batch touches), every sequence's visible cache rows, and
+            # reads + writes its fp32 state
+            bytes_ += 2.0 * (dense + ff_step) + B * (2.0 * cache + 8.0 * state)
+        return flops + 2.0 * h * v, bytes_ + 2.0 * h * v
     qd, kvd = mc.n_q_heads * 128, mc.n_kv_heads * 128
     per_layer = h * (qd + 2 * kvd) + qd * h + 3 * h * mc.ffn
     flops = mc.n_layers * 2.0 * (per_layer + mc.n_q_heads * ctx * 2 * 128) + 2.0 * h * v
@@ -910,7 +937,9 @@ def run_arch_compare(args) -> None:
 
     from vllm_tgis_adapter_b200.engine.bisuzen import PRESETS as BSZ
 
-    PNX = {**PNX, **FLX, **RVP, **SKZ, **BSZ}   # the presets of the layer-list families
+    from vllm_tgis_adapter_b200.engine.ludelix import PRESETS as LDX
+
+    PNX = {**PNX, **FLX, **RVP, **SKZ, **BSZ, **LDX}   # the presets of the layer-list families
 
     torch.cuda.set_device(0)
     hbm_gbs, _ = peaks()

@@ -124,6 +124,11 @@ int tgis_k_rmsnorm_f32(const float* x, int32_t ldx, const float* w, float w_off,
 int tgis_k_resid_tail(const float* y_main, const float* y_rows, const int32_t* inv, const float* mix_w, int32_t top,
                       const float* y_side, const float* side_gate, const float* w_post, const float* w_pre, float* resid,
                       void* out, int32_t out_dt, float mult, float w_off, float eps, int32_t T, int32_t hidden);
+/* resid += y (no norm of its own); out = rmsnorm(resid) * w_pre; y = y_main, or mix_const * sum_k y_rows[inv[t * top + k]] +
+ * side_gate[t] * y_side[t]; dot_out (optional): sigmoid(normed row . w_dot) */
+int tgis_k_resid_tail_plain(const float* y_main, const float* y_rows, const int32_t* inv, float mix_const, int32_t top, const float* y_side,
+                            const float* side_gate, const float* w_pre, float* resid, void* out, int32_t out_dt, const float* w_dot,
+                            float* dot_out, float eps, int32_t T, int32_t hidden);
 typedef struct tgis_k_latent_geom {
   int32_t heads, dim, rot_dim, vdim, kv_rank, q_rank, window, rot_dims;
   float scale;
@@ -151,6 +156,9 @@ int tgis_k_dyt_tail(const float* y_main, const float* b_main, const float* y_pai
                     const float* y_rows, const int32_t* inv, const int32_t* ids, const float* mix_w, int32_t top, int32_t n_experts,
                     const float* in_w, const float* in_b, const float* in_alpha, float* resid, const float* w, const float* b,
                     const float* alpha, float out_scale, void* out, int32_t out_dt, int32_t T, int32_t hidden);
+/* the same row lists when a table names every token id's experts: table [vocab, top], tok [T] */
+int tgis_k_moe_table_align(const int32_t* table, int32_t vocab, const int32_t* tok, int32_t T, int32_t top, int32_t E, int32_t* seg_off,
+                           int32_t* order, int32_t* inv);
 int tgis_k_moe_align(const int32_t* ids, int32_t T, int32_t top, int32_t E, int32_t* seg_off, int32_t* order, int32_t* inv);
 
 /* ---- softcapped grouped-query attention (csrc/attention_capped.cu) ---- */
@@ -182,9 +190,14 @@ typedef struct tgis_k_poolattn_geom {
   int32_t unit_norm;
   int32_t keep_first, chunk, rot_interleaved;   /* the first keep_first tokens stay visible behind the window; chunks of `chunk` positions */
   const float* sink;                            /* device, fp32 [heads], or NULL */
+  const float* head_gate;                       /* head h's output of token t times sigmoid(head_gate[t * gate_ld + h]), or NULL */
+  int32_t gate_ld, out_ld;                      /* out_ld: elements between output rows (0: heads * vdim) */
+  float out_mul;                                /* factor on every output (0: one) */
+  int32_t reserved;
+  const float *q_norm, *k_norm;                 /* norms over all query / key heads at once, or NULL */
 } tgis_k_poolattn_geom;
-/* y fp32 [T, ldy] = [.. q .. k .. v ..] at the given columns (+ bias [q | k | v] or NULL) -> rotated, unit-normed queries and
- * cache rows at slots[t] */
+/* y fp32 [T, ldy] = [.. q .. k .. v ..] at the given columns (+ bias [q | k | v] or NULL) -> normed, rotated queries and
+ * cache rows at slots[t]; v_off == k_off: the values are the keys as projected (bias [q | k]) */
 int tgis_k_poolattn_prep(const float* y, int32_t ldy, int32_t q_off, int32_t k_off, int32_t v_off, const float* bias,
                          const tgis_k_poolattn_geom* g, const float* cos_sin, float eps, const int32_t* positions,
                          const int32_t* slots, void* q_out, void* k_cache, void* v_cache, int32_t dt, int32_t T);
@@ -233,6 +246,16 @@ int tgis_k_outer_scan(int32_t mode, const float* q, const float* k, const float*
 int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_t ldq, int32_t ldk, int32_t ldv, const float* decay,
                           float* S, float* out, int32_t ldo, int32_t heads, int32_t dim, int32_t vdim, const int32_t* seqs_host,
                           int32_t n_seqs, const int32_t* tok_slot, int32_t chunked);
+/* retention: queries and keys of x [T, ld] turned by cos_sin [positions][rot_dims] (in place), keys times k_mul, then
+ * S <- decay_h S + k v^T, o = S^T q; chunked as above */
+int tgis_k_retention_scan(float* x, int32_t ld, int32_t q_off, int32_t k_off, int32_t v_off, const float* cos_sin, const int32_t* positions,
+                          int32_t rot_dims, float k_mul, const float* decay, float* S, float* out, int32_t ldo, int32_t heads, int32_t dim,
+                          int32_t vdim, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot, int32_t T, int32_t chunked);
+/* gated linear attention: x [T, ld] holds q, k, v and the low-rank map's inner row a1; a2 bf16 [heads * dim, rank];
+ * f = sigmoid(a2 a1 + bias)^inv_tau, S <- diag(f) S + k v^T, o = S^T q * q_scale; chunked != 0: GLA_CHUNK tokens at a time on the tensor cores */
+int tgis_k_gla_scan(const float* x, int32_t ld, int32_t q_off, int32_t k_off, int32_t v_off, int32_t a1_off, float q_scale, const void* a2,
+                    int32_t rank, const float* bias, float inv_tau, float* S, float* out, int32_t ldo, int32_t heads, int32_t dim,
+                    int32_t vdim, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot, int32_t T, int32_t chunked);
 int tgis_k_head_norm_gate(const float* o, int32_t ldo, int32_t heads, int32_t vdim, const float* w, const float* gate, int32_t ldg,
                           int32_t act, float eps, void* out, int32_t out_dt, int32_t T);
 /* resid += rmsnorm((rmsnorm(y_main) * w_main + rmsnorm(y_pair) * w_pair) / 2) * w_post; out = rmsnorm(resid) * w_pre, or the

@@ -23,7 +23,7 @@ class LiveServer:
         from vllm_tgis_adapter_b200.engine.tokenizer import build_synthetic_tokenizer
         from vllm_tgis_adapter_b200.grpc import grpc_server
 
-        if cfg_name.startswith(("revepel-", "sikazen-", "bisuzen-")):   # layer-list families (tests/test_zz_<family>_gpu.py): preset sizes, seeded CPU weights, fp32
+        if cfg_name.startswith(("revepel-", "sikazen-", "bisuzen-", "ludelix-")):   # layer-list families (tests/test_zz_<family>_gpu.py): preset sizes, seeded CPU weights, fp32
             import dataclasses
             import importlib
             import types

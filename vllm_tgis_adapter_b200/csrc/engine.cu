@@ -1446,7 +1446,10 @@ struct tgis_engine {
           l.o_cols = up8((int)hv);
           pnx_expected_tensors += 9;  // q, k, v, g, o, norm, a1, a2, a2.b
           m_f1 = std::max(m_f1, hv); m_f2 = std::max(m_f2, hd);
-          m_mix = std::max(m_mix, 2 * hd + hv);
+          if (pnx_dt == DT_BF16 && gla_chunk_eligible(s.dim, s.vdim, s.decay_rank)) {
+            m_mix = std::max(m_mix, (size_t)H * gla_row(s.dim) + hv);
+            m_f3 = std::max(m_f3, hd);
+          }
         } else {
           const bool par = s.mixer == TGIS_MIXER_CHUNK_RETENTION, shared_kv = (s.flags & TGIS_LAYER_SHARED_KV) != 0;
           l.c_q = cols(H * s.dim); l.c_k = cols(G * s.dim);
@@ -2861,7 +2864,18 @@ struct tgis_engine {
     pnx_gemm(pnx_hA, A, W, l.w_in, pnx_y1, DT_F32, ld, T, ld, W);
     if (s.mixer == TGIS_MIXER_GLA) {
       const int hd = s.heads * s.dim;
-      pnx_gemm(pnx_y1 + l.c_a1, DT_F32, ld, l.w_w2, flx_f2, DT_F32, hd, T, hd, s.decay_rank);
+      // bf16 portions: chunk by chunk on the tensor cores; single tokens (the step's first sequences) and fp32: token by token
+      const int lead = step_n_lead1;
+      const bool chunked = A == DT_BF16 && lead < S && gla_chunk_eligible(s.dim, s.vdim, s.decay_rank) && l.c_v % 2 == 0;
+      const int n_scan = chunked ? lead : T;   // rows of the scan
+      if (n_scan > 0) pnx_gemm(pnx_y1 + l.c_a1, DT_F32, ld, l.w_w2, flx_f2, DT_F32, hd, n_scan, hd, s.decay_rank);
+      if (chunked) {
+        GlaChunk gc{pnx_y1 + l.c_q, pnx_y1 + l.c_k, pnx_y1 + l.c_v, pnx_y1 + l.c_a1, ld, 1.f / sqrtf((float)s.dim), l.w_w2, s.decay_rank, l.w0,
+                    1.f / s.tau, flx_mix, reinterpret_cast<bf16*>(flx_mix) + pnx_rows_alloc * s.heads * gla_row(s.dim), flx_f3, l.st_S, flx_f1, hv,
+                    s.heads, s.dim, s.vdim};
+        CK(gla_chunk_launch(gc, d_seqs, lead, S, ds<LatentTile>(off_ltiles16), step_n_ltiles16, d_tokslot, stream));
+        n_launches += 2;
+      }
       OuterScan os{};
       os.mode = OUTER_SCAN_GLA;
       os.q = pnx_y1 + l.c_q; os.k = pnx_y1 + l.c_k; os.v = pnx_y1 + l.c_v; os.ldq = os.ldk = os.ldv = ld;
@@ -2870,10 +2884,10 @@ struct tgis_engine {
       os.S = l.st_S;
       os.out = flx_f1; os.ldo = hv;
       os.heads = s.heads; os.dim = s.dim; os.vdim = s.vdim;
-      CK(outer_scan_launch(os, d_seqs, S, d_tokslot, stream));
+      if (n_scan > 0) CK(outer_scan_launch(os, d_seqs, chunked ? lead : S, d_tokslot, stream));
       CK(head_norm_gate_launch(flx_f1, hv, s.heads, s.vdim, l.mm_norm, pnx_y1 + l.c_mg, ld, /*silu*/ 1, eps, pnx_oA, A, T, stream, 0, 1.f,
                                l.o_cols));
-      n_launches += 2;
+      n_launches += n_scan > 0 ? 2 : 1;
     } else {
       const bool par = s.mixer == TGIS_MIXER_CHUNK_RETENTION;
       auto retention = [&](cudaStream_t st) {   // -> columns [c_o2, ..) of pnx_oA

@@ -563,6 +563,24 @@ struct RotaryRows {
 };
 cudaError_t rotary_rows_launch(const RotaryRows& a, int T, cudaStream_t stream);
 cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs, int n_seqs, const int32_t* tok_slot, cudaStream_t stream);
+// Gated linear attention (OUTER_SCAN_GLA) over whole portions, GLA_CHUNK tokens at a time on the tensor cores.  The decay logits are
+// the low-rank map's second product, a2 a1 + bias, made inside.
+constexpr int GLA_CHUNK = 32;
+struct GlaChunk {
+  const float *q, *k, *v, *a1; int ld;            // fp32 [T, ld]: q, k [heads * dim], v [heads * vdim], a1 [rank]
+  float q_scale;
+  const void* a2; int rank; const float* bias;    // bf16 [heads * dim, rank]; fp32 [heads * dim]
+  float inv_tau;
+  void *ops, *vb; float* chunk_decay;             // scratch: bf16 [T][heads][gla_row(dim)], bf16 [T][heads * vdim], fp32 [T][heads * dim]
+  float* S;                                       // [slots][heads][dim][vdim]
+  float* out; int ldo;                            // fp32 [T, heads * vdim]
+  int heads, dim, vdim;
+};
+__host__ __device__ constexpr int gla_row(int dim) { return 4 * dim + 2 * GLA_CHUNK; }
+bool gla_chunk_eligible(int dim, int vdim, int rank);
+// sequences [first_seq, n_seqs) of the step; tiles: the step's 16-token query tiles
+cudaError_t gla_chunk_launch(const GlaChunk& a, const AttnSeq* seqs, int first_seq, int n_seqs, const LatentTile* tiles, int n_tiles,
+                             const int32_t* tok_slot, cudaStream_t stream);
 // out[t, h, :] = rmsnorm(o[t, h, :]) * w[h, :] * act(gate[t, h, :])    act: 0 sigmoid, 1 silu, 2 none (gate may be nullptr)
 // gate_first != 0: out[t, h, :] = rmsnorm(o[t, h, :] * act(gate[t, h, :])) * w[h, :]   (the gate enters the norm)
 // w == nullptr: no weight; mult multiplies every output; out rows are out_ld elements apart (0: heads * vdim)

@@ -1,4 +1,5 @@
-// Lightning attention over the portions of a step, chunk by chunk on the tensor cores (kernels.h: LightningChunk).
+// Outer-product memories over the portions of a step, chunk by chunk on the tensor cores: lightning attention and retention (kernels.h:
+// LightningChunk) here, gated linear attention (GlaChunk) further down.
 // Per head  S_t = r S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t  with one fixed decay r and q, k, v = silu of their projections
 // (lightning attention), or q and k rotated by their position and v as projected (retention).  For the n <= 64
 // tokens i, j = 0 .. n-1 of a chunk and the state S that the tokens before it left, this is
@@ -330,6 +331,427 @@ cudaError_t launch_chunks(const LightningChunk& a, const AttnSeq* seqs, int n_se
   return launch_k(lightning_chunk_kernel<DKS>, dim3(n_seqs, a.heads, (a.vdim + LV - 1) / LV), dim3(L_THREADS), smem, stream, a, seqs, tok_slot);
 }
 
+// ---------------------------------------------------------------------------------------------------------------- gated linear attention
+// Per head  S_t = diag(f_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t  with a decay f_t per key channel (kernels.h: GlaChunk).  For the n <= GC
+// tokens of a chunk, with F(j, i] the product of f over the tokens j + 1 .. i (per channel) and S what the tokens before left,
+//     o_i = (q_i F(-1, i])^T S + sum_{j <= i} A_ij v_j,   A_ij = sum_c q_ic k_jc F(j, i]_c
+//     S  <- diag(F(-1, n - 1]) S + sum_j (k_j F(j, n - 1]) v_j^T
+// Every factor is a product of decays over an INTERVAL: nothing is ever divided by a decay, so strong decays cannot overflow.  Two
+// kernels:
+//   gla_prep_kernel   all chunks of the step at once: decays from their low-rank map, prefix and suffix products, the decayed queries
+//                     and keys, and the chunk's scores A -- inside 16-token blocks by running products in fp32 (a lane owns channels,
+//                     32 scores are reduced over the lanes together), between the two blocks as a product of operands decayed to the
+//                     border between them
+//   gla_chunk_kernel  the recurrence over a portion's chunks, as lightning_chunk_kernel: a warp owns 16 value columns and keeps the
+//                     transposed state in accumulator fragments
+// What carries decays goes into products as the sum of two bf16 numbers; v is rounded to bf16 once, q and k are not rounded.
+constexpr int GC = GLA_CHUNK, GB = 16, G_THREADS = 128;
+static_assert(GC == 2 * GB, "one off-diagonal block per chunk");
+constexpr int LDGA = GC + 8;
+
+__device__ __forceinline__ float l_logsigmoid(float z) { return z >= 0.f ? -log1pf(expf(-z)) : z - log1pf(expf(z)); }
+
+// lane l leaves with the sum over all lanes of v[l]
+__device__ __forceinline__ float reduce32(float (&v)[32], int lane) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const bool up = (lane & o) != 0;
+#pragma unroll
+    for (int n = 0; n < o; ++n) {
+      const float keep = up ? v[n + o] : v[n], send = up ? v[n] : v[n + o];
+      v[n] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+    }
+  }
+  return v[0];
+}
+template <int DPL>
+__device__ __forceinline__ void ld_row(float (&r)[DPL], const float* p, bool live) {
+  if (DPL == 4) {
+    const float4 x = live ? *reinterpret_cast<const float4*>(p) : make_float4(0.f, 0.f, 0.f, 0.f);
+    r[0] = x.x; r[1] = x.y; r[2 % DPL] = x.z; r[3 % DPL] = x.w;
+  } else {
+    const float2 x = live ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
+    r[0] = x.x; r[1] = x.y;
+  }
+}
+// scores of rows [I0, I1) of one 16-token block: pair p = i (i + 1) / 2 + delta is A[i][i - delta]; rows of q / k / f are ldf floats apart
+template <int I0, int I1, int DPL>
+__device__ __forceinline__ void gla_block_scores(const float* q, const float* k, const float* f, int ldf, float* A, int lda, int D, int lane) {
+  float kr[I1][DPL], fr[I1][DPL];
+  const bool live = lane * DPL < D;
+#pragma unroll
+  for (int j = 0; j < I1; ++j) {
+    ld_row<DPL>(kr[j], k + j * ldf + lane * DPL, live);
+    ld_row<DPL>(fr[j], f + j * ldf + lane * DPL, live);
+  }
+  constexpr int P0 = I0 * (I0 + 1) / 2, P1 = I1 * (I1 + 1) / 2;
+  float v[32];
+#pragma unroll
+  for (int i = I0; i < I1; ++i) {
+    float cur[DPL];
+    ld_row<DPL>(cur, q + i * ldf + lane * DPL, live);
+#pragma unroll
+    for (int dl = 0; dl <= i; ++dl) {
+      const int p = i * (i + 1) / 2 + dl, n = (p - P0) & 31, j = i - dl;
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < DPL; ++e) {
+        s = fmaf(cur[e], kr[j][e], s);
+        cur[e] *= fr[j][e];
+      }
+      v[n] = s;
+      if (n == 31 || p == P1 - 1) {
+#pragma unroll
+        for (int z = 0; z < 32; ++z)
+          if (z > n) v[z] = 0.f;
+        const float tot = reduce32(v, lane);
+        const int mine = p - n + lane;   // the pair whose sum this lane holds
+        if (mine < P1) {
+          int r = 0;
+          while ((r + 1) * (r + 2) / 2 <= mine) ++r;
+          A[r * lda + r - (mine - r * (r + 1) / 2)] = tot;
+        }
+      }
+    }
+  }
+}
+
+// grid (16-token tiles, heads): the CTA of a tile whose first token opens a chunk of its portion takes the chunk's GC tokens
+template <int DPL>
+__global__ void __launch_bounds__(G_THREADS)
+gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* __restrict__ tiles, int first_seq) {
+  extern __shared__ __align__(16) uint8_t g_smem[];
+  griddep_launch();
+  griddep_wait();
+  const LatentTile tl = tiles[blockIdx.x];
+  if (tl.q0 % GC != 0 || tl.seq < first_seq) return;
+  const AttnSeq sq = seqs[tl.seq];
+  const int nt = min(GC, sq.q_len - tl.q0), row0 = sq.q_start + tl.q0, h = blockIdx.y;
+  const int D = a.dim, LD = D + 4, LDQ = D + 8, R = a.rank;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* fs = reinterpret_cast<float*>(g_smem);   // [GC][LD] decays (1 past the chunk)
+  float* qs = fs + GC * LD;                       // [GC][LD]
+  float* ks = qs + GC * LD;                       // [GC][LD]
+  float* As = ks + GC * LD;                       // [GC][GC + 1]
+  bf* qlh = reinterpret_cast<bf*>(As + GC * (GC + 1) + (GC * (GC + 1)) % 4);   // [GB][LDQ] second block's queries decayed from its start
+  bf* qll = qlh + GB * LDQ;
+  bf* klh = qll + GB * LDQ;                       // [GB][LDQ] first block's keys decayed to its end
+  bf* kll = klh + GB * LDQ;
+  float* a1s = reinterpret_cast<float*>(qlh);     // [GC][R], consumed before qlh is written
+  for (int i = tid; i < GC * R; i += G_THREADS) {
+    const int t = i / R;
+    a1s[i] = t < nt ? a.a1[(size_t)(row0 + t) * a.ld + i % R] : 0.f;
+  }
+  __syncthreads();
+  const int c2 = (tid & 63) * 2, half = tid >> 6;   // two channels; half 0: tokens 0..15 / queries, half 1: tokens 16..31 / keys
+  const bool ch_ok = c2 < D;
+  if (ch_ok) {
+    const size_t hc = (size_t)h * D + c2;
+    float z0[GB], z1[GB];
+    const float b0 = a.bias[hc], b1 = a.bias[hc + 1];
+#pragma unroll
+    for (int t = 0; t < GB; ++t) { z0[t] = b0; z1[t] = b1; }
+    const bf *w0 = reinterpret_cast<const bf*>(a.a2) + hc * R, *w1 = w0 + R;
+    for (int r = 0; r < R; ++r) {
+      const float x0 = __bfloat162float(w0[r]), x1 = __bfloat162float(w1[r]);
+#pragma unroll
+      for (int t = 0; t < GB; ++t) {
+        const float y = a1s[(half * GB + t) * R + r];
+        z0[t] = fmaf(y, x0, z0[t]);
+        z1[t] = fmaf(y, x1, z1[t]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < GB; ++t) {
+      const int tt = half * GB + t;
+      float2 f = make_float2(1.f, 1.f);
+      if (tt < nt) f = make_float2(expf(l_logsigmoid(z0[t]) * a.inv_tau), expf(l_logsigmoid(z1[t]) * a.inv_tau));
+      *reinterpret_cast<float2*>(fs + tt * LD + c2) = f;
+    }
+  }
+  __syncthreads();
+  const int W = gla_row(D);
+  bf* ops = reinterpret_cast<bf*>(a.ops);
+  auto put = [&](bf* hi, bf* lo, float x, float y) {
+    uint32_t ph, pl;
+    split2(x, y, ph, pl);
+    *reinterpret_cast<uint32_t*>(hi) = ph;
+    *reinterpret_cast<uint32_t*>(lo) = pl;
+  };
+  if (ch_ok && half == 0) {   // queries, forward
+    const float* src = a.q + (size_t)row0 * a.ld + (size_t)h * D + c2;
+    float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
+#pragma unroll 8
+    for (int t = 0; t < GC; ++t) {
+      float2 x = make_float2(0.f, 0.f);
+      if (t < nt) x = *reinterpret_cast<const float2*>(src + (size_t)t * a.ld);
+      x.x *= a.q_scale;
+      x.y *= a.q_scale;
+      *reinterpret_cast<float2*>(qs + t * LD + c2) = x;
+      const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
+      p0 *= f.x;
+      p1 *= f.y;
+      if (t >= GB) {
+        l0 *= f.x;
+        l1 *= f.y;
+        put(qlh + (t - GB) * LDQ + c2, qll + (t - GB) * LDQ + c2, x.x * l0, x.y * l1);
+      }
+      if (t < nt) {
+        bf* o = ops + ((size_t)(row0 + t) * a.heads + h) * W + c2;
+        put(o, o + D, x.x * p0, x.y * p1);
+      }
+    }
+    *reinterpret_cast<float2*>(a.chunk_decay + (size_t)row0 * a.heads * D + (size_t)h * D + c2) = make_float2(p0, p1);
+  } else if (ch_ok) {         // keys, backward
+    const float* src = a.k + (size_t)row0 * a.ld + (size_t)h * D + c2;
+    float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
+#pragma unroll 8
+    for (int t = GC - 1; t >= 0; --t) {
+      float2 x = make_float2(0.f, 0.f);
+      if (t < nt) x = *reinterpret_cast<const float2*>(src + (size_t)t * a.ld);
+      *reinterpret_cast<float2*>(ks + t * LD + c2) = x;
+      const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
+      if (t < nt) {
+        bf* o = ops + ((size_t)(row0 + t) * a.heads + h) * W + 2 * D + c2;
+        put(o, o + D, x.x * p0, x.y * p1);
+      }
+      p0 *= f.x;
+      p1 *= f.y;
+      if (t < GB) {
+        put(klh + t * LDQ + c2, kll + t * LDQ + c2, x.x * l0, x.y * l1);
+        l0 *= f.x;
+        l1 *= f.y;
+      }
+    }
+  }
+  for (int i = tid; i < nt * (a.vdim / 2); i += G_THREADS) {   // the values, rounded once
+    const int t = i / (a.vdim / 2), c = i % (a.vdim / 2) * 2;
+    const float2 x = *reinterpret_cast<const float2*>(a.v + (size_t)(row0 + t) * a.ld + (size_t)h * a.vdim + c);
+    *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf*>(a.vb) + (size_t)(row0 + t) * a.heads * a.vdim + (size_t)h * a.vdim + c) =
+        __floats2bfloat162_rn(x.x, x.y);
+  }
+  __syncthreads();
+  // ---- scores: warps 0 and 1 the first block (rows 0..10 | 11..15: as many pairs each), warps 2 and 3 the second
+  const int blk = warp >> 1, b0 = blk * GB;
+  if (b0 < nt) {
+    const float *qb = qs + b0 * LD, *kb = ks + b0 * LD, *fb = fs + b0 * LD;
+    float* Ab = As + b0 * (GC + 1) + b0;
+    if ((warp & 1) == 0) gla_block_scores<0, 11, DPL>(qb, kb, fb, LD, Ab, GC + 1, D, lane);
+    else gla_block_scores<11, 16, DPL>(qb, kb, fb, LD, Ab, GC + 1, D, lane);
+  }
+  if (warp < 2 && nt > GB) {   // second block's rows x first block's keys 8 warp .. 8 warp + 7
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k0 = 0; k0 < D; k0 += 16) {
+      uint32_t qh[4], ql[4], kh[4], kl[4];
+      const size_t qa = (size_t)(lane & 15) * LDQ + k0 + (lane >> 4) * 8, ka = (size_t)((lane >> 4) * 8 + (lane & 7)) * LDQ + k0 + ((lane >> 3) & 1) * 8;
+      l_ldsm_x4(qh, qlh + qa);
+      l_ldsm_x4(ql, qll + qa);
+      l_ldsm_x4(kh, klh + ka);
+      l_ldsm_x4(kl, kll + ka);
+      l_mma(s, qh, kh[2 * warp], kh[2 * warp + 1]);
+      l_mma(s, qh, kl[2 * warp], kl[2 * warp + 1]);
+      l_mma(s, ql, kh[2 * warp], kh[2 * warp + 1]);
+    }
+    const int g = lane >> 2, t2 = (lane & 3) * 2 + 8 * warp;
+    As[(GB + g) * (GC + 1) + t2] = s[0];
+    As[(GB + g) * (GC + 1) + t2 + 1] = s[1];
+    As[(GB + g + 8) * (GC + 1) + t2] = s[2];
+    As[(GB + g + 8) * (GC + 1) + t2 + 1] = s[3];
+  }
+  __syncthreads();
+  for (int i = tid; i < nt * (GC / 2); i += G_THREADS) {
+    const int t = i / (GC / 2), j = i % (GC / 2) * 2;
+    bf* o = ops + ((size_t)(row0 + t) * a.heads + h) * W + 4 * D + j;
+    put(o, o + GC, j <= t ? As[t * (GC + 1) + j] : 0.f, j + 1 <= t ? As[t * (GC + 1) + j + 1] : 0.f);
+  }
+}
+
+// grid (sequences, heads, 64-column slices), four warps of 16 value columns; DKS as above
+template <int DKS>
+__global__ void __launch_bounds__(L_THREADS)
+gla_chunk_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const int32_t* __restrict__ tok_slot) {
+  extern __shared__ __align__(16) uint8_t l_smem[];
+  const int D = a.dim, LDQ = D + 8, nks = D / 16, W = gla_row(D);
+  const int ring = GC * (4 * LDQ + LDV_ + 2 * LDGA);   // one buffer: Q hi | Q lo | K hi | K lo [GC][LDQ] each | V [GC][LDV_] | A hi | A lo [GC][LDGA]
+  bf* RB = reinterpret_cast<bf*>(l_smem);              // two of them
+  float* EB = reinterpret_cast<float*>(RB + 2 * ring); // [2][D] the chunk's whole decay
+  griddep_launch();
+  griddep_wait();
+  const AttnSeq sq = seqs[blockIdx.x];
+  const int h = blockIdx.y, c0 = blockIdx.z * LV;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gq = lane >> 2, t2 = (lane & 3) * 2;
+  const int slot = tok_slot[sq.q_start];
+  const bool fresh = sq.kv_len - sq.q_len == 0;
+  const int n_col = min(LV, a.vdim - c0);   // a multiple of 8
+  const bf* ops = reinterpret_cast<const bf*>(a.ops) + (size_t)h * W;
+  const bf* vb = reinterpret_cast<const bf*>(a.vb) + (size_t)h * a.vdim + c0;
+  auto fetch = [&](int t0, int buf) {   // rows up to the next multiple of 16 and columns past the slice are zeros
+    const int nt = min(GC, sq.q_len - t0), qv = D / 8, av = GC / 8, per = 4 * qv + 2 * av + LV / 8;
+    bf* B = RB + buf * ring;
+    for (int t = warp; t < (nt + 15) / 16 * 16; t += L_THREADS / 32) {
+      const size_t row = (size_t)(sq.q_start + t0 + t);
+      for (int e = lane; e < per; e += 32) {
+        bf* dst;
+        const bf* src;
+        bool ok = t < nt;
+        if (e < 4 * qv) {
+          const int m = e / qv, c = (e - m * qv) * 8;
+          dst = B + (size_t)(m * GC + t) * LDQ + c;
+          src = ops + row * a.heads * W + e * 8;
+        } else if (e < 4 * qv + 2 * av) {
+          const int x = e - 4 * qv, m = x / av, c = (x - m * av) * 8;
+          dst = B + GC * (4 * LDQ + LDV_) + (size_t)(m * GC + t) * LDGA + c;
+          src = ops + row * a.heads * W + e * 8;
+        } else {
+          const int c = (e - 4 * qv - 2 * av) * 8;
+          dst = B + GC * 4 * LDQ + (size_t)t * LDV_ + c;
+          src = vb + row * a.heads * a.vdim + c;
+          ok = ok && c < n_col;
+        }
+        if (ok) l_cp_async16(dst, src);
+        else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+      }
+    }
+    for (int e = tid; e < D / 4; e += L_THREADS) l_cp_async16(EB + buf * D + e * 4, a.chunk_decay + ((size_t)(sq.q_start + t0) * a.heads + h) * D + e * 4);
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  fetch(0, 0);
+  // S^T fragments: tile n holds rows (value columns) v0 + gq, v0 + gq + 8 and entries 8 n + t2, + 1 of dim
+  float S[2 * DKS][4];
+  const int v0 = warp * 16;
+  float* Sg = a.S + ((size_t)slot * a.heads + h) * D * a.vdim + c0;
+#pragma unroll
+  for (int n = 0; n < 2 * DKS; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int v = v0 + gq + (e >> 1) * 8, i = n * 8 + t2 + (e & 1);
+      S[n][e] = (!fresh && v < n_col && i < D) ? Sg[(size_t)i * a.vdim + v] : 0.f;
+    }
+  int buf = 0;
+  for (int t0 = 0; t0 < sq.q_len; t0 += GC, buf ^= 1) {
+    const int nt = min(GC, sq.q_len - t0), n_mt = (nt + 15) / 16;   // rows past nt inside the last 16 are zeros
+    asm volatile("cp.async.wait_group 0;\n" ::: "memory");
+    __syncthreads();   // the chunk has landed; the previous chunk's operands are consumed
+    if (t0 + GC < sq.q_len) fetch(t0 + GC, buf ^ 1);   // lands while this chunk is worked through
+    const bf *Qh = RB + buf * ring, *Ql = Qh + GC * LDQ, *Kh = Ql + GC * LDQ, *Kl = Kh + GC * LDQ, *Vs = Kl + GC * LDQ, *Ah = Vs + GC * LDV_,
+             *Al = Ah + GC * LDGA;
+    const float* E = EB + buf * D;
+    // ---- read-out of the warp's 16 value columns: decayed queries times the state, then the chunk's own tokens
+    float o[GC / 16][2][4];
+#pragma unroll
+    for (int mt = 0; mt < GC / 16; ++mt)
+#pragma unroll
+      for (int n = 0; n < 2; ++n) o[mt][n][0] = o[mt][n][1] = o[mt][n][2] = o[mt][n][3] = 0.f;
+    if (!fresh || t0 > 0) {
+#pragma unroll
+      for (int ks = 0; ks < DKS; ++ks)
+        if (ks < nks) {
+          uint32_t bh[2][2], bl[2][2];   // [value half][dim half of the k-step]
+#pragma unroll
+          for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int k = 0; k < 2; ++k) split2(S[2 * ks + k][2 * n], S[2 * ks + k][2 * n + 1], bh[n][k], bl[n][k]);
+#pragma unroll
+          for (int mt = 0; mt < GC / 16; ++mt)
+            if (mt < n_mt) {
+              uint32_t qh[4], ql[4];
+              const size_t at = (size_t)(mt * 16 + (lane & 15)) * LDQ + ks * 16 + (lane >> 4) * 8;
+              l_ldsm_x4(qh, Qh + at);
+              l_ldsm_x4(ql, Ql + at);
+#pragma unroll
+              for (int n = 0; n < 2; ++n) {
+                l_mma(o[mt][n], qh, bh[n][0], bh[n][1]);
+                l_mma(o[mt][n], qh, bl[n][0], bl[n][1]);
+                l_mma(o[mt][n], ql, bh[n][0], bh[n][1]);
+              }
+            }
+        }
+    }
+#pragma unroll
+    for (int kk = 0; kk < GC / 16; ++kk)
+      if (kk < n_mt) {
+        uint32_t vf[4];
+        l_ldsm_x4_trans(vf, Vs + (size_t)(kk * 16 + (lane & 15)) * LDV_ + v0 + (lane >> 4) * 8);
+#pragma unroll
+        for (int mt = kk; mt < GC / 16; ++mt)
+          if (mt < n_mt) {
+            uint32_t ah[4], al[4];
+            const size_t at = (size_t)(mt * 16 + (lane & 15)) * LDGA + kk * 16 + (lane >> 4) * 8;
+            l_ldsm_x4(ah, Ah + at);
+            l_ldsm_x4(al, Al + at);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+              l_mma(o[mt][n], ah, vf[2 * n], vf[2 * n + 1]);
+              l_mma(o[mt][n], al, vf[2 * n], vf[2 * n + 1]);
+            }
+          }
+      }
+#pragma unroll
+    for (int mt = 0; mt < GC / 16; ++mt)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const int t = mt * 16 + gq + r * 8;
+        if (t >= nt) continue;
+        float* dst = a.out + (size_t)(sq.q_start + t0 + t) * a.ldo + (size_t)h * a.vdim + c0 + v0 + t2;
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+          if (v0 + n * 8 < n_col) *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[mt][n][2 * r], o[mt][n][2 * r + 1]);
+      }
+    // ---- the state behind the chunk: its whole decay per channel, then V^T K
+#pragma unroll
+    for (int n = 0; n < 2 * DKS; ++n)
+      if (n < 2 * nks) {
+        const float2 f = *reinterpret_cast<const float2*>(E + n * 8 + t2);
+        S[n][0] *= f.x; S[n][1] *= f.y; S[n][2] *= f.x; S[n][3] *= f.y;
+      }
+#pragma unroll
+    for (int kk = 0; kk < GC / 16; ++kk)
+      if (kk < n_mt) {
+        uint32_t va[4];   // A fragments of V^T: rows = values, k = tokens
+        l_ldsm_x4_trans(va, Vs + (size_t)(kk * 16 + (lane & 7) + (lane >> 4) * 8) * LDV_ + v0 + ((lane >> 3) & 1) * 8);
+#pragma unroll
+        for (int ks = 0; ks < DKS; ++ks)
+          if (ks < nks) {
+            uint32_t kh[4], kl[4];
+            const size_t at = (size_t)(kk * 16 + (lane & 15)) * LDQ + ks * 16 + (lane >> 4) * 8;
+            l_ldsm_x4_trans(kh, Kh + at);
+            l_ldsm_x4_trans(kl, Kl + at);
+            l_mma(S[2 * ks], va, kh[0], kh[1]);
+            l_mma(S[2 * ks + 1], va, kh[2], kh[3]);
+            l_mma(S[2 * ks], va, kl[0], kl[1]);
+            l_mma(S[2 * ks + 1], va, kl[2], kl[3]);
+          }
+      }
+  }
+#pragma unroll
+  for (int n = 0; n < 2 * DKS; ++n)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int v = v0 + gq + (e >> 1) * 8, i = n * 8 + t2 + (e & 1);
+      if (v < n_col && i < D) Sg[(size_t)i * a.vdim + v] = S[n][e];
+    }
+}
+
+template <int DKS>
+cudaError_t launch_gla(const GlaChunk& a, const AttnSeq* seqs, int first_seq, int n_seqs, const LatentTile* tiles, int n_tiles,
+                       const int32_t* tok_slot, cudaStream_t stream) {
+  constexpr int DPL = DKS <= 4 ? 2 : 4;
+  const size_t tail = std::max((size_t)4 * GB * (a.dim + 8) * sizeof(bf), (size_t)GC * a.rank * sizeof(float));
+  const size_t smem_p = ((size_t)3 * GC * (a.dim + 4) + GC * (GC + 1)) * sizeof(float) + tail;                       // <= 73 KB
+  const size_t smem_c = (size_t)2 * GC * (4 * (a.dim + 8) + LDV_ + 2 * LDGA) * sizeof(bf) + (size_t)2 * a.dim * sizeof(float);   // <= 90 KB
+  static bool attr_set = false;
+  if (!attr_set) {
+    cudaError_t e = cudaFuncSetAttribute(gla_prep_kernel<DPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_chunk_kernel<DKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    if (e != cudaSuccess) return e;
+    attr_set = true;
+  }
+  const cudaError_t e = launch_k(gla_prep_kernel<DPL>, dim3(n_tiles, a.heads), dim3(G_THREADS), smem_p, stream, a, seqs, tiles, first_seq);
+  if (e != cudaSuccess) return e;
+  return launch_k(gla_chunk_kernel<DKS>, dim3(n_seqs - first_seq, a.heads, (a.vdim + LV - 1) / LV), dim3(L_THREADS), smem_c, stream, a, seqs + first_seq,
+                  tok_slot);
+}
+
 }  // namespace
 
 bool lightning_chunk_eligible(int dim, int vdim) {
@@ -362,6 +784,19 @@ cudaError_t lightning_chunk_launch(const LightningChunk& a, const AttnSeq* seqs,
       (reinterpret_cast<uintptr_t>(a.out) & 7) != 0)
     return cudaErrorInvalidValue;
   return a.dim <= 64 ? launch_chunks<4>(a, seqs, n_seqs, tok_slot, stream) : launch_chunks<8>(a, seqs, n_seqs, tok_slot, stream);
+}
+
+bool gla_chunk_eligible(int dim, int vdim, int rank) { return lightning_chunk_eligible(dim, vdim) && rank >= 1 && rank <= 64; }
+
+cudaError_t gla_chunk_launch(const GlaChunk& a, const AttnSeq* seqs, int first_seq, int n_seqs, const LatentTile* tiles, int n_tiles,
+                             const int32_t* tok_slot, cudaStream_t stream) {
+  if (n_seqs <= first_seq || n_tiles <= 0) return cudaSuccess;
+  auto al = [](const void* p, int n) { return (reinterpret_cast<uintptr_t>(p) & (n - 1)) == 0; };
+  if (!gla_chunk_eligible(a.dim, a.vdim, a.rank) || a.heads < 1 || a.heads > 65535 || a.ld % 2 != 0 || !al(a.q, 8) || !al(a.k, 8) || !al(a.v, 8) ||
+      !al(a.ops, 16) || !al(a.vb, 16) || !al(a.chunk_decay, 16) || !al(a.out, 8) || a.ldo % 2 != 0 || a.bias == nullptr || !(a.inv_tau > 0.f))
+    return cudaErrorInvalidValue;
+  return a.dim <= 64 ? launch_gla<4>(a, seqs, first_seq, n_seqs, tiles, n_tiles, tok_slot, stream)
+                     : launch_gla<8>(a, seqs, first_seq, n_seqs, tiles, n_tiles, tok_slot, stream);
 }
 
 }  // namespace tgis

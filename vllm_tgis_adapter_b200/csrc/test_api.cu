@@ -534,6 +534,17 @@ int tgis_k_rmsnorm_f32(const float* x, int32_t ldx, const float* w, float w_off,
   return 0;
 }
 
+int tgis_k_resid_tail_plain(const float* y_main, const float* y_rows, const int32_t* inv, float mix_const, int32_t top, const float* y_side,
+                            const float* side_gate, const float* w_pre, float* resid, void* out, int32_t out_dt, const float* w_dot,
+                            float* dot_out, float eps, int32_t T, int32_t hidden) {
+  ResidTail a{};
+  a.y_main = y_main; a.y_rows = y_rows; a.inv = inv; a.mix_const = mix_const; a.top = top; a.y_side = y_side; a.side_gate = side_gate;
+  a.w_pre = w_pre; a.resid = resid; a.out = out; a.out_dtype = out_dt; a.w_dot = w_dot; a.dot_out = dot_out;
+  a.mult = 1.f; a.eps = eps;
+  KCK(resid_tail_launch(a, T, hidden, 0));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
 int tgis_k_resid_tail(const float* y_main, const float* y_rows, const int32_t* inv, const float* mix_w, int32_t top,
                       const float* y_side, const float* side_gate, const float* w_post, const float* w_pre, float* resid,
                       void* out, int32_t out_dt, float mult, float w_off, float eps, int32_t T, int32_t hidden) {
@@ -621,6 +632,15 @@ int tgis_k_dyt_tail(const float* y_main, const float* b_main, const float* y_pai
   return 0;
 }
 
+int tgis_k_moe_table_align(const int32_t* table, int32_t vocab, const int32_t* tok, int32_t T, int32_t top, int32_t E, int32_t* seg_off,
+                           int32_t* order, int32_t* inv) {
+  const MoeTable h{table, seg_off, order, inv, E, top};
+  Tmp<MoeTable> d;
+  KCK(d.upload(&h, 1));
+  KCK(moe_table_align_launch(d.p, 1, E, tok, vocab, T, 0));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
 int tgis_k_moe_align(const int32_t* ids, int32_t T, int32_t top, int32_t E, int32_t* seg_off, int32_t* order, int32_t* inv) {
   KCK(moe_align_launch(ids, T, top, E, seg_off, order, inv, 0));
   KCK(cudaDeviceSynchronize());
@@ -695,8 +715,15 @@ int tgis_k_sigattn(const void* q, const void* k_cache, const void* v_cache, int3
 }
 
 static PoolAttnGeom to_pool(const tgis_k_poolattn_geom* g) {
-  return PoolAttnGeom{g->heads, g->kv_heads, g->dim, g->vdim, g->window, g->window > 0 ? g->pool : 0, g->rot_dims, g->scale, g->unit_norm,
-                      g->keep_first, g->chunk, g->rot_interleaved, g->sink};
+  PoolAttnGeom p{g->heads, g->kv_heads, g->dim, g->vdim, g->window, g->window > 0 ? g->pool : 0, g->rot_dims, g->scale, g->unit_norm,
+                 g->keep_first, g->chunk, g->rot_interleaved, g->sink};
+  p.head_gate = g->head_gate;
+  p.gate_ld = g->gate_ld;
+  p.out_ld = g->out_ld;
+  p.out_mul = g->out_mul != 0.f ? g->out_mul : 1.f;
+  p.q_norm = g->q_norm;
+  p.k_norm = g->k_norm;
+  return p;
 }
 
 int tgis_k_poolattn_prep(const float* y, int32_t ldy, int32_t q_off, int32_t k_off, int32_t v_off, const float* bias,
@@ -849,6 +876,67 @@ int tgis_k_lightning_scan(const float* q, const float* k, const float* v, int32_
   return 0;
 }
 
+int tgis_k_retention_scan(float* x, int32_t ld, int32_t q_off, int32_t k_off, int32_t v_off, const float* cos_sin, const int32_t* positions,
+                          int32_t rot_dims, float k_mul, const float* decay, float* S, float* out, int32_t ldo, int32_t heads, int32_t dim,
+                          int32_t vdim, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot, int32_t T, int32_t chunked) {
+  std::vector<AttnSeq> seqs;
+  host_seqs(seqs_host, n_seqs, seqs);
+  Tmp<AttnSeq> d_seqs;
+  KCK(d_seqs.upload(seqs.data(), seqs.size()));
+  const int hd = heads * dim, hv = heads * vdim, n = 2 * hd + hv;
+  Tmp<__nv_bfloat16> qkv;
+  KCK(qkv.alloc((size_t)T * n));
+  KCK(rotary_rows_launch(RotaryRows{x, ld, q_off, k_off, v_off, heads, dim, vdim, rot_dims, 1.f, k_mul, cos_sin, positions,
+                                    chunked ? qkv.p : nullptr, n, 0}, T, 0));
+  if (chunked) {
+    KCK(lightning_chunk_launch(LightningChunk{qkv.p, n, 0, hd, 2 * hd, decay, S, out, ldo, heads, dim, vdim}, d_seqs.p, n_seqs, tok_slot, 0));
+  } else {
+    OuterScan a{};
+    a.mode = OUTER_SCAN_RETENTION;
+    a.q = x + q_off; a.k = x + k_off; a.v = x + v_off; a.ldq = a.ldk = a.ldv = ld; a.q_scale = 1.f;
+    a.decay = decay; a.S = S; a.out = out; a.ldo = ldo; a.heads = heads; a.dim = dim; a.vdim = vdim;
+    KCK(outer_scan_launch(a, d_seqs.p, n_seqs, tok_slot, 0));
+  }
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
+int tgis_k_gla_scan(const float* x, int32_t ld, int32_t q_off, int32_t k_off, int32_t v_off, int32_t a1_off, float q_scale, const void* a2,
+                    int32_t rank, const float* bias, float inv_tau, float* S, float* out, int32_t ldo, int32_t heads, int32_t dim,
+                    int32_t vdim, const int32_t* seqs_host, int32_t n_seqs, const int32_t* tok_slot, int32_t T, int32_t chunked) {
+  std::vector<AttnSeq> seqs;
+  host_seqs(seqs_host, n_seqs, seqs);
+  Tmp<AttnSeq> d_seqs;
+  KCK(d_seqs.upload(seqs.data(), seqs.size()));
+  const int hd = heads * dim, hv = heads * vdim;
+  Tmp<float> z;
+  KCK(z.alloc((size_t)T * hd));
+  if (chunked) {
+    std::vector<LatentTile> tiles;
+    for (int i = 0; i < n_seqs; ++i)
+      for (int q0 = 0; q0 < seqs[i].q_len; q0 += POOLATTN_TILE) tiles.push_back(LatentTile{i, q0, std::min(POOLATTN_TILE, seqs[i].q_len - q0), 0});
+    Tmp<LatentTile> d_tiles;
+    Tmp<__nv_bfloat16> ops, vb;
+    KCK(d_tiles.upload(tiles.data(), tiles.size()));
+    KCK(ops.alloc((size_t)T * heads * gla_row(dim)));
+    KCK(vb.alloc((size_t)T * hv));
+    const GlaChunk a{x + q_off, x + k_off, x + v_off, x + a1_off, ld, q_scale, a2, rank, bias, inv_tau, ops.p, vb.p, z.p, S, out, ldo, heads, dim, vdim};
+    KCK(gla_chunk_launch(a, d_seqs.p, 0, n_seqs, d_tiles.p, (int)tiles.size(), tok_slot, 0));
+    KCK(cudaDeviceSynchronize());
+    return 0;
+  }
+  GemmAny g{};
+  g.X = x + a1_off; g.W = a2; g.Y = z.p; g.x_dtype = DT_F32; g.w_dtype = DT_BF16; g.y_dtype = DT_F32;
+  g.T = T; g.N = hd; g.K = rank; g.ldx = ld; g.ldw = rank; g.ldy = hd; g.batch = 1;
+  KCK(gemm_any_launch(g, 0));
+  OuterScan a{};
+  a.mode = OUTER_SCAN_GLA;
+  a.q = x + q_off; a.k = x + k_off; a.v = x + v_off; a.ldq = a.ldk = a.ldv = ld; a.q_scale = q_scale;
+  a.decay_raw = z.p; a.ldd = hd; a.w0 = bias; a.inv_tau = inv_tau;
+  a.S = S; a.out = out; a.ldo = ldo; a.heads = heads; a.dim = dim; a.vdim = vdim;
+  KCK(outer_scan_launch(a, d_seqs.p, n_seqs, tok_slot, 0));
+  KCK(cudaDeviceSynchronize());
+  return 0;
+}
 int tgis_k_head_norm_gate(const float* o, int32_t ldo, int32_t heads, int32_t vdim, const float* w, const float* gate, int32_t ldg,
                           int32_t act, float eps, void* out, int32_t out_dt, int32_t T) {
   KCK(head_norm_gate_launch(o, ldo, heads, vdim, w, gate, ldg, act, eps, out, out_dt, T, 0));

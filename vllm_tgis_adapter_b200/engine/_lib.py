@@ -87,6 +87,8 @@ class TgisKPoolAttnGeom(C.Structure):
         ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("window", C.c_int32),
         ("pool", C.c_int32), ("rot_dims", C.c_int32), ("scale", C.c_float), ("unit_norm", C.c_int32),
         ("keep_first", C.c_int32), ("chunk", C.c_int32), ("rot_interleaved", C.c_int32), ("sink", C.c_void_p),
+        ("head_gate", C.c_void_p), ("gate_ld", C.c_int32), ("out_ld", C.c_int32), ("out_mul", C.c_float), ("reserved", C.c_int32),
+        ("q_norm", C.c_void_p), ("k_norm", C.c_void_p),
     ]
 
 
@@ -150,7 +152,7 @@ ENGINE_SYMBOLS = [
 KERNEL_SYMBOLS = [
     "tgis_k_last_error", "tgis_k_gemm_timeline", "tgis_k_step_timeline_enable", "tgis_k_step_timeline_read", "tgis_k_gemm", "tgis_k_rmsnorm", "tgis_k_opt_layernorm", "tgis_k_opt_bias_act", "tgis_k_opt_embed", "tgis_k_silu_mul", "tgis_k_rope_kv", "tgis_k_gemm_rope", "tgis_k_gemm_norm_chain", "tgis_k_attention",
     "tgis_k_attention_bench", "tgis_k_decode_items", "tgis_k_gemm_plan", "tgis_k_gemm_unit_rows",
-    "tgis_k_sampler", "tgis_k_sampler_ex", "tgis_k_sampler_masked", "tgis_k_lora", "tgis_k_lora_bench", "tgis_k_silu_mul_interleaved", "tgis_k_gemm_any", "tgis_k_rmsnorm_f32", "tgis_k_resid_tail", "tgis_k_latent_prep", "tgis_k_latent_q_rope", "tgis_k_latent_attn", "tgis_k_moe_route", "tgis_k_moe_align", "tgis_k_moe_route_grouped", "tgis_k_dyt_tail", "tgis_k_lightning_scan", "tgis_k_capattn_prep", "tgis_k_capattn", "tgis_k_sigattn_prep", "tgis_k_sigattn", "tgis_k_poolattn_prep", "tgis_k_poolattn", "tgis_k_delta_scan", "tgis_k_ssd_scan", "tgis_k_token_shift", "tgis_k_short_conv", "tgis_k_selective_scan", "tgis_k_outer_scan", "tgis_k_head_norm_gate", "tgis_k_resid_tail_pair", "tgis_k_sizeof_sample_row", "tgis_k_sizeof_sample_out", "tgis_k_kv_block",
+    "tgis_k_sampler", "tgis_k_sampler_ex", "tgis_k_sampler_masked", "tgis_k_lora", "tgis_k_lora_bench", "tgis_k_silu_mul_interleaved", "tgis_k_gemm_any", "tgis_k_rmsnorm_f32", "tgis_k_resid_tail", "tgis_k_latent_prep", "tgis_k_latent_q_rope", "tgis_k_latent_attn", "tgis_k_moe_route", "tgis_k_moe_align", "tgis_k_moe_route_grouped", "tgis_k_dyt_tail", "tgis_k_lightning_scan", "tgis_k_retention_scan", "tgis_k_gla_scan", "tgis_k_moe_table_align", "tgis_k_resid_tail_plain", "tgis_k_capattn_prep", "tgis_k_capattn", "tgis_k_sigattn_prep", "tgis_k_sigattn", "tgis_k_poolattn_prep", "tgis_k_poolattn", "tgis_k_delta_scan", "tgis_k_ssd_scan", "tgis_k_token_shift", "tgis_k_short_conv", "tgis_k_selective_scan", "tgis_k_outer_scan", "tgis_k_head_norm_gate", "tgis_k_resid_tail_pair", "tgis_k_sizeof_sample_row", "tgis_k_sizeof_sample_out", "tgis_k_kv_block",
 ]
 
 _LIB: C.CDLL | None = None
@@ -247,6 +249,10 @@ def load_library() -> C.CDLL:
     lib.tgis_k_outer_scan.argtypes = [i32, vp, vp, vp, i32, i32, i32, f32, vp, i32, vp, vp, vp, vp, i32, vp, vp, f32, vp, vp, vp,
                                       vp, i32, i32, i32, i32, vp, vp, i32, ip, i32, vp]
     lib.tgis_k_lightning_scan.argtypes = [vp, vp, vp, i32, i32, i32, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp, i32]
+    lib.tgis_k_retention_scan.argtypes = [vp, i32, i32, i32, i32, vp, vp, i32, f32, vp, vp, vp, i32, i32, i32, i32, ip, i32, vp, i32, i32]
+    lib.tgis_k_gla_scan.argtypes = [vp, i32, i32, i32, i32, i32, f32, vp, i32, vp, f32, vp, vp, i32, i32, i32, i32, ip, i32, vp, i32, i32]
+    lib.tgis_k_moe_table_align.argtypes = [vp, i32, vp, i32, i32, i32, vp, vp, vp]
+    lib.tgis_k_resid_tail_plain.argtypes = [vp, vp, vp, f32, i32, vp, vp, vp, vp, vp, i32, vp, vp, f32, i32, i32]
     lib.tgis_k_head_norm_gate.argtypes = [vp, i32, i32, i32, vp, vp, i32, i32, f32, vp, i32, i32]
     lib.tgis_k_resid_tail_pair.argtypes = [vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, f32, i32, i32]
     _LIB = lib
