@@ -201,6 +201,88 @@ poolattn_prep_full_kernel(const float* __restrict__ y, int ldy, int q_off, int k
   }
 }
 
+// poolattn_prep_full_kernel for interleaved pairs (or none) with shared keys and values, sizes that are multiples of four and rows
+// on 16-byte boundaries: two pairs per thread and step, kept in registers between the passes
+constexpr int PREPF_V = 4;   // (heads + kv_heads) * dim <= 4 PREPF_THREADS PREPF_V
+template <class CT>
+__device__ __forceinline__ void st4(CT* p, float4 v);
+template <>
+__device__ __forceinline__ void st4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <>
+__device__ __forceinline__ void st4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+  pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+template <class CT>
+__global__ void __launch_bounds__(PREPF_THREADS)
+poolattn_prep_full_vec_kernel(const float* __restrict__ y, int ldy, int q_off, int k_off, const float* __restrict__ bias, PoolAttnGeom g,
+                              const float* __restrict__ cos_sin, float eps, const int32_t* __restrict__ positions,
+                              const int32_t* __restrict__ slot_mapping, CT* __restrict__ q_out, CT* __restrict__ k_cache,
+                              CT* __restrict__ v_cache) {
+  __shared__ float red[2][PREPF_THREADS / 32];
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x, tid = threadIdx.x, slot = slot_mapping[t];
+  const int nq = g.heads * g.dim, nk = g.kv_heads * g.dim;
+  const float* src = y + (size_t)t * ldy;
+  float4 v[PREPF_V];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int e = 0; e < PREPF_V; ++e) {
+    const int i = (e * PREPF_THREADS + tid) * 4;
+    v[e] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < nq + nk) {
+      v[e] = *reinterpret_cast<const float4*>(src + (i < nq ? q_off + i : k_off + i - nq));
+      if (bias != nullptr) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + i);
+        v[e].x += b.x; v[e].y += b.y; v[e].z += b.z; v[e].w += b.w;
+      }
+    }
+    const float s = fmaf(v[e].x, v[e].x, fmaf(v[e].y, v[e].y, fmaf(v[e].z, v[e].z, v[e].w * v[e].w)));
+    if (i < nq) sq += s;
+    else sk += s;
+  }
+  sq = warp_sum_f(sq);
+  sk = warp_sum_f(sk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = sq;
+    red[1][tid >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int w = 0; w < PREPF_THREADS / 32; ++w) {   // the same order in every thread
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float rq = 1.f / sqrtf(sq / (float)nq + eps), rk = 1.f / sqrtf(sk / (float)nk + eps);
+  const float* cs = cos_sin != nullptr ? cos_sin + (size_t)positions[t] * g.rot_dims : nullptr;
+  const int half = g.rot_dims / 2;
+#pragma unroll
+  for (int e = 0; e < PREPF_V; ++e) {
+    const int i = (e * PREPF_THREADS + tid) * 4;
+    const bool is_q = i < nq;
+    if (i >= nq + nk || (!is_q && slot < 0)) break;
+    const float4 w = *reinterpret_cast<const float4*>(is_q ? g.q_norm + i : g.k_norm + i - nq);
+    const float rs = is_q ? rq : rk;
+    const int d = (is_q ? i : i - nq) % g.dim;
+    float4 x = make_float4(v[e].x * rs * w.x, v[e].y * rs * w.y, v[e].z * rs * w.z, v[e].w * rs * w.w);
+    if (d < g.rot_dims) {
+      const float2 c = *reinterpret_cast<const float2*>(cs + d / 2), s = *reinterpret_cast<const float2*>(cs + half + d / 2);
+      x = make_float4(x.x * c.x - x.y * s.x, x.y * c.x + x.x * s.x, x.z * c.y - x.w * s.y, x.w * c.y + x.z * s.y);
+    }
+    if (is_q) {
+      st4(q_out + (size_t)t * nq + i, x);
+    } else {
+      st4(k_cache + (size_t)slot * nk + i - nq, x);
+      st4(v_cache + (size_t)slot * nk + i - nq, v[e]);
+    }
+  }
+}
+
 // ---------------------------------------------------------------------------------------------------------------- pool
 // grid (sequences, blocks per sequence in strides of gridDim.y), 128 threads over the columns of a K | V row
 template <class CT>
@@ -773,6 +855,16 @@ cudaError_t poolattn_prep_launch(const float* y, int ldy, int q_off, int k_off, 
   using bf = __nv_bfloat16;
   if (g.q_norm != nullptr || g.k_norm != nullptr) {
     if (g.q_norm == nullptr || g.k_norm == nullptr || g.unit_norm) return cudaErrorInvalidValue;
+    auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+    if (v_off == k_off && (g.rot_interleaved || g.rot_dims == 0) && g.dim % 4 == 0 && g.rot_dims % 4 == 0 && ldy % 4 == 0 && q_off % 4 == 0 &&
+        k_off % 4 == 0 && (g.heads + g.kv_heads) * g.dim <= 4 * PREPF_THREADS * PREPF_V && al16(y) && al16(bias) && al16(g.q_norm) &&
+        al16(g.k_norm) && al16(cos_sin) && al16(q_out) && al16(k_cache) && al16(v_cache)) {
+      if (dtype == DT_BF16)
+        return launch_k(poolattn_prep_full_vec_kernel<bf>, dim3(T), dim3(PREPF_THREADS), 0, stream, y, ldy, q_off, k_off, bias, g, cos_sin, eps,
+                        positions, slot_mapping, reinterpret_cast<bf*>(q_out), reinterpret_cast<bf*>(k_cache), reinterpret_cast<bf*>(v_cache));
+      return launch_k(poolattn_prep_full_vec_kernel<float>, dim3(T), dim3(PREPF_THREADS), 0, stream, y, ldy, q_off, k_off, bias, g, cos_sin, eps,
+                      positions, slot_mapping, reinterpret_cast<float*>(q_out), reinterpret_cast<float*>(k_cache), reinterpret_cast<float*>(v_cache));
+    }
     const size_t smem = (size_t)(g.heads + g.kv_heads) * g.dim * sizeof(float);
     if (smem > 160 * 1024) return cudaErrorInvalidValue;
     static bool attr_set = false;

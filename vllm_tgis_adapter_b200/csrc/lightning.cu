@@ -83,6 +83,54 @@ silu_cast_kernel(const float* __restrict__ x, int ldx, bf* __restrict__ out, int
   }
 }
 
+// rotary_rows_kernel for heads whose sizes are multiples of eight and rows on 16-byte boundaries: four pairs (or eight entries that pass)
+// per thread and step
+__global__ void __launch_bounds__(256)
+rotary_rows_vec_kernel(RotaryRows a) {
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x, D = a.dim, half = a.rot_dims / 2, hd = a.heads * D, per = D / 8;
+  float* row = a.x + (size_t)t * a.ld;
+  const float* cs = a.cos_sin != nullptr ? a.cos_sin + (size_t)a.positions[t] * a.rot_dims : nullptr;
+  bf* dst = (a.cast != nullptr && t >= a.n_inplace) ? reinterpret_cast<bf*>(a.cast) + (size_t)t * a.cast_ld : nullptr;
+  const int n_v = dst != nullptr ? a.heads * a.vdim / 8 : 0;
+  auto put = [&](float* f, bf* b, float4 v) {
+    if (b == nullptr) {
+      *reinterpret_cast<float4*>(f) = v;
+    } else {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+      uint2 pk;
+      pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+      pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>(b) = pk;
+    }
+  };
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < 2 * a.heads * per + n_v; i += gridDim.y * 256) {
+    if (i >= 2 * a.heads * per) {   // values
+      const int c = (i - 2 * a.heads * per) * 8;
+      put(nullptr, dst + 2 * hd + c, *reinterpret_cast<const float4*>(row + a.v_off + c));
+      put(nullptr, dst + 2 * hd + c + 4, *reinterpret_cast<const float4*>(row + a.v_off + c + 4));
+      continue;
+    }
+    const bool is_k = i >= a.heads * per;
+    const int r = is_k ? i - a.heads * per : i, h = r / per, e = r % per;
+    const float m = is_k ? a.k_mul : a.q_mul;
+    const bool turn = e * 4 < half;
+    const int p0 = turn ? e * 4 : a.rot_dims + (e * 4 - half) * 2, p1 = turn ? p0 + half : p0 + 4;
+    float* src = row + (is_k ? a.k_off : a.q_off) + h * D;
+    bf* out = dst != nullptr ? dst + (is_k ? hd : 0) + h * D : nullptr;
+    float4 u = *reinterpret_cast<const float4*>(src + p0), v = *reinterpret_cast<const float4*>(src + p1);
+    if (turn) {
+      const float4 c = *reinterpret_cast<const float4*>(cs + p0), s = *reinterpret_cast<const float4*>(cs + half + p0);
+      const float4 u2 = make_float4(u.x * c.x - v.x * s.x, u.y * c.y - v.y * s.y, u.z * c.z - v.z * s.z, u.w * c.w - v.w * s.w);
+      v = make_float4(v.x * c.x + u.x * s.x, v.y * c.y + u.y * s.y, v.z * c.z + u.z * s.z, v.w * c.w + u.w * s.w);
+      u = u2;
+    }
+    put(src + p0, out != nullptr ? out + p0 : nullptr, make_float4(u.x * m, u.y * m, u.z * m, u.w * m));
+    put(src + p1, out != nullptr ? out + p1 : nullptr, make_float4(v.x * m, v.y * m, v.z * m, v.w * m));
+  }
+}
+
 // grid (T, y): one token per x; pairs / values of the row in strides of the CTA (kernels.h: RotaryRows)
 __global__ void __launch_bounds__(256)
 rotary_rows_kernel(RotaryRows a) {
@@ -442,9 +490,15 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
     const int t = i / R;
     a1s[i] = t < nt ? a.a1[(size_t)(row0 + t) * a.ld + i % R] : 0.f;
   }
-  __syncthreads();
   const int c2 = (tid & 63) * 2, half = tid >> 6;   // two channels; half 0: tokens 0..15 / queries, half 1: tokens 16..31 / keys
   const bool ch_ok = c2 < D;
+  float2 xr[GC];   // this thread's two channels of the chunk's queries or keys: on their way while the decays are made
+  {
+    const float* src = (half == 0 ? a.q : a.k) + (size_t)row0 * a.ld + (size_t)h * D + c2;
+#pragma unroll
+    for (int t = 0; t < GC; ++t) xr[t] = ch_ok && t < nt ? *reinterpret_cast<const float2*>(src + (size_t)t * a.ld) : make_float2(0.f, 0.f);
+  }
+  __syncthreads();
   if (ch_ok) {
     const size_t hc = (size_t)h * D + c2;
     float z0[GB], z1[GB];
@@ -479,14 +533,10 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
     *reinterpret_cast<uint32_t*>(lo) = pl;
   };
   if (ch_ok && half == 0) {   // queries, forward
-    const float* src = a.q + (size_t)row0 * a.ld + (size_t)h * D + c2;
     float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
-#pragma unroll 8
+#pragma unroll
     for (int t = 0; t < GC; ++t) {
-      float2 x = make_float2(0.f, 0.f);
-      if (t < nt) x = *reinterpret_cast<const float2*>(src + (size_t)t * a.ld);
-      x.x *= a.q_scale;
-      x.y *= a.q_scale;
+      const float2 x = make_float2(xr[t].x * a.q_scale, xr[t].y * a.q_scale);
       *reinterpret_cast<float2*>(qs + t * LD + c2) = x;
       const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
       p0 *= f.x;
@@ -503,12 +553,10 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
     }
     *reinterpret_cast<float2*>(a.chunk_decay + (size_t)row0 * a.heads * D + (size_t)h * D + c2) = make_float2(p0, p1);
   } else if (ch_ok) {         // keys, backward
-    const float* src = a.k + (size_t)row0 * a.ld + (size_t)h * D + c2;
     float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
-#pragma unroll 8
+#pragma unroll
     for (int t = GC - 1; t >= 0; --t) {
-      float2 x = make_float2(0.f, 0.f);
-      if (t < nt) x = *reinterpret_cast<const float2*>(src + (size_t)t * a.ld);
+      const float2 x = xr[t];
       *reinterpret_cast<float2*>(ks + t * LD + c2) = x;
       const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
       if (t < nt) {
@@ -585,30 +633,35 @@ gla_chunk_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const int32_t* __
   const int n_col = min(LV, a.vdim - c0);   // a multiple of 8
   const bf* ops = reinterpret_cast<const bf*>(a.ops) + (size_t)h * W;
   const bf* vb = reinterpret_cast<const bf*>(a.vb) + (size_t)h * a.vdim + c0;
+  // a row of a chunk is `per` 16-byte pieces, a lane's are lane, lane + 32, ..: where each comes from and goes to (kind 0: none,
+  // 1: decayed queries, keys and scores, 2: values, 3: a value column past the slice -- zeros)
+  constexpr int PPL = (2 * DKS * 4 + 2 * GC / 8 + LV / 8 + 31) / 32;
+  int p_kind[PPL], p_dst[PPL], p_ld[PPL], p_src[PPL];
+#pragma unroll
+  for (int i = 0; i < PPL; ++i) {
+    const int e = lane + 32 * i, qv = D / 8, av = GC / 8;
+    p_kind[i] = p_dst[i] = p_ld[i] = p_src[i] = 0;
+    if (e < 4 * qv) {
+      p_kind[i] = 1; p_src[i] = e * 8; p_ld[i] = LDQ; p_dst[i] = e / qv * GC * LDQ + e % qv * 8;
+    } else if (e < 4 * qv + 2 * av) {
+      const int x = e - 4 * qv;
+      p_kind[i] = 1; p_src[i] = e * 8; p_ld[i] = LDGA; p_dst[i] = GC * (4 * LDQ + LDV_) + x / av * GC * LDGA + x % av * 8;
+    } else if (e < 4 * qv + 2 * av + LV / 8) {
+      const int c = (e - 4 * qv - 2 * av) * 8;
+      p_kind[i] = c < n_col ? 2 : 3; p_src[i] = c; p_ld[i] = LDV_; p_dst[i] = GC * 4 * LDQ + c;
+    }
+  }
   auto fetch = [&](int t0, int buf) {   // rows up to the next multiple of 16 and columns past the slice are zeros
-    const int nt = min(GC, sq.q_len - t0), qv = D / 8, av = GC / 8, per = 4 * qv + 2 * av + LV / 8;
+    const int nt = min(GC, sq.q_len - t0);
     bf* B = RB + buf * ring;
+    const bf* o_row = ops + (size_t)(sq.q_start + t0) * a.heads * W;
+    const bf* v_row = vb + (size_t)(sq.q_start + t0) * a.heads * a.vdim;
     for (int t = warp; t < (nt + 15) / 16 * 16; t += L_THREADS / 32) {
-      const size_t row = (size_t)(sq.q_start + t0 + t);
-      for (int e = lane; e < per; e += 32) {
-        bf* dst;
-        const bf* src;
-        bool ok = t < nt;
-        if (e < 4 * qv) {
-          const int m = e / qv, c = (e - m * qv) * 8;
-          dst = B + (size_t)(m * GC + t) * LDQ + c;
-          src = ops + row * a.heads * W + e * 8;
-        } else if (e < 4 * qv + 2 * av) {
-          const int x = e - 4 * qv, m = x / av, c = (x - m * av) * 8;
-          dst = B + GC * (4 * LDQ + LDV_) + (size_t)(m * GC + t) * LDGA + c;
-          src = ops + row * a.heads * W + e * 8;
-        } else {
-          const int c = (e - 4 * qv - 2 * av) * 8;
-          dst = B + GC * 4 * LDQ + (size_t)t * LDV_ + c;
-          src = vb + row * a.heads * a.vdim + c;
-          ok = ok && c < n_col;
-        }
-        if (ok) l_cp_async16(dst, src);
+#pragma unroll
+      for (int i = 0; i < PPL; ++i) {
+        if (p_kind[i] == 0) continue;
+        bf* dst = B + p_dst[i] + t * p_ld[i];
+        if (t < nt && p_kind[i] < 3) l_cp_async16(dst, (p_kind[i] == 1 ? o_row + (size_t)t * a.heads * W : v_row + (size_t)t * a.heads * a.vdim) + p_src[i]);
         else *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
       }
     }
@@ -774,6 +827,10 @@ cudaError_t rotary_rows_launch(const RotaryRows& a, int T, cudaStream_t stream) 
   if (T <= 0) return cudaSuccess;
   if (a.heads < 1 || a.dim < 1 || a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims & 1) || (a.rot_dims > 0 && a.cos_sin == nullptr))
     return cudaErrorInvalidValue;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (a.dim % 8 == 0 && a.rot_dims % 8 == 0 && a.vdim % 8 == 0 && a.ld % 4 == 0 && a.q_off % 4 == 0 && a.k_off % 4 == 0 && a.v_off % 4 == 0 &&
+      a.cast_ld % 8 == 0 && al16(a.x) && al16(a.cast) && al16(a.cos_sin))
+    return launch_k(rotary_rows_vec_kernel, dim3(T, std::min((a.heads * (2 * a.dim + a.vdim) + 2047) / 2048, 8)), dim3(256), 0, stream, a);
   return launch_k(rotary_rows_kernel, dim3(T, std::min((a.heads * a.dim + 511) / 512, 8)), dim3(256), 0, stream, a);
 }
 

@@ -646,6 +646,56 @@ head_norm_gate_kernel(const float* __restrict__ o, int ldo, int heads, int vdim,
   }
 }
 
+// the same for heads of a multiple of four values (<= 512) whose rows start on 16-byte boundaries: four values per lane and step, kept
+// in registers between the two passes
+constexpr int HNG_V = 4;
+__global__ void __launch_bounds__(128)
+head_norm_gate_vec_kernel(const float* __restrict__ o, int ldo, int heads, int vdim, const float* __restrict__ w,
+                          const float* __restrict__ gate, int ldg, int act, float eps, void* __restrict__ out, int out_dtype,
+                          int out_ld, float mult) {
+  griddep_launch();
+  griddep_wait();
+  const int t = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= heads) return;
+  const float* orow = o + (size_t)t * ldo + (size_t)h * vdim;
+  const float* grow = act != 2 ? gate + (size_t)t * ldg + (size_t)h * vdim : nullptr;
+  float4 v[HNG_V], g[HNG_V];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < HNG_V; ++j) {
+    const int i = (j * 32 + lane) * 4;
+    v[j] = i < vdim ? *reinterpret_cast<const float4*>(orow + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (grow != nullptr && i < vdim) g[j] = *reinterpret_cast<const float4*>(grow + i);
+    ss = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, ss))));
+  }
+  const float rs = mult / sqrtf(warp_sum_f(ss) / (float)vdim + eps);
+#pragma unroll
+  for (int j = 0; j < HNG_V; ++j) {
+    const int i = (j * 32 + lane) * 4;
+    if (i >= vdim) break;
+    float r[4] = {v[j].x * rs, v[j].y * rs, v[j].z * rs, v[j].w * rs};
+    if (w != nullptr) {
+      const float4 x = *reinterpret_cast<const float4*>(w + (size_t)h * vdim + i);
+      r[0] *= x.x; r[1] *= x.y; r[2] *= x.z; r[3] *= x.w;
+    }
+    if (grow != nullptr) {
+      const float z[4] = {g[j].x, g[j].y, g[j].z, g[j].w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) r[e] *= act == 1 ? silu_f(z[e]) : sigmoid_f(z[e]);
+    }
+    const size_t at = (size_t)t * out_ld + (size_t)h * vdim + i;
+    if (out_dtype == DT_BF16) {
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(r[0], r[1]), hi = __floats2bfloat162_rn(r[2], r[3]);
+      uint2 pk;
+      pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+      pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+      *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(out) + at) = pk;
+    } else {
+      *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + at) = make_float4(r[0], r[1], r[2], r[3]);
+    }
+  }
+}
+
 // wide groups (a whole row normed as one or a few groups): grid (T, heads), 256 threads, one CTA per (token, group)
 __global__ void __launch_bounds__(256)
 head_norm_gate_wide_kernel(const float* __restrict__ o, int ldo, int heads, int vdim, const float* __restrict__ w,
@@ -777,11 +827,17 @@ cudaError_t head_norm_gate_launch(const float* o, int ldo, int heads, int vdim, 
   if (T <= 0) return cudaSuccess;
   if (act == 2) gate_first = 0;
   else if (gate == nullptr) return cudaErrorInvalidValue;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  if (out_ld <= 0) out_ld = heads * vdim;
+  if (gate_first == 0 && vdim % 4 == 0 && vdim <= 128 * HNG_V && ldo % 4 == 0 && out_ld % 4 == 0 && al16(o) && al16(w) && al16(out) &&
+      (act == 2 || (ldg % 4 == 0 && al16(gate))))
+    return launch_k(head_norm_gate_vec_kernel, dim3(T, (heads + 3) / 4), dim3(128), 0, stream, o, ldo, heads, vdim, w, gate, ldg, act, eps,
+                    out, out_dtype, out_ld, mult);
   if (vdim >= 1024 && heads <= 65535)
     return launch_k(head_norm_gate_wide_kernel, dim3(T, heads), dim3(256), 0, stream, o, ldo, heads, vdim, w, gate, ldg, act, eps, out,
-                    out_dtype, out_ld > 0 ? out_ld : heads * vdim, gate_first, mult);
+                    out_dtype, out_ld, gate_first, mult);
   return launch_k(head_norm_gate_kernel, dim3(T, (heads + 3) / 4), dim3(128), 0, stream, o, ldo, heads, vdim, w, gate, ldg, act,
-                  eps, out, out_dtype, out_ld > 0 ? out_ld : heads * vdim, gate_first, mult);
+                  eps, out, out_dtype, out_ld, gate_first, mult);
 }
 
 cudaError_t conv_state_save_launch(const float* x, int ld, int n, int taps, const AttnSeq* seqs, int n_seqs,
