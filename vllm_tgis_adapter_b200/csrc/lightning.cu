@@ -397,7 +397,7 @@ constexpr int GC = GLA_CHUNK, GB = 16, G_THREADS = 128;
 static_assert(GC == 2 * GB, "one off-diagonal block per chunk");
 constexpr int LDGA = GC + 8;
 
-__device__ __forceinline__ float l_logsigmoid(float z) { return z >= 0.f ? -log1pf(expf(-z)) : z - log1pf(expf(z)); }
+__device__ __forceinline__ float l_logsigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
 
 // lane l leaves with the sum over all lanes of v[l]
 __device__ __forceinline__ float reduce32(float (&v)[32], int lane) {
@@ -455,8 +455,7 @@ __device__ __forceinline__ void gla_block_scores(const float* q, const float* k,
         const float tot = reduce32(v, lane);
         const int mine = p - n + lane;   // the pair whose sum this lane holds
         if (mine < P1) {
-          int r = 0;
-          while ((r + 1) * (r + 2) / 2 <= mine) ++r;
+          const int r = (int)((sqrtf(8.f * (float)mine + 1.f) - 1.f) * 0.5f);   // (exact: 8 p + 1 is a square where r steps)
           A[r * lda + r - (mine - r * (r + 1) / 2)] = tot;
         }
       }
@@ -466,7 +465,7 @@ __device__ __forceinline__ void gla_block_scores(const float* q, const float* k,
 
 // grid (16-token tiles, heads): the CTA of a tile whose first token opens a chunk of its portion takes the chunk's GC tokens
 template <int DPL>
-__global__ void __launch_bounds__(G_THREADS)
+__global__ void __launch_bounds__(G_THREADS, 3)
 gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* __restrict__ tiles, int first_seq) {
   extern __shared__ __align__(16) uint8_t g_smem[];
   griddep_launch();
@@ -485,18 +484,30 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
   bf* qll = qlh + GB * LDQ;
   bf* klh = qll + GB * LDQ;                       // [GB][LDQ] first block's keys decayed to its end
   bf* kll = klh + GB * LDQ;
-  float* a1s = reinterpret_cast<float*>(qlh);     // [GC][R], consumed before qlh is written
-  for (int i = tid; i < GC * R; i += G_THREADS) {
-    const int t = i / R;
-    a1s[i] = t < nt ? a.a1[(size_t)(row0 + t) * a.ld + i % R] : 0.f;
-  }
+  float* a1s = reinterpret_cast<float*>(qlh);     // [R][GC], consumed before qlh is written, and
+  float* a2s = a1s + R * GC;                      // [R][D + 2]
+  // (read-only inputs through __ldg: their loads may pass the stores)
   const int c2 = (tid & 63) * 2, half = tid >> 6;   // two channels; half 0: tokens 0..15 / queries, half 1: tokens 16..31 / keys
   const bool ch_ok = c2 < D;
-  float2 xr[GC];   // this thread's two channels of the chunk's queries or keys: on their way while the decays are made
   {
+    float2 xr[GC];
     const float* src = (half == 0 ? a.q : a.k) + (size_t)row0 * a.ld + (size_t)h * D + c2;
 #pragma unroll
-    for (int t = 0; t < GC; ++t) xr[t] = ch_ok && t < nt ? *reinterpret_cast<const float2*>(src + (size_t)t * a.ld) : make_float2(0.f, 0.f);
+    for (int t = 0; t < GC; ++t) xr[t] = ch_ok && t < nt ? __ldg(reinterpret_cast<const float2*>(src + (size_t)t * a.ld)) : make_float2(0.f, 0.f);
+#pragma unroll 4
+    for (int i = tid; i < GC * R; i += G_THREADS) {
+      const int t = i / R;
+      a1s[(i % R) * GC + t] = t < nt ? __ldg(a.a1 + (size_t)(row0 + t) * a.ld + i % R) : 0.f;
+    }
+    const uint16_t* w2 = reinterpret_cast<const uint16_t*>(a.a2) + (size_t)h * D * R;
+#pragma unroll 8
+    for (int i = tid; i < D * R; i += G_THREADS) a2s[(i % R) * (D + 2) + i / R] = __uint_as_float((uint32_t)__ldg(w2 + i) << 16);
+    if (ch_ok) {
+      float* dst = (half == 0 ? qs : ks) + c2;
+      const float m = half == 0 ? a.q_scale : 1.f;
+#pragma unroll
+      for (int t = 0; t < GC; ++t) *reinterpret_cast<float2*>(dst + t * LD) = make_float2(xr[t].x * m, xr[t].y * m);
+    }
   }
   __syncthreads();
   if (ch_ok) {
@@ -505,14 +516,15 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
     const float b0 = a.bias[hc], b1 = a.bias[hc + 1];
 #pragma unroll
     for (int t = 0; t < GB; ++t) { z0[t] = b0; z1[t] = b1; }
-    const bf *w0 = reinterpret_cast<const bf*>(a.a2) + hc * R, *w1 = w0 + R;
     for (int r = 0; r < R; ++r) {
-      const float x0 = __bfloat162float(w0[r]), x1 = __bfloat162float(w1[r]);
+      const float2 x = *reinterpret_cast<const float2*>(a2s + r * (D + 2) + c2);
 #pragma unroll
-      for (int t = 0; t < GB; ++t) {
-        const float y = a1s[(half * GB + t) * R + r];
-        z0[t] = fmaf(y, x0, z0[t]);
-        z1[t] = fmaf(y, x1, z1[t]);
+      for (int t = 0; t < GB; t += 4) {
+        const float4 y = *reinterpret_cast<const float4*>(a1s + r * GC + half * GB + t);
+        z0[t] = fmaf(y.x, x.x, z0[t]); z1[t] = fmaf(y.x, x.y, z1[t]);
+        z0[t + 1] = fmaf(y.y, x.x, z0[t + 1]); z1[t + 1] = fmaf(y.y, x.y, z1[t + 1]);
+        z0[t + 2] = fmaf(y.z, x.x, z0[t + 2]); z1[t + 2] = fmaf(y.z, x.y, z1[t + 2]);
+        z0[t + 3] = fmaf(y.w, x.x, z0[t + 3]); z1[t + 3] = fmaf(y.w, x.y, z1[t + 3]);
       }
     }
 #pragma unroll
@@ -534,10 +546,9 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
   };
   if (ch_ok && half == 0) {   // queries, forward
     float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
-#pragma unroll
+#pragma unroll 4
     for (int t = 0; t < GC; ++t) {
-      const float2 x = make_float2(xr[t].x * a.q_scale, xr[t].y * a.q_scale);
-      *reinterpret_cast<float2*>(qs + t * LD + c2) = x;
+      const float2 x = *reinterpret_cast<const float2*>(qs + t * LD + c2);
       const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
       p0 *= f.x;
       p1 *= f.y;
@@ -554,10 +565,9 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
     *reinterpret_cast<float2*>(a.chunk_decay + (size_t)row0 * a.heads * D + (size_t)h * D + c2) = make_float2(p0, p1);
   } else if (ch_ok) {         // keys, backward
     float p0 = 1.f, p1 = 1.f, l0 = 1.f, l1 = 1.f;
-#pragma unroll
+#pragma unroll 4
     for (int t = GC - 1; t >= 0; --t) {
-      const float2 x = xr[t];
-      *reinterpret_cast<float2*>(ks + t * LD + c2) = x;
+      const float2 x = *reinterpret_cast<const float2*>(ks + t * LD + c2);
       const float2 f = *reinterpret_cast<const float2*>(fs + t * LD + c2);
       if (t < nt) {
         bf* o = ops + ((size_t)(row0 + t) * a.heads + h) * W + 2 * D + c2;
@@ -572,11 +582,17 @@ gla_prep_kernel(GlaChunk a, const AttnSeq* __restrict__ seqs, const LatentTile* 
       }
     }
   }
-  for (int i = tid; i < nt * (a.vdim / 2); i += G_THREADS) {   // the values, rounded once
-    const int t = i / (a.vdim / 2), c = i % (a.vdim / 2) * 2;
-    const float2 x = *reinterpret_cast<const float2*>(a.v + (size_t)(row0 + t) * a.ld + (size_t)h * a.vdim + c);
-    *reinterpret_cast<__nv_bfloat162*>(reinterpret_cast<bf*>(a.vb) + (size_t)(row0 + t) * a.heads * a.vdim + (size_t)h * a.vdim + c) =
-        __floats2bfloat162_rn(x.x, x.y);
+  const int v4 = a.vdim / 4;
+#pragma unroll 4
+  for (int i = tid; i < nt * v4; i += G_THREADS) {   // the values, rounded once
+    const int t = i / v4, c = i % v4 * 4;
+    const float* src = a.v + (size_t)(row0 + t) * a.ld + (size_t)h * a.vdim + c;
+    const float2 x = __ldg(reinterpret_cast<const float2*>(src)), y = __ldg(reinterpret_cast<const float2*>(src + 2));
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(x.x, x.y), hi = __floats2bfloat162_rn(y.x, y.y);
+    uint2 pk;
+    pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+    pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(reinterpret_cast<bf*>(a.vb) + (size_t)(row0 + t) * a.heads * a.vdim + (size_t)h * a.vdim + c) = pk;
   }
   __syncthreads();
   // ---- scores: warps 0 and 1 the first block (rows 0..10 | 11..15: as many pairs each), warps 2 and 3 the second
@@ -789,12 +805,12 @@ template <int DKS>
 cudaError_t launch_gla(const GlaChunk& a, const AttnSeq* seqs, int first_seq, int n_seqs, const LatentTile* tiles, int n_tiles,
                        const int32_t* tok_slot, cudaStream_t stream) {
   constexpr int DPL = DKS <= 4 ? 2 : 4;
-  const size_t tail = std::max((size_t)4 * GB * (a.dim + 8) * sizeof(bf), (size_t)GC * a.rank * sizeof(float));
-  const size_t smem_p = ((size_t)3 * GC * (a.dim + 4) + GC * (GC + 1)) * sizeof(float) + tail;                       // <= 73 KB
+  const size_t tail = std::max((size_t)4 * GB * (a.dim + 8) * sizeof(bf), (size_t)a.rank * (GC + a.dim + 2) * sizeof(float));
+  const size_t smem_p = ((size_t)3 * GC * (a.dim + 4) + GC * (GC + 1)) * sizeof(float) + tail;                       // <= 97 KB (73 KB up to a rank of 26)
   const size_t smem_c = (size_t)2 * GC * (4 * (a.dim + 8) + LDV_ + 2 * LDGA) * sizeof(bf) + (size_t)2 * a.dim * sizeof(float);   // <= 90 KB
   static bool attr_set = false;
   if (!attr_set) {
-    cudaError_t e = cudaFuncSetAttribute(gla_prep_kernel<DPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
+    cudaError_t e = cudaFuncSetAttribute(gla_prep_kernel<DPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
     if (e == cudaSuccess) e = cudaFuncSetAttribute(gla_chunk_kernel<DKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024);
     if (e != cudaSuccess) return e;
     attr_set = true;
