@@ -190,7 +190,7 @@ typedef struct tgis_config {
 #define TGIS_LAYER_QKV_BIAS 8        /* "l<i>.mix.q.b|k.b|v.b" are added to the projections */
 #define TGIS_LAYER_UNIT_QK 16        /* queries and keys are divided by their root mean square per head after the rotation */
 #define TGIS_LAYER_OUT_BIAS 32       /* the attention's output projection has a bias: "o.b" */
-#define TGIS_LAYER_SHARED_KV 64      /* no value projection: values are the keys as projected (bias included, before norm and rotation) */
+#define TGIS_LAYER_SHARED_KV 64      /* one projection serves keys and values: the value row is its biased output, the key row that output normed and turned */
 #define TGIS_LAYER_FULL_QK_NORM 128  /* queries and keys are rms-normed over all heads at once before the rotation ("q.norm", "k.norm") */
 #define TGIS_LAYER_HEAD_GATE 256     /* head h's output times sigmoid(W_g h)_h ("g": [heads, width]) */
 typedef struct tgis_layer_spec {

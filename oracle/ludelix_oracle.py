@@ -112,7 +112,7 @@ def attend(q, k, v, mask, scale: float, sink=None) -> torch.Tensor:
 
 
 def shared_attention(h: torch.Tensor, w: dict, m: dict, eps: float) -> torch.Tensor:
-    """Sliding-window attention whose values are the keys as projected (bias included, before norm and rotation)."""
+    """Sliding-window attention with one projection for keys and values: the value is its biased output, the key that output normed and turned."""
     T = h.shape[0]
     H, G, d = int(m["heads"]), int(m["kv_heads"]), int(m["dim"])
     q, k = h @ w["q"].T + w["q.b"], h @ w["k"].T + w["k.b"]

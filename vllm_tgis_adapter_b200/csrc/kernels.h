@@ -458,8 +458,8 @@ struct PoolAttnGeom {
 constexpr int POOLATTN_TILE = 16;      // query tokens per CTA
 constexpr int POOLATTN_MAX_VDIM = 512; // value columns per head the FMA kernel's accumulators cover
 // y fp32 [T, ldy] holds q at column q_off (heads * dim), k at k_off (kv_heads * dim), v at v_off (kv_heads * vdim); bias fp32
-// (q | k | v, in that order, or nullptr) is added first.  v_off == k_off: the values ARE the keys as projected (bias included, before
-// any norm and rotation; dim == vdim, bias holds q | k).  cos_sin fp32 [max_pos][rot_dims] = cos | sin.  q_out DT_* [T, heads * dim];
+// (q | k | v, in that order, or nullptr) is added first.  v_off == k_off: keys and values share one projection; the value is its biased output (not the normed and turned
+// key; dim == vdim, bias holds q | k).  cos_sin fp32 [max_pos][rot_dims] = cos | sin.  q_out DT_* [T, heads * dim];
 // cache rows K [num_blocks][KV_BLOCK][kv_heads * dim], V [..][kv_heads * vdim] at slot[t].
 cudaError_t poolattn_prep_launch(const float* y, int ldy, int q_off, int k_off, int v_off, const float* bias,
                                  const PoolAttnGeom& g, const float* cos_sin, float eps, const int32_t* positions,
